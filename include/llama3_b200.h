@@ -69,7 +69,7 @@ int l3_load_weight(L3Model* m, const char* key, const float* host, const int64_t
 /* Random-init on the device for shapes that are impractical to build on the host
  * (8B-shaped benches).  Same scales as synth.make_weights, different stream of numbers. */
 int l3_fill_random(L3Model* m, uint64_t seed);
-/* Packed device-layout weight cache (SURVEY.md 8(f)-3; replaces a repeat of np.load + per-tensor packing,
+/* Packed device-layout weight cache (replaces a repeat of np.load + per-tensor packing,
  * llama3.py:269 / utils.py:4-5, on the second and later starts).  l3_save_packed writes the weight matrices
  * exactly as they sit on the device after the l3_load_weight calls (fused q|k|v rows, interleaved gate/up rows,
  * this rank's tensor-parallel slices, model dtype) to `path` (atomically: temp file + rename) together with
@@ -146,8 +146,11 @@ int l3_generate_ragged(L3Model* m, const int32_t* ids, const int32_t* lens, int 
 #define L3_MIX_LATENT 3        /* causal softmax attention over ONE cached latent row per token: queries through a
                                   normed latent of width q_rank; the cache row is [normed latent (kv_rank) | rotated key
                                   part (rot_dim)] shared by all heads; per-head keys / values are expanded from the latent
-                                  (here: folded into the query and the output); rotary pairs (2i, 2i + 1) on the first
-                                  rot_dims entries of the rotated part; sigmoid gate per head                          */
+                                  (here: folded into the query and the output); rotary positions on the first rot_dims
+                                  entries of the rotated part (rot_layout as below); a sigmoid gate per head, or per value
+                                  (gate_wide); sink 1: the softmax denominator also holds exp(sink_h) (tensor mix.sink
+                                  [heads]); kv_source j > 0: the layer has no key / value latent of its own and attends over
+                                  the cache rows of layer j - 1                                                          */
 #define L3_MIX_MINGRU 4        /* element-wise gated recurrence of width dim (heads = vdim = 1):
                                   S <- (1 - z) S + z c,  z = sigmoid(Wz h + bz),  c = u + 1/2 (u >= 0) | sigmoid(u),
                                   u = Wx h + bx;  output Wo (S * silu(Wg h))                                            */
@@ -181,6 +184,7 @@ int l3_generate_ragged(L3Model* m, const int32_t* ids, const int32_t* lens, int 
 #define L3_ATTN_SIGMOID 1
 /* feed-forward kinds (L3LayerSpec::ff_kind) */
 #define L3_FF_GLU 0            /* down(act(gate x) * (up x)), act = L3StackConfig::glu_act; experts: down relu(up x)^2 */
+#define L3_FF_RELU2 2          /* down(relu(up x)^2), no gate matrix */
 #define L3_FF_POLYNORM 1       /* down(P(up x)),  P(z) = a N(z) + b N(z^2) + c N(z^3) + e with element-wise powers and
                                   N(v) = v / sqrt(mean(v^2) + eps) over the ff values of a token; tensor l<i>.mlp.act = (a, b, c, e) */
 /* router kinds (L3LayerSpec::router_kind) */
@@ -221,7 +225,7 @@ typedef struct L3LayerSpec {
   int32_t ff_kind;           /* L3_FF_* of the dense feed-forward */
   int32_t router_kind;       /* L3_ROUTE_* of the mixture of experts */
   int32_t shared_ff;         /* L3_ROUTE_SIGMOID_IN: width of the shared expert; 0 = none */
-  /* L3_MIX_WINDOW (also uses heads, kv_heads, dim, vdim, scale, window, rot_dims, rot_base) */
+  /* L3_MIX_WINDOW (also uses heads, kv_heads, dim, vdim, scale, window, rot_dims, rot_base); rot_layout: L3_MIX_LATENT, too */
   int32_t keep_first;        /* the first keep_first tokens stay visible behind the window */
   int32_t attn_kind;         /* L3_ATTN_* */
   int32_t rot_layout;        /* 0: entry 2i turns with 2i + 1; 1: entry i with i + rot_dims / 2 */
@@ -233,6 +237,11 @@ typedef struct L3LayerSpec {
    * l<i>.mix.left.*, the second's l<i>.mix.right.*; of the pair spec only the mixer fields are read (no ff, no pair). */
   const struct L3LayerSpec* pair;
   float mix_scale, pair_scale;
+  /* L3_MIX_LATENT */
+  int32_t kv_source;         /* 0: own cache rows; j + 1: those of layer j, which has rows of its own and comes first; its
+                                kv_rank, rot_dim, rot_dims, rot_base and rot_layout must be this layer's (no mix.dkv here) */
+  int32_t sink;              /* 1: a learned logit per head in the softmax denominator (tensor mix.sink) */
+  int32_t gate_wide;         /* 1: mix.g has heads * vdim rows and gates value by value; 0: heads rows */
 } L3LayerSpec;
 
 typedef struct L3StackConfig {
@@ -256,7 +265,7 @@ typedef struct L3StackConfig {
   /* parallel layers (needs norm_input): ONE norm per layer, h = norm1(x), and both sublayers read it:
    *   X_(i+1) = x + ls1 * mixer(h + conv1(h)) + ls2 * ff(h + conv2(h))
    * norm_center 1: the norms (layer norms and the final norm) subtract the mean first (layer norm with a weight, no bias);
-   * layer_scale 1: tensors l<i>.ls1 / ls2 [width] multiply the sublayers' results (0: ones);
+   * layer_scale 1 (pre-norm stacks, too): tensors l<i>.ls1 / ls2 [width] multiply the sublayers' results (0: ones);
    * canon_taps T > 0: every sublayer reads h + conv(h), conv(h)_t = sum_j w[:, j] h_(t - T + 1 + j), a causal convolution
    *   over time per channel (tensors l<i>.canon1 / canon2 [width, T], zeros ahead of position 0; the last T - 1 rows of h
    *   are kept per sequence slot and layer run);
@@ -271,6 +280,16 @@ typedef struct L3StackConfig {
    * logit_softcap c > 0: logits <- c tanh(logits / c). */
   int32_t norm_groups, embed_norm, loop_in;
   float logit_softcap;
+  /* pre-norm stacks without loop, token shift or grouped norms:
+   * streams S > 0: S residual rows X_1 .. X_S per token, all equal to the embedding output at first.  Sublayer q (1 the mixer,
+   *   2 the feed-forward) reads u = sum_s in[s] X_s ahead of its norm, and its result y (times ls<q> with layer_scale) moves
+   *   all of them at once: X_t <- sum_s mix[s, t] X_s + out[t] y (tensors l<i>.hc<q>.in [S], .out [S], .mix [S, S], indexed
+   *   [from, to]).  The final norm reads the sum of the streams, and so does the residual trace of l3_forward_rows.
+   *   0: one residual row, x <- x + y; layer_scale 1 works with either.
+   * tied_head 1: the output projection is the embedding table (no tensor "head"; without embed_scale);
+   * logit_scale: multiplier of the logits, ahead of the soft cap; 0 = 1. */
+  int32_t streams, tied_head;
+  float logit_scale;
 } L3StackConfig;
 
 int l3_create_stack(const L3StackConfig* cfg, const L3LayerSpec* layers, L3Model** out);
@@ -359,7 +378,7 @@ int l3_bench_gemv(int device, int n, int k, int w_bf16, int rows, int iters, flo
  * tcgen05.mma of M = 128, K = 32 bytes, width n (16..256), kind 0 = bf16 / 1 = tf32, issued by one thread
  * rotating over nacc TMEM accumulators (nacc * n <= 512), `iters` groups of four, on `ctas` CTAs at once.
  * cycles_per_mma[0] = issue loop, [1] = issue + completion (maximum over the CTAs).  No reference
- * counterpart: a design input for the GEMM kernels (DESIGN.md 6). */
+ * counterpart: a design input for the GEMM kernels. */
 int l3_probe_mma(int device, int kind, int n, int nacc, int iters, int ctas, double* cycles_per_mma);
 
 #ifdef __cplusplus

@@ -27,7 +27,7 @@ class L3Config(C.Structure):
 MIX_SOFTMAX, MIX_DECAY_LINEAR, MIX_GATED_DELTA, MIX_LATENT, MIX_MINGRU, MIX_DIFF = 0, 1, 2, 3, 4, 5
 MIX_WINDOW, MIX_SSD, MIX_GLA = 6, 7, 8
 ATTN_SINK, ATTN_SIGMOID = 0, 1
-FF_GLU, FF_POLYNORM = 0, 1
+FF_GLU, FF_POLYNORM, FF_RELU2 = 0, 1, 2
 ROUTE_SOFTMAX, ROUTE_SIGMOID_IN = 0, 1
 GLU_SILU, GLU_GELU_TANH = 0, 1
 
@@ -48,7 +48,8 @@ L3LayerSpec._fields_ = [("mixer", C.c_int32), ("heads", C.c_int32), ("kv_heads",
                 ("router_kind", C.c_int32), ("shared_ff", C.c_int32),
                 ("keep_first", C.c_int32), ("attn_kind", C.c_int32), ("rot_layout", C.c_int32), ("qk_unit", C.c_int32),
                 ("out_norm_groups", C.c_int32), ("tau", C.c_float), ("pair", C.POINTER(L3LayerSpec)),
-                ("mix_scale", C.c_float), ("pair_scale", C.c_float)]
+                ("mix_scale", C.c_float), ("pair_scale", C.c_float),
+                ("kv_source", C.c_int32), ("sink", C.c_int32), ("gate_wide", C.c_int32)]
 
 
 class L3StackConfig(C.Structure):
@@ -60,7 +61,7 @@ class L3StackConfig(C.Structure):
                 ("embed_scale", C.c_float), ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32),
                 ("parallel", C.c_int32), ("norm_center", C.c_int32), ("layer_scale", C.c_int32), ("canon_taps", C.c_int32),
                 ("depth_avg", C.c_int32), ("norm_groups", C.c_int32), ("embed_norm", C.c_int32), ("loop_in", C.c_int32),
-                ("logit_softcap", C.c_float)]
+                ("logit_softcap", C.c_float), ("streams", C.c_int32), ("tied_head", C.c_int32), ("logit_scale", C.c_float)]
 
 
 _P = C.c_void_p

@@ -4,14 +4,16 @@
 // q~_j . [c | k_r] and the output Wuv_j (sum_i p_i c_i): attention runs on the cache rows themselves, all heads
 // of a token against the same rows, the value of a row being its first kv_rank entries.
 //
-//  * latent_prep_kernel        norms of the two latents, rotation of k_r, cache append (one CTA per token)
-//  * latent_q_rope_kernel      rotated query part into the folded query
+//  * latent_prep_kernel        norms of the two latents, rotation of k_r, cache append (one CTA per token); the query latent
+//                              alone for a layer that reads another layer's cache
 //  * head_gemm_kernel          batched per-head product (Wuk_j^T q_c and Wuv_j ctx): 64 x 64 FFMA tiles, 4 x 4 per thread;
-//                              head_gemv_kernel for up to 8 rows (decode)
+//                              head_gemv_kernel for up to 8 rows (decode).  The launch that folds the queries also turns
+//                              their rotated part; the one that expands the values also applies an element-wise gate
 //  * attn_latent_kernel        flash-style exact attention: a CTA holds 32 (token, head) query rows in shared memory
 //                              and walks the visible cache rows 32 at a time; a lane scores one key for its warp's
 //                              four query rows, then the lanes own output columns.  Scores, weights and sums fp32.
-//                              Decode splits the keys over CTAs; attn_latent_combine_kernel merges the parts.
+//                              Decode splits the keys over CTAs; attn_latent_combine_kernel merges the parts.  A sink
+//                              (one logit per head without a value) joins the denominator once, at the very end.
 #include <algorithm>
 
 #include "common.cuh"
@@ -30,13 +32,19 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return t;
 }
 
-// pair (u, v) of entries (2i, 2i + 1) at position pos: (u cos a - v sin a, v cos a + u sin a), a = pos * f_i in fp32
-__device__ __forceinline__ void rotate_pair(float u, float v, int pos, float f, float& ru, float& rv) {
-  const float ang = (float)pos * f;
+// dst = src with its first `dims` entries turned at position pos: the pair (u, v) of entries (2i, 2i + 1) (layout 0) or
+// (i, i + dims / 2) (layout 1) becomes (u cos a - v sin a, v cos a + u sin a), a = pos * f_i in fp32.  Work item i: pair i,
+// or for i >= dims / 2 the unchanged entry i + dims / 2.
+template <typename T>
+__device__ __forceinline__ void rotate_item(const float* src, T* dst, int i, int dims, int layout, int pos, const float* __restrict__ freq) {
+  const int half = dims >> 1;
+  if (i >= half) { dst[i + half] = from_f32<T>(src[i + half]); return; }
+  const int iu = layout ? i : 2 * i, iv = layout ? i + half : 2 * i + 1;
+  const float u = src[iu], v = src[iv];
   float sn, cs;
-  sincosf(ang, &sn, &cs);
-  ru = u * cs - v * sn;
-  rv = v * cs + u * sn;
+  sincosf((float)pos * freq[i], &sn, &cs);
+  dst[iu] = from_f32<T>(u * cs - v * sn);
+  dst[iv] = from_f32<T>(v * cs + u * sn);
 }
 
 template <typename KVT>
@@ -56,6 +64,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrepArgs a) {
     a.cq[(size_t)r * a.q_rank + i] = v;
     if (a.cq16) a.cq16[(size_t)r * a.q_rank + i] = __float2bfloat16_rn(v);
   }
+  if (a.k_off < 0) return;
   const float* kv = row + a.k_off;
   ss = 0.f;
   for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) { const float v = kv[i]; ss = fmaf(v, v, ss); }
@@ -63,42 +72,26 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrepArgs a) {
   KVT* dst = (KVT*)a.cache + ((size_t)b * a.M + pos) * (a.kv_rank + a.rot_dim);
   for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) dst[i] = from_f32<KVT>(kv[i] * rk * a.wk[i]);
   const float* kr = kv + a.kv_rank;
-  for (int i = threadIdx.x; i < a.rot_dims / 2; i += blockDim.x) {
-    float ru, rv;
-    rotate_pair(kr[2 * i], kr[2 * i + 1], pos, a.inv_freq[i], ru, rv);
-    dst[a.kv_rank + 2 * i] = from_f32<KVT>(ru);
-    dst[a.kv_rank + 2 * i + 1] = from_f32<KVT>(rv);
-  }
-  for (int i = a.rot_dims + threadIdx.x; i < a.rot_dim; i += blockDim.x) dst[a.kv_rank + i] = from_f32<KVT>(kr[i]);
-}
-
-__global__ void latent_q_rope_kernel(const float* __restrict__ q, float* __restrict__ qlat, const float* __restrict__ inv_freq,
-                                     const int* __restrict__ pos_ptr, int rows, int L, int H, int dim, int rot_dim, int rot_dims,
-                                     int kv_rank) {
-  pdl_launch();
-  pdl_wait();
-  const int half = (rot_dim + 1) / 2;  // work items per (row, head): one per pair, the tail entries one each
-  const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (idx >= (int64_t)rows * H * half) return;
-  const int i = (int)(idx % half);
-  const int64_t rh = idx / half;
-  const int r = (int)(rh / H);
-  const int pos = *pos_ptr + r % L;
-  const float* src = q + rh * (dim + rot_dim) + dim;
-  float* dst = qlat + rh * (kv_rank + rot_dim) + kv_rank;
-  if (2 * i + 1 < rot_dims) {
-    float ru, rv;
-    rotate_pair(src[2 * i], src[2 * i + 1], pos, inv_freq[i], ru, rv);
-    dst[2 * i] = ru;
-    dst[2 * i + 1] = rv;
-  } else {
-    dst[2 * i] = src[2 * i];
-    if (2 * i + 1 < rot_dim) dst[2 * i + 1] = src[2 * i + 1];
-  }
+  for (int i = threadIdx.x; i < a.rot_dim - a.rot_dims / 2; i += blockDim.x)
+    rotate_item(kr, dst + a.kv_rank, i, a.rot_dims, a.rot_layout, pos, a.inv_freq);
 }
 
 // ---------------------------------------------------------------- batched per-head product
 constexpr int HG_BM = 64, HG_BN = 64, HG_BK = 16;
+
+// rotated query part of rows [r0, r1), head h: C[r, h, J ..] = rot(A[r, h, K ..])
+__device__ __forceinline__ void head_rotate(const HeadGemmArgs& a, int h, int r0, int r1) {
+  const int items = a.rot_dim - a.rot_dims / 2;
+  for (int e = threadIdx.x; e < (r1 - r0) * items; e += blockDim.x) {
+    const int r = r0 + e / items, i = e % items;
+    rotate_item(a.A + (size_t)r * a.lda + (size_t)h * a.a_hs + a.K, a.C + (size_t)r * a.ldc + (size_t)h * a.c_hs + a.J, i, a.rot_dims,
+                a.rot_layout, *a.pos_ptr + r % a.L, a.inv_freq);
+  }
+}
+
+__device__ __forceinline__ float head_gate(const HeadGemmArgs& a, int r, int h, int j) {
+  return a.gate ? 1.0f / (1.0f + expf(-a.gate[(size_t)r * a.ld_gate + (size_t)h * a.c_hs + j])) : 1.0f;
+}
 
 template <typename WT>
 __global__ void __launch_bounds__(256) head_gemm_kernel(HeadGemmArgs a) {
@@ -157,10 +150,12 @@ __global__ void __launch_bounds__(256) head_gemm_kernel(HeadGemmArgs a) {
       const int jj = j0 + tx * 4 + j;
       if (jj >= a.J) continue;
       const size_t o = (size_t)r * a.ldc + (size_t)h * a.c_hs + jj;
-      a.C[o] = acc[i][j];
-      if (a.C16) a.C16[o] = __float2bfloat16_rn(acc[i][j]);
+      const float v = acc[i][j] * head_gate(a, r, h, jj);
+      if (a.C) a.C[o] = v;
+      if (a.C16) a.C16[o] = __float2bfloat16_rn(v);
     }
   }
+  if (a.rot_dim > 0 && blockIdx.y == 0) head_rotate(a, h, r0, min(r0 + HG_BM, a.rows));
 }
 
 // ---------------------------------------------------------------- attention over the latent cache
@@ -170,6 +165,17 @@ __host__ __device__ inline int la_kstride(int Dk) {
   // 16-byte loads by 8 lanes at a time want an odd stride in 16-byte units; scalar loads an odd stride in words
   if (Dk % 4 == 0) return ((Dk / 4) & 1) ? Dk : Dk + 4;
   return (Dk & 1) ? Dk : Dk + 1;
+}
+
+// What the weighted sum of values is multiplied by at the end: 1 / denominator, the sink's term included, times the head's
+// gate.  m, l: maximum and sum of exp(score - m) over the visible keys (never empty: a token sees itself).
+__device__ __forceinline__ float latent_out_scale(const LatentAttnArgs& a, size_t tok, int head, float m, float l) {
+  const float g = a.gate ? 1.0f / (1.0f + expf(-a.gate[tok * a.ld_gate + head])) : 1.0f;
+  if (!a.sink) return g / l;
+  const float sk = a.sink[head];
+  if (sk <= m) return g / (l + expf(sk - m));
+  const float c = expf(m - sk);  // the sink is the largest logit
+  return g * c / fmaf(l, c, 1.0f);
 }
 
 // ND: output columns per lane (Dv <= 32 * ND)
@@ -343,8 +349,7 @@ __global__ void __launch_bounds__(256) attn_latent_kernel(LatentAttnArgs a) {
     } else {
       const size_t tok = row / a.H;
       const int head = (int)(row - tok * a.H);
-      const float g = a.gate ? 1.0f / (1.0f + expf(-a.gate[tok * a.ld_gate + head])) : 1.0f;
-      const float inv = g / lrun[i];
+      const float inv = latent_out_scale(a, tok, head, mrun[i], lrun[i]);
 #pragma unroll
       for (int c = 0; c < ND; ++c) { const int d = lane + 32 * c; if (d < Dv) a.out[row * Dv + d] = acc[i][c] * inv; }
     }
@@ -365,8 +370,7 @@ __global__ void __launch_bounds__(128) attn_latent_combine_kernel(LatentAttnArgs
   for (int s = 0; s < a.nsplit; ++s) l = fmaf(wsplit[s], ml[2 * s + 1], l);
   const size_t tok = row / a.H;
   const int head = (int)(row - tok * a.H);
-  const float g = a.gate ? 1.0f / (1.0f + expf(-a.gate[tok * a.ld_gate + head])) : 1.0f;
-  const float inv = g / l;
+  const float inv = latent_out_scale(a, tok, head, mx, l);
   const float* po = a.part_o + row * a.nsplit * a.Dv;
   for (int d = threadIdx.x; d < a.Dv; d += blockDim.x) {
     float o = 0.f;
@@ -385,6 +389,7 @@ __global__ void __launch_bounds__(256) head_gemv_kernel(HeadGemmArgs a) {
   const int h = blockIdx.y, r = blockIdx.z, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const float* A = a.A + (size_t)r * a.lda + (size_t)h * a.a_hs;
   const WT* W = (const WT*)a.W + (size_t)h * a.w_hs;
+  if (a.rot_dim > 0 && blockIdx.x == 0) head_rotate(a, h, r, r + 1);
   float v;
   int j;
   if (a.w_ks == 1) {
@@ -405,7 +410,8 @@ __global__ void __launch_bounds__(256) head_gemv_kernel(HeadGemmArgs a) {
     v = acc;
   }
   const size_t o = (size_t)r * a.ldc + (size_t)h * a.c_hs + j;
-  a.C[o] = v;
+  v *= head_gate(a, r, h, j);
+  if (a.C) a.C[o] = v;
   if (a.C16) a.C16[o] = __float2bfloat16_rn(v);
 }
 
@@ -446,13 +452,6 @@ cudaError_t launch_latent_attn(const LatentAttnArgs& a, bool kv_bf16, cudaStream
 cudaError_t launch_latent_prep(const LatentPrepArgs& a, int rows, bool kv_bf16, cudaStream_t s) {
   if (kv_bf16) return launch_k(latent_prep_kernel<bf16>, dim3(rows), dim3(256), 0, s, a);
   return launch_k(latent_prep_kernel<float>, dim3(rows), dim3(256), 0, s, a);
-}
-
-cudaError_t launch_latent_q_rope(const float* q, float* qlat, const float* inv_freq, const int* pos_ptr, int rows, int L,
-                                 int H, int dim, int rot_dim, int rot_dims, int kv_rank, cudaStream_t s) {
-  const int64_t n = (int64_t)rows * H * ((rot_dim + 1) / 2);
-  return launch_k(latent_q_rope_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, s, q, qlat, inv_freq, pos_ptr, rows, L, H,
-                  dim, rot_dim, rot_dims, kv_rank);
 }
 
 cudaError_t launch_head_gemm(const HeadGemmArgs& a, bool w_bf16, cudaStream_t s) {

@@ -160,6 +160,13 @@ __device__ __forceinline__ unsigned long long argmax_key(float v, int idx) {
   return ((unsigned long long)b << 32) | (unsigned long long)(0xffffffffu - (uint32_t)idx);
 }
 
+// element-wise activation of a plain projection's output (EPI_STORE)
+enum UnaryAct : int { UNARY_NONE = 0, UNARY_RELU2 = 1 };
+__device__ __forceinline__ float unary_act(int kind, float v) {
+  if (kind == UNARY_RELU2) { v = fmaxf(v, 0.f); return v * v; }
+  return v;
+}
+
 struct EpiArgs {
   float* out;            // fp32 destination (STORE / RESID / SWIGLU / q of ROPE_KV); may be null
   bf16* out_bf16;        // optional bf16 mirror of `out` for tensor-core consumers; may be null
@@ -180,6 +187,7 @@ struct EpiArgs {
   int L;                 // tokens per sequence in this call: row m -> (b = m / L, t = m % L)
   int HD, HN, KVHN, M;   // head_dim, local heads, local kv heads, max_seq_len
   int act;               // SWIGLU: GluAct of the gate column (0 = silu)
+  int unary;             // STORE: UnaryAct applied to every output value
   // SWIGLU with a routing weight on the unit's INPUT: output j of row m is act(w g) * (w u) with
   // w = glu_w[m * glu_w_ld + j / glu_group] for j < glu_groups * glu_group and 1 beyond (a shared expert); w = 0 gives 0.
   const float* glu_w;    // null: no weight
@@ -196,6 +204,7 @@ template <typename KVT>
 __device__ __forceinline__ void epilogue_pair(int epi, const EpiArgs& e, int m, int col, float v0, float v1,
                                               bool has1) {
   if (epi == EPI_STORE) {
+    if (e.unary) { v0 = unary_act(e.unary, v0); v1 = unary_act(e.unary, v1); }
     const size_t o = (size_t)m * e.ld_out + col;
     const bool vec = has1 && !(e.ld_out & 1);  // col is even: 8-byte aligned pair
     if (e.out_lo) {

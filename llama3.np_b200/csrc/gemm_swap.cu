@@ -299,6 +299,10 @@ gemm_swap_kernel(const __grid_constant__ CUtensorMap tmW0, const __grid_constant
           }
         }
         if constexpr (EPI == EPI_STORE) {
+          if (e.unary) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = unary_act(e.unary, v[j]);
+          }
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const int m = c0 + j;

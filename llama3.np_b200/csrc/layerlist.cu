@@ -22,10 +22,15 @@
 //                 [latent | rotated part] row to the run's cache -> query up-projection -> queries folded onto the
 //                 latent per head (Wuk^T q) -> attention over the cache rows themselves, all heads of a token against
 //                 the same rows (attn_latent.cu), gate per head -> values out of the latent per head (Wuv o)
+//                 Variants: a layer may read ANOTHER layer's rows (kv_source: no dkv rows in its projection), the softmax may
+//                 have a sink per head, the gate may be one value per output (then applied where the values are expanded)
 //   minGRU        fused z|x|g projection -> element-wise gated recurrence (prenorm_ops.cu)
 //   and a feed-forward that is a mixture of experts (moe.cu): fp32 router -> few rows: only the chosen experts' weights
 //   are read; many rows: ONE up-projection over all experts, relu^2 times the routing weight (zero where not chosen),
 //   ONE down-projection whose K runs over all experts and so sums them.
+//   or dense: a gated unit, or down(relu(up x)^2) with the square in the up projection's epilogue.
+// With residual streams (L3StackConfig::streams, stream_ops.cu) the sublayers' output projections store their result and one
+// launch per sublayer border re-mixes the S residual rows of a token and forms the next sublayer's normed input.
 // Parallel stacks (L3StackConfig::parallel, ll_enqueue_parallel):  h = norm1(x);  X_new = x + ls1 mixer(h + conv1(h)) +
 // ls2 ff(h + conv2(h));  x <- sum_j dwa[j] X_j over the embedding output and every layer result so far.  One mixer:
 //
@@ -93,7 +98,10 @@ static int check_spec(const L3StackConfig* c, const L3LayerSpec& s, int i) {
     if (rc != L3_OK) return rc;
   }
   REQUIRE(nullptr, (s.mixer == L3_MIX_DIFF) == (c->parallel != 0), "layer %d: differential attention and parallel layers come together", i);
-  REQUIRE(nullptr, s.ff_kind == L3_FF_GLU || (s.ff_kind == L3_FF_POLYNORM && c->parallel), "layer %d: this feed-forward kind is built for parallel layers", i);
+  REQUIRE(nullptr, s.ff_kind == L3_FF_GLU || (s.ff_kind == L3_FF_POLYNORM && c->parallel) || (s.ff_kind == L3_FF_RELU2 && c->norm_input && !c->parallel),
+          "layer %d: this feed-forward kind is built for %s layers", i, s.ff_kind == L3_FF_RELU2 ? "pre-norm" : "parallel");
+  REQUIRE(nullptr, s.ff_kind != L3_FF_RELU2 || s.experts == 0, "layer %d: experts have a feed-forward kind of their own", i);
+  REQUIRE(nullptr, s.mixer == L3_MIX_LATENT || (!s.kv_source && !s.sink && !s.gate_wide), "layer %d: shared caches, the sink switch and wide gates belong to latent attention", i);
   REQUIRE(nullptr, s.router_kind == L3_ROUTE_SOFTMAX || (s.router_kind == L3_ROUTE_SIGMOID_IN && c->parallel), "layer %d: this router kind is built for parallel layers", i);
   REQUIRE(nullptr, !(c->parallel && s.experts > 0) || s.router_kind == L3_ROUTE_SIGMOID_IN, "layer %d: parallel layers take the sigmoid router", i);
   REQUIRE(nullptr, s.heads >= 1 && s.dim >= 1 && s.vdim >= 1 && s.ff >= 0, "layer %d: bad sizes", i);
@@ -111,6 +119,7 @@ static int check_spec(const L3StackConfig* c, const L3LayerSpec& s, int i) {
     REQUIRE(nullptr, s.q_rank >= 1 && s.kv_rank >= 1 && s.rot_dim >= 0 && s.rot_dims >= 0 && s.rot_dims <= s.rot_dim && s.rot_dims % 2 == 0,
             "layer %d: bad latent / rotary sizes", i);
     REQUIRE(nullptr, s.rot_dims == 0 || s.rot_base > 0, "layer %d: rotary base must be positive", i);
+    REQUIRE(nullptr, s.rot_layout == 0 || s.rot_layout == 1, "layer %d: bad rot_layout", i);
     REQUIRE(nullptr, latent_attn_supported(s.kv_rank + s.rot_dim, s.kv_rank), "layer %d: latent row of %d + %d entries unsupported", i, s.kv_rank, s.rot_dim);
   } else if (s.mixer == L3_MIX_DIFF) {
     REQUIRE(nullptr, s.kv_heads >= 1 && s.heads % s.kv_heads == 0, "layer %d: heads %% kv_heads != 0", i);
@@ -191,13 +200,30 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
   for (int i = 0; i < c->n_layers; ++i) {
     const int rc = check_spec(c, specs[i], i);
     if (rc != L3_OK) return rc;
+    if (specs[i].kv_source) {
+      const int j = specs[i].kv_source - 1;
+      REQUIRE(nullptr, c->loop_times == 0, "layer %d: a shared cache inside a loop is not built", i);
+      REQUIRE(nullptr, j >= 0 && j < i && specs[j].mixer == L3_MIX_LATENT && !specs[j].kv_source, "layer %d: layer %d has no cache rows to share", i, j);
+      const L3LayerSpec &s = specs[i], &o = specs[j];
+      REQUIRE(nullptr, s.kv_rank == o.kv_rank && s.rot_dim == o.rot_dim && s.rot_dims == o.rot_dims && s.rot_layout == o.rot_layout && s.rot_base == o.rot_base,
+              "layer %d: its kv_rank / rotation differ from those of layer %d, whose cache it reads", i, j);
+    }
   }
   REQUIRE(nullptr, c->loop_times >= 0 && (c->loop_times == 0 || (c->loop_start >= 0 && c->loop_start <= c->loop_stop && c->loop_stop <= c->n_layers)),
           "bad loop bounds");
   REQUIRE(nullptr, !c->norm_input || c->side_dim == 0, "pre-norm stacks have no per-layer token input");
   REQUIRE(nullptr, c->norm_input || (!c->token_shift && !c->norm_scalar), "token shift and single-weight norms are built for pre-norm stacks");
   REQUIRE(nullptr, !c->parallel || (c->norm_input && !c->token_shift && !c->norm_scalar && c->loop_times == 0), "parallel layers are pre-norm layers without token shift, single-weight norms or loops");
-  REQUIRE(nullptr, c->parallel || (!c->norm_center && !c->layer_scale && !c->canon_taps && !c->depth_avg), "centred norms, layer scales, input convolutions and the depth average are built for parallel layers");
+  REQUIRE(nullptr, c->parallel || (!c->norm_center && !c->canon_taps && !c->depth_avg), "centred norms, input convolutions and the depth average are built for parallel layers");
+  const bool pre = c->norm_input && !c->parallel;
+  REQUIRE(nullptr, c->norm_input || !c->layer_scale, "layer scales are built for pre-norm and parallel layers");
+  REQUIRE(nullptr, c->streams >= 0 && (c->streams == 0 || (pre && streams_supported(c->streams, c->width))), "%d residual streams unsupported", c->streams);
+  REQUIRE(nullptr, pre || (!c->tied_head && (c->logit_scale == 0.f || c->logit_scale == 1.f)), "a tied output projection and the logit scale are built for pre-norm stacks");
+  if (c->streams > 0 || (pre && c->layer_scale)) {
+    REQUIRE(nullptr, c->loop_times == 0 && !c->token_shift && c->norm_groups <= 1 && !c->embed_norm, "residual streams and layer scales of pre-norm stacks exclude loops, token shift, grouped norms and the embedding norm");
+    REQUIRE(nullptr, streams_supported(1, c->width), "width %d unsupported with layer scales", c->width);
+    for (int i = 0; i < c->n_layers; ++i) REQUIRE(nullptr, specs[i].experts == 0, "layer %d: experts are not built for residual streams / layer scales", i);
+  }
   REQUIRE(nullptr, c->canon_taps >= 0 && c->canon_taps <= 64, "bad canon_taps");
   REQUIRE(nullptr, c->norm_groups >= 0 && c->norm_groups <= 128 && (c->norm_groups <= 1 || c->width % c->norm_groups == 0), "bad norm_groups");
   REQUIRE(nullptr, (c->norm_input && !c->parallel) || (c->norm_groups <= 1 && !c->embed_norm && !c->loop_in && !(c->logit_softcap > 0.f)),
@@ -232,9 +258,16 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
     return L3_ENOMEM;                                                                         \
   }
   AL(m->embed, (size_t)c->vocab * W * w);
-  AL(m->lm_head, (size_t)c->vocab * W * w);
+  if (c->tied_head) m->lm_head = m->embed;
+  else AL(m->lm_head, (size_t)c->vocab * W * w);
   AL(m->norm_final, (size_t)W * 4);
   if (sd) AL(ll->side_embed, (size_t)c->vocab * c->n_layers * sd * w);
+  ll->streams = c->streams > 0 ? c->streams : (pre && c->layer_scale) ? 1 : 0;
+  if (ll->streams && !c->streams) {
+    const float v = 1.f;
+    AL(ll->one, 4);
+    cudaMemcpy(ll->one, &v, 4, cudaMemcpyHostToDevice);
+  }
   ll->layers.resize(c->n_layers);
   for (int i = 0; i < c->n_layers; ++i) {
     LLLayer& L = ll->layers[i];
@@ -255,11 +288,12 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
       if (rc == L3_OK && L.pair) rc = ll_alloc_unit(*L.pair, w);
       if (rc != L3_OK) { l3_destroy(m); return rc; }
     } else if (s.mixer == L3_MIX_LATENT) {
-      // dq | dkv | g rows, every segment on a multiple of 8 columns of the projection's output
-      const int Dk = s.kv_rank + s.rot_dim;
-      L.off_q = 0; L.off_k = pad8(s.q_rank); L.off_g = pad8(L.off_k + Dk); L.n_in = pad8(L.off_g + H);
+      // dq | dkv | g rows, every segment on a multiple of 8 columns of the projection's output (no dkv with a shared cache)
+      const int Dk = s.kv_source ? 0 : s.kv_rank + s.rot_dim;
+      L.off_q = 0; L.off_k = pad8(s.q_rank); L.off_g = pad8(L.off_k + Dk); L.n_in = pad8(L.off_g + (s.gate_wide ? H * DV : H));
       AL(L.q_norm, (size_t)s.q_rank * 4);
-      AL(L.k_norm, (size_t)s.kv_rank * 4);
+      if (!s.kv_source) AL(L.k_norm, (size_t)s.kv_rank * 4);
+      if (s.sink) AL(L.head_vec, (size_t)H * 4);
       AL(L.w_uq, (size_t)H * (DK + s.rot_dim) * s.q_rank * w);
       AL(L.w_uk, (size_t)H * DK * s.kv_rank * w);
       AL(L.w_uv, (size_t)H * DV * s.kv_rank * w);
@@ -336,6 +370,14 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
     if (c->layer_scale) { AL(L.ls1, (size_t)W * 4); if (s.ff > 0) AL(L.ls2, (size_t)W * 4); }
     if (c->canon_taps > 0) { AL(L.canon1, (size_t)W * c->canon_taps * 4); if (s.ff > 0) AL(L.canon2, (size_t)W * c->canon_taps * 4); }
     if (c->depth_avg) AL(L.dwa, (size_t)(i + 2) * 4);
+    for (int q = 0; q < 2 && ll->streams; ++q) {
+      const int S = c->streams;
+      if (!S) { L.hc_in[q] = L.hc_out[q] = L.hc_mix[q] = ll->one; continue; }
+      if (q == 1 && s.ff == 0) continue;
+      AL(L.hc_in[q], (size_t)S * 4);
+      AL(L.hc_out[q], (size_t)S * 4);
+      AL(L.hc_mix[q], (size_t)S * S * 4);
+    }
     if (s.experts > 0 && s.router_kind == L3_ROUTE_SIGMOID_IN) {
       L.ff_total = s.experts * s.ff + s.shared_ff;
       AL(L.w13, (size_t)2 * L.ff_total * W * w);
@@ -352,7 +394,7 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
       AL(L.router, (size_t)(s.experts + s.identity) * W * 4);
       AL(L.correction, (size_t)(s.experts + s.identity) * 4);
     } else if (s.ff > 0) {
-      AL(L.w13, (size_t)2 * s.ff * W * w);
+      AL(L.w13, (size_t)(s.ff_kind == L3_FF_RELU2 ? 1 : 2) * s.ff * W * w);
       AL(L.w2, (size_t)W * s.ff * w);
       if (!c->parallel) AL(L.norm2, (size_t)W * 4);
     }
@@ -507,7 +549,7 @@ static bool ll_place(L3Model* m, const std::string& name, LLPlace* p) {
     return d != nullptr;
   };
   if (name == "embed") { const bool ok = mat(m->embed, V, W); p->scale = pre ? 0.1f : 1.0f; return ok; }
-  if (name == "head") return mat(m->lm_head, V, W);
+  if (name == "head") return !ll->cfg.tied_head && mat(m->lm_head, V, W);
   if (name == "final.norm") return norm(m->norm_final);
   if (name == "loop.step") return ll->loop_step && fmat(ll->loop_step, ll->cfg.loop_times, W, 0.3f);
   if (name == "loop.in") { const bool ok = ll->loop_in && mat(ll->loop_in, W, (int64_t)2 * W); p->scale *= 1.4f; return ok; }
@@ -521,6 +563,13 @@ static bool ll_place(L3Model* m, const std::string& name, LLPlace* p) {
   const int H = s.heads, G = s.kv_heads, DK = s.dim, DV = s.vdim;
   if (r == "norm1") return norm(L.norm1);
   if (r == "norm2") return s.ff > 0 && L.norm2 && norm(L.norm2);
+  for (int q = 0; q < 2 && ll->cfg.streams > 0; ++q) {
+    const int S = ll->cfg.streams;
+    const std::string h = q ? "hc2." : "hc1.";
+    if (r == h + "in") return L.hc_in[q] && vec(L.hc_in[q], S, 1.f / (float)S, 0.3f / (float)S);
+    if (r == h + "out") return L.hc_out[q] && vec(L.hc_out[q], S, 1.f, 0.2f);
+    if (r == h + "mix") { const bool ok = L.hc_mix[q] && fmat(L.hc_mix[q], S, S, 0.3f / (float)S); p->bias = 1.f / (float)S; return ok; }
+  }
   if (r == "ls1") return L.ls1 && vec(L.ls1, W, 1.f, 0.2f);
   if (r == "ls2") return L.ls2 && vec(L.ls2, W, 1.f, 0.2f);
   if (r == "canon1") return L.canon1 && fmat(L.canon1, W, ll->cfg.canon_taps, 0.3f / (float)ll->cfg.canon_taps);
@@ -566,6 +615,9 @@ static bool ll_place(L3Model* m, const std::string& name, LLPlace* p) {
       }
     }
     if (r.compare(0, 4, "mlp.") == 0) return false;
+  } else if (s.ff_kind == L3_FF_RELU2) {
+    if (r == "mlp.up") return s.ff > 0 && mat(L.w13, s.ff, W);
+    if (r == "mlp.down") return s.ff > 0 && mat(L.w2, W, s.ff);
   } else {
     if (r == "mlp.gate") return s.ff > 0 && mat(L.w13, s.ff, W, 0, 2);
     if (r == "mlp.up") return s.ff > 0 && mat(L.w13, s.ff, W, 1, 2);
@@ -584,8 +636,10 @@ static bool ll_place(L3Model* m, const std::string& name, LLPlace* p) {
   auto seg = [&](int off, int64_t rows) { const bool ok = mat(L.w_in, rows, W, off, 1); return ok; };
   if (s.mixer == L3_MIX_LATENT) {
     if (r == "mix.dq") return seg(L.off_q, s.q_rank);
+    if (s.kv_source && r.compare(0, 7, "mix.dkv") == 0) return false;
+    if (r == "mix.sink") return s.sink && vec(L.head_vec, H, 0.5f, 0.5f);
     if (r == "mix.dkv") { const bool ok = seg(L.off_k, (int64_t)s.kv_rank + s.rot_dim); p->scale *= 2.f; return ok; }
-    if (r == "mix.g") return seg(L.off_g, H);
+    if (r == "mix.g") return seg(L.off_g, s.gate_wide ? (int64_t)H * DV : H);
     if (r == "mix.dq.norm") return vec(L.q_norm, s.q_rank, 1.f, 0.1f);
     if (r == "mix.dkv.norm") return vec(L.k_norm, s.kv_rank, 1.f, 0.1f);
     if (r == "mix.uq") { const bool ok = mat(L.w_uq, (int64_t)H * (DK + s.rot_dim), s.q_rank); p->scale *= 2.f; return ok; }
@@ -658,7 +712,8 @@ static bool ll_place(L3Model* m, const std::string& name, LLPlace* p) {
 
 static std::vector<std::string> ll_expected(const L3Model* m) {
   const LayerList* ll = m->ll;
-  std::vector<std::string> v = {"embed", "head", "final.norm"};
+  std::vector<std::string> v = {"embed", "final.norm"};
+  if (!ll->cfg.tied_head) v.push_back("head");
   if (ll->cfg.side_dim) v.push_back("side.embed");
   if (ll->loop_step) v.push_back("loop.step");
   if (ll->loop_in) v.push_back("loop.in");
@@ -674,7 +729,11 @@ static std::vector<std::string> ll_expected(const L3Model* m) {
       const LLLayer& Lu = ll->layers[i];
       for (auto nme : ll_unit_names(s)) v.push_back(p + (Lu.pair ? "mix.left." : "mix.") + nme);
       if (Lu.pair) for (auto nme : ll_unit_names(Lu.pair->spec)) v.push_back(p + "mix.right." + nme);
-    } else if (s.mixer == L3_MIX_LATENT) names.insert(names.end(), {"mix.dq", "mix.dq.norm", "mix.uq", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv", "mix.g"});
+    } else if (s.mixer == L3_MIX_LATENT) {
+      names.insert(names.end(), {"mix.dq", "mix.dq.norm", "mix.uq", "mix.uk", "mix.uv", "mix.g"});
+      if (!s.kv_source) names.insert(names.end(), {"mix.dkv", "mix.dkv.norm"});
+      if (s.sink) names.push_back("mix.sink");
+    }
     else if (s.mixer == L3_MIX_MINGRU) names.insert(names.end(), {"mix.z", "mix.z.b", "mix.x", "mix.x.b", "mix.g"});
     else if (s.mixer == L3_MIX_DIFF) names.insert(names.end(), {"mix.q", "mix.q.b", "mix.k", "mix.k.b", "mix.v", "mix.v.b", "mix.q.norm", "mix.k.norm",
                                                                 "mix.lq1", "mix.lk1", "mix.lq2", "mix.lk2"});
@@ -685,6 +744,10 @@ static std::vector<std::string> ll_expected(const L3Model* m) {
     const LLLayer& Lx = ll->layers[i];
     if (Lx.ls1) names.push_back("ls1");
     if (Lx.ls2) names.push_back("ls2");
+    if (ll->cfg.streams > 0) {
+      names.insert(names.end(), {"hc1.in", "hc1.out", "hc1.mix"});
+      if (s.ff > 0) names.insert(names.end(), {"hc2.in", "hc2.out", "hc2.mix"});
+    }
     if (Lx.canon1) names.push_back("canon1");
     if (Lx.canon2) names.push_back("canon2");
     if (Lx.dwa) names.push_back("dwa");
@@ -705,7 +768,8 @@ static std::vector<std::string> ll_expected(const L3Model* m) {
       }
     } else if (s.ff > 0) {
       if (Lx.norm2) names.push_back("norm2");
-      names.insert(names.end(), {"mlp.gate", "mlp.up", "mlp.down"});
+      if (s.ff_kind != L3_FF_RELU2) names.push_back("mlp.gate");
+      names.insert(names.end(), {"mlp.up", "mlp.down"});
     }
     if (ll->cfg.side_dim) names.insert(names.end(), {"side.gate", "side.proj", "side.norm"});
     for (auto nme : names) v.push_back(p + nme);
@@ -821,7 +885,8 @@ int ll_finalize(L3Model* m) {
       if (rc == L3_OK && L.pair) { St.pair = new LLState(); rc = ll_alloc_unit_state(m, L.pair->spec, *St.pair); }
       if (rc != L3_OK) return rc;
     } else if (s.mixer == L3_MIX_LATENT) {
-      CK(m, cudaMalloc(&St.lat, (size_t)m->maxB * m->M * (s.kv_rank + s.rot_dim) * kvb));
+      if (s.kv_source) { St.lat = ll->state[s.kv_source - 1].lat; St.lat_shared = true; }  // without a loop a run is a layer
+      else CK(m, cudaMalloc(&St.lat, (size_t)m->maxB * m->M * (s.kv_rank + s.rot_dim) * kvb));
     } else if (s.mixer == L3_MIX_DIFF) {
       CK(m, cudaMalloc(&St.ck, (size_t)m->maxB * 2 * G * m->M * DK * kvb));
       CK(m, cudaMalloc(&St.cv, (size_t)m->maxB * G * m->M * DV * kvb));
@@ -906,6 +971,12 @@ int ll_finalize(L3Model* m) {
   CK(m, cudaMalloc((void**)&ll->o, ct * ll->max_o * 4));
   CK(m, cudaMalloc((void**)&ll->sg, ct * std::max(1, sd) * 4));
   if (max_qlat) CK(m, cudaMalloc((void**)&ll->qlat, ct * max_qlat * 4));
+  if (ll->streams) {
+    CK(m, cudaMalloc((void**)&ll->X, ct * ll->streams * W * 4));
+    CK(m, cudaMalloc((void**)&ll->y1, ct * W * 4));
+  }
+  // the logit scale rides on the final norm's weight
+  if (ll->cfg.logit_scale != 0.f && ll->cfg.logit_scale != 1.f) LAUNCH(m, launch_scale_add_rows(m->norm_final, ll->cfg.logit_scale, nullptr, 1, W, m->stream));
   if (max_xs) CK(m, cudaMalloc((void**)&ll->xs, ct * max_xs * 4));
   if (win_part) {
     CK(m, cudaMalloc((void**)&ll->win_part_o, win_part * 4));
@@ -999,7 +1070,8 @@ void ll_destroy(L3Model* m) {
   LayerList* ll = m->ll;
   if (!ll) return;
   auto fr = [](void* p) { if (p) cudaFree(p); };
-  fr(ll->side_embed);
+  fr(ll->side_embed); fr(ll->one); fr(ll->X);
+  if (m->lm_head == m->embed) m->lm_head = nullptr;  // a tied output projection has no storage of its own
   for (auto& L : ll->layers) {
     fr(L.w_in); fr(L.w_o); fr(L.w_a2); fr(L.w_g2); fr(L.w13); fr(L.w2); fr(L.side_gate); fr(L.side_proj);
     fr(L.norm1); fr(L.norm2); fr(L.side_norm); fr(L.mix_norm); fr(L.q_norm); fr(L.k_norm); fr(L.conv_w);
@@ -1007,6 +1079,7 @@ void ll_destroy(L3Model* m) {
     fr(L.w_uq); fr(L.w_uk); fr(L.w_uv); fr(L.inv_freq); fr(L.in_bias); fr(L.shift); fr(L.router); fr(L.correction);
     fr(L.canon1); fr(L.canon2); fr(L.canon1t); fr(L.canon2t); fr(L.ls1); fr(L.ls2); fr(L.dwa); fr(L.lam_vec); fr(L.lambda); fr(L.poly);
     fr(L.head_vec); fr(L.conv_b); fr(L.skip_d); fr(L.a2_bias);
+    for (int q = 0; q < 2 && ll->cfg.streams > 0; ++q) { fr(L.hc_in[q]); fr(L.hc_out[q]); fr(L.hc_mix[q]); }
     if (LLLayer* R = L.pair) {  // its w_in / w_o are views of the first mixer's
       fr(R->w_a2); fr(R->w_g2); fr(R->mix_norm); fr(R->conv_w); fr(R->A_log); fr(R->dt_bias); fr(R->inv_freq);
       fr(R->head_vec); fr(R->conv_b); fr(R->skip_d); fr(R->a2_bias);
@@ -1015,7 +1088,7 @@ void ll_destroy(L3Model* m) {
     }
   }
   for (auto& St : ll->state) {
-    fr(St.ck); fr(St.cv); fr(St.S); fr(St.conv_tail); fr(St.lat); fr(St.hprev);
+    fr(St.ck); fr(St.cv); fr(St.S); fr(St.conv_tail); fr(St.lat_shared ? nullptr : St.lat); fr(St.hprev);
     if (LLState* P = St.pair) { fr(P->ck); fr(P->cv); fr(P->S); fr(P->conv_tail); delete P; St.pair = nullptr; }
   }
   fr(ll->loop_in); fr(ll->embed_norm); fr(ll->x0); fr(ll->cat); fr(ll->cat16); fr(ll->win_part_o); fr(ll->win_part_ml); fr(ll->xs);
@@ -1052,7 +1125,7 @@ int ll_reset_slots(L3Model* m, int slot0, int n, bool kv_too) {
       continue;
     }
     if (s.mixer == L3_MIX_LATENT) {
-      if (!kv_too) continue;  // rows past a slot's position are never read: a new sequence overwrites them
+      if (!kv_too || St.lat_shared) continue;  // rows past a slot's position are never read: a new sequence overwrites them
       const size_t per = (size_t)m->M * (s.kv_rank + s.rot_dim) * kvb;
       CK(m, cudaMemsetAsync((char*)St.lat + slot0 * per, 0, n * per, m->stream));
     } else if (s.mixer == L3_MIX_SOFTMAX) {
@@ -1150,10 +1223,16 @@ static int ll_settle(L3Model* m, LLPending& pd, int rows) {
   return L3_OK;
 }
 
+// does a projection of contiguous rows with a bf16 mirror run on the tensor cores (and so read the mirror alone)?
+static bool ll_takes_mirror(const L3Model* m, int rows, int N, int K) {
+  return m->tc_ok && !linear_rows_supported(rows, K) && K % 8 == 0 && K >= 64 && N >= 64;
+}
+
 // y = x W^T (+ epilogue).  x32: fp32 rows with stride lda (0 = K); x16: bf16 mirror with stride K, or null.
 // pd: non-null when x32 is the residual stream (ll->xcur) - a deferred step is applied on the way.
+// norm_w: the row-streaming GEMV norms the rows while staging them (only where linear_rows_supported says it runs).
 static int ll_linear(L3Model* m, const void* W, const float* x32, const void* x16, int lda, int rows, int N, int K, int epi,
-                     const EpiArgs& e, LLPending* pd = nullptr) {
+                     const EpiArgs& e, LLPending* pd = nullptr, const float* norm_w = nullptr) {
   LayerList* ll = m->ll;
   LinearArgs a{};
   a.W = W; a.x = x32; a.lda = lda; a.rows = rows; a.N = N; a.K = K; a.src_mul = 1; a.src_add = 0; a.epi = epi; a.e = e;
@@ -1171,6 +1250,7 @@ static int ll_linear(L3Model* m, const void* W, const float* x32, const void* x1
       std::swap(ll->xcur, ll->xalt);
       pd->y = nullptr;
     } else if (pd) a.x = ll->xcur;
+    a.norm_w = norm_w; a.eps = ll->cfg.norm_eps;
     LAUNCH(m, launch_linear_rows(a, m->bf16, m->bf16, m->stream));
     return L3_OK;
   }
@@ -1179,7 +1259,7 @@ static int ll_linear(L3Model* m, const void* W, const float* x32, const void* x1
     if (rc != L3_OK) return rc;
     a.x = ll->xcur;
   }
-  if (m->tc_ok && x16 && ld == K && K % 8 == 0 && K >= 64 && N >= 64) {
+  if (x16 && ld == K && ll_takes_mirror(m, rows, N, K)) {
     TcGemmArgs t{};
     t.kind = TC_BF16; t.A[0] = x16; t.W[0] = W;
     t.rows = rows; t.N = N; t.K = K; t.epi = epi; t.e = e; t.bn = 0;
@@ -1203,7 +1283,8 @@ static EpiArgs store_to(float* out, void* out16, int ld) {
 // ------------------------------------------------------------------------------ pre-norm layers
 // x <- x + mixer(shift(norm1(x)));  x <- x + ff(norm2(x)).  The residual stream stays in m->x (fp32); the normed rows
 // live in m->xn (+ the bf16 mirror m->xn16 for the tensor-core projections); the sublayers' output projections add
-// into x in their epilogue.
+// into x in their epilogue.  With residual streams (ll->streams) they store their result instead and the next stream launch
+// applies it (stream_ops.cu); m->x then holds the embedding output at first and the sum of the streams at the end.
 static EpiArgs resid_into(float* x, int ld) {
   EpiArgs e{};
   e.out = x; e.resid = x; e.ld_out = ld;
@@ -1297,7 +1378,39 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
   bf16* hn16 = (bf16*)m->xn16;  // null in fp32 mode
   int rc;
   ll->xcur = m->x;
-  if (ll->cfg.embed_scale != 0.f && ll->cfg.embed_scale != 1.f) LAUNCH(m, launch_scale_add_rows(m->x, ll->cfg.embed_scale, nullptr, ntok, W, m->stream));
+  const float embed_mul = ll->cfg.embed_scale != 0.f ? ll->cfg.embed_scale : 1.f;
+  if (embed_mul != 1.f && !ll->streams) LAUNCH(m, launch_scale_add_rows(m->x, embed_mul, nullptr, ntok, W, m->stream));
+  StreamArgs sa{};  // the streams' side of the step: sa.y is the sublayer result they have not taken yet
+  sa.x0 = m->x; sa.x_mul = embed_mul; sa.X = ll->X; sa.eps = eps; sa.S = ll->streams; sa.D = W;
+  const bool gemv = linear_rows_supported(ntok, W);  // few rows: the GEMV norms what the stream launch leaves un-normed
+  // the normed input of sublayer q into hn / hn16 (or, for few rows of a streamed stack, its un-normed form: *in_norm)
+  auto sublayer_in = [&](LLLayer& Ly, int q, const float* norm, const float* shift, float* hprev, int n_out, const float** in_norm) -> int {
+    *in_norm = nullptr;
+    if (!ll->streams) {
+      LAUNCH(m, launch_prenorm_shift(m->x, norm, eps, shift, hprev, B, L, W, hn, hn16, m->stream, std::max(1, ll->cfg.norm_groups)));
+      return L3_OK;
+    }
+    StreamArgs a = sa;
+    a.store = 1; a.in_w = Ly.hc_in[q];
+    if (gemv) { a.h = hn; *in_norm = norm; }
+    else { a.norm_w = norm; a.h16 = hn16; a.h = hn16 && ll_takes_mirror(m, ntok, n_out, W) ? nullptr : hn; }
+    LAUNCH(m, launch_streams(a, ntok, m->stream));
+    if (sa.y) sa.x0 = nullptr;  // from here on X holds the streams
+    sa.y = nullptr;
+    return L3_OK;
+  };
+  // after sublayer q's output projection (epilogue out_epi / out_e)
+  const int out_epi = ll->streams ? EPI_STORE : EPI_RESID;
+  const EpiArgs out_e = ll->streams ? store_to(ll->y1, nullptr, W) : resid_into(m->x, W);
+  auto sublayer_out = [&](LLLayer& Ly, int q) { sa.y = ll->y1; sa.ls = q ? Ly.ls2 : Ly.ls1; sa.mix = Ly.hc_mix[q]; sa.out_w = Ly.hc_out[q]; };
+  // the sum of the streams into m->x; `store`: the streams themselves go on
+  auto streams_sum = [&](bool store) -> int {
+    StreamArgs a = sa;
+    a.store = store; a.sum = m->x;
+    LAUNCH(m, launch_streams(a, ntok, m->stream));
+    sa.x0 = nullptr; sa.y = nullptr;
+    return L3_OK;
+  };
   const int ng = std::max(1, ll->cfg.norm_groups);
   if (ll->embed_norm) LAUNCH(m, launch_rmsnorm_rows(m->x, ll->embed_norm, eps, ntok, W, 1, 0, nullptr, m->x, nullptr, m->stream, ng));  // in place, row by row
   if (ll->x0) CK(m, cudaMemcpyAsync(ll->x0, m->x, (size_t)ntok * W * 4, cudaMemcpyDeviceToDevice, m->stream));  // the embedding output
@@ -1311,9 +1424,10 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
       if ((rc = ll_linear(m, ll->loop_in, ll->cat, ll->cat16, 0, ntok, W, 2 * W, EPI_STORE, store_to(m->x, nullptr, W))) != L3_OK) return rc;
     } else if (ll->runs[ri].pass >= 0)
       LAUNCH(m, launch_scale_add_rows(m->x, 1.0f, ll->loop_step + (size_t)ll->runs[ri].pass * W, ntok, W, m->stream));
-    LAUNCH(m, launch_prenorm_shift(m->x, Ly.norm1, eps, Ly.shift, St.hprev, B, L, W, hn, hn16, m->stream, ng));
+    const float* in_norm;
+    if ((rc = sublayer_in(Ly, 0, Ly.norm1, Ly.shift, St.hprev, Ly.n_in, &in_norm)) != L3_OK) return rc;
     // every projection of the mixer's input in one GEMM
-    if ((rc = ll_linear(m, Ly.w_in, hn, hn16, 0, ntok, Ly.n_in, W, EPI_STORE, store_to(ll->pin, nullptr, Ly.n_in))) != L3_OK) return rc;
+    if ((rc = ll_linear(m, Ly.w_in, hn, hn16, 0, ntok, Ly.n_in, W, EPI_STORE, store_to(ll->pin, nullptr, Ly.n_in), nullptr, in_norm)) != L3_OK) return rc;
     int n_ctx = H * DV;
     if (unit_mixer(s.mixer)) {
       n_ctx = Ly.ctx_ld;
@@ -1322,9 +1436,10 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
     } else if (s.mixer == L3_MIX_LATENT) {
       const int Dk = s.kv_rank + s.rot_dim, nq = H * (DK + s.rot_dim);
       LatentPrepArgs pa{};
-      pa.proj = ll->pin; pa.ld = Ly.n_in; pa.k_off = Ly.off_k; pa.wq = Ly.q_norm; pa.wk = Ly.k_norm; pa.eps = eps;
+      pa.proj = ll->pin; pa.ld = Ly.n_in; pa.k_off = s.kv_source ? -1 : Ly.off_k; pa.wq = Ly.q_norm; pa.wk = Ly.k_norm; pa.eps = eps;
       pa.cq = ll->aux; pa.cq16 = (bf16*)ll->aux16; pa.cache = St.lat; pa.inv_freq = Ly.inv_freq; pa.pos_ptr = d_pos;
       pa.L = L; pa.M = m->M; pa.q_rank = s.q_rank; pa.kv_rank = s.kv_rank; pa.rot_dim = s.rot_dim; pa.rot_dims = s.rot_dims;
+      pa.rot_layout = s.rot_layout;
       LAUNCH(m, launch_latent_prep(pa, ntok, m->bf16, m->stream));
       if ((rc = ll_linear(m, Ly.w_uq, ll->aux, ll->aux16, 0, ntok, nq, s.q_rank, EPI_STORE, store_to(m->q, nullptr, nq))) != L3_OK) return rc;
       // queries onto the latent: qlat[r, h] = [Wuk_h^T q_c | rot(q_r)]
@@ -1333,11 +1448,11 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
       ga.W = Ly.w_uk; ga.w_hs = (int64_t)DK * s.kv_rank; ga.w_ks = s.kv_rank; ga.w_js = 1;
       ga.C = ll->qlat; ga.C16 = nullptr; ga.ldc = H * Dk; ga.c_hs = Dk;
       ga.rows = ntok; ga.H = H; ga.J = s.kv_rank; ga.K = DK;
+      ga.inv_freq = Ly.inv_freq; ga.pos_ptr = d_pos; ga.L = L; ga.rot_dim = s.rot_dim; ga.rot_dims = s.rot_dims; ga.rot_layout = s.rot_layout;
       LAUNCH(m, launch_head_gemm(ga, m->bf16, m->stream));
-      if (s.rot_dim > 0)
-        LAUNCH(m, launch_latent_q_rope(m->q, ll->qlat, Ly.inv_freq, d_pos, ntok, L, H, DK, s.rot_dim, s.rot_dims, s.kv_rank, m->stream));
       LatentAttnArgs at{};
-      at.q = ll->qlat; at.cache = St.lat; at.out = ll->o; at.gate = ll->pin + Ly.off_g; at.ld_gate = Ly.n_in;
+      at.q = ll->qlat; at.cache = St.lat; at.out = ll->o; at.gate = s.gate_wide ? nullptr : ll->pin + Ly.off_g; at.ld_gate = Ly.n_in;
+      at.sink = s.sink ? Ly.head_vec : nullptr;
       at.pos_ptr = d_pos; at.scale = s.scale; at.B = B; at.L = L; at.H = H; at.Dk = Dk; at.Dv = s.kv_rank; at.M = m->M;
       at.part_o = m->part_o; at.part_ml = m->part_ml;
       at.nsplit = 1;
@@ -1351,7 +1466,8 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
       HeadGemmArgs gv{};
       gv.A = ll->o; gv.lda = H * s.kv_rank; gv.a_hs = s.kv_rank;
       gv.W = Ly.w_uv; gv.w_hs = (int64_t)DV * s.kv_rank; gv.w_ks = 1; gv.w_js = s.kv_rank;
-      gv.C = m->ctx; gv.C16 = (bf16*)m->ctx16; gv.ldc = H * DV; gv.c_hs = DV;
+      gv.C = m->ctx16 && ll_takes_mirror(m, ntok, W, H * DV) ? nullptr : m->ctx; gv.C16 = (bf16*)m->ctx16; gv.ldc = H * DV; gv.c_hs = DV;
+      if (s.gate_wide) { gv.gate = ll->pin + Ly.off_g; gv.ld_gate = Ly.n_in; }
       gv.rows = ntok; gv.H = H; gv.J = DV; gv.K = s.kv_rank;
       LAUNCH(m, launch_head_gemm(gv, m->bf16, m->stream));
     } else if (s.mixer == L3_MIX_MINGRU) {
@@ -1361,7 +1477,8 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
       set_err(m, "mixer %d is not built for pre-norm layers", s.mixer);
       return L3_EINVAL;
     }
-    if ((rc = ll_linear(m, Ly.w_o, m->ctx, m->ctx16, 0, ntok, W, n_ctx, EPI_RESID, resid_into(m->x, W))) != L3_OK) return rc;
+    if ((rc = ll_linear(m, Ly.w_o, m->ctx, m->ctx16, 0, ntok, W, n_ctx, out_epi, out_e)) != L3_OK) return rc;
+    sublayer_out(Ly, 0);
     if (s.experts > 0) {
       const int E = s.experts, ff = s.ff;
       LAUNCH(m, launch_prenorm_shift(m->x, Ly.norm2, eps, nullptr, nullptr, B, L, W, hn, hn16, m->stream, ng));
@@ -1381,12 +1498,16 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
         if (s.identity > 0) LAUNCH(m, launch_moe_identity(m->x, hn, ll->moe_idw, ntok, W, m->stream));
       }
     } else if (s.ff > 0) {
-      LAUNCH(m, launch_prenorm_shift(m->x, Ly.norm2, eps, nullptr, nullptr, B, L, W, hn, hn16, m->stream, ng));
-      EpiArgs e = store_to(m->h, m->h16, s.ff);
-      e.act = ll->cfg.glu_act;
-      if ((rc = ll_linear(m, Ly.w13, hn, hn16, 0, ntok, 2 * s.ff, W, EPI_SWIGLU, e)) != L3_OK) return rc;
-      if ((rc = ll_linear(m, Ly.w2, m->h, m->h16, 0, ntok, W, s.ff, EPI_RESID, resid_into(m->x, W))) != L3_OK) return rc;
+      const bool glu = s.ff_kind != L3_FF_RELU2;
+      const int n_up = glu ? 2 * s.ff : s.ff;
+      if ((rc = sublayer_in(Ly, 1, Ly.norm2, nullptr, nullptr, n_up, &in_norm)) != L3_OK) return rc;
+      EpiArgs e = store_to(m->h16 && ll_takes_mirror(m, ntok, W, s.ff) ? nullptr : m->h, m->h16, s.ff);
+      if (glu) e.act = ll->cfg.glu_act; else e.unary = UNARY_RELU2;
+      if ((rc = ll_linear(m, Ly.w13, hn, hn16, 0, ntok, n_up, W, glu ? EPI_SWIGLU : EPI_STORE, e, nullptr, in_norm)) != L3_OK) return rc;
+      if ((rc = ll_linear(m, Ly.w2, m->h, m->h16, 0, ntok, W, s.ff, out_epi, out_e)) != L3_OK) return rc;
+      sublayer_out(Ly, 1);
     }
+    if (ll->streams && (d_resid || ri + 1 == (int)ll->runs.size()) && (rc = streams_sum(ri + 1 < (int)ll->runs.size())) != L3_OK) return rc;
     if (d_resid) CK(m, cudaMemcpyAsync(d_resid + (size_t)ri * ntok * W, m->x, (size_t)ntok * W * 4, cudaMemcpyDeviceToDevice, m->stream));
   }
   return L3_OK;
@@ -1507,9 +1628,9 @@ int ll_enqueue_layers(L3Model* m, const int32_t* d_ids, int ids_ld, int ids_off,
   ll->xalt = ll->x2;
   LLPending pd;
   if (ll->cfg.parallel) return ll_enqueue_parallel(m, B, L, d_resid);
+  if (ll->cfg.norm_input) return ll_enqueue_prenorm(m, B, L, d_resid);
   // rows <= 8 never reach a tensor-core projection of the residual stream: no mirror needed
   if (x16 && !linear_rows_supported(ntok, W)) LAUNCH(m, launch_to_bf16(m->x, (int64_t)ntok * W, x16, m->stream));
-  if (ll->cfg.norm_input) return ll_enqueue_prenorm(m, B, L, d_resid);
   for (int ri = 0; ri < (int)ll->runs.size(); ++ri) {
     const int li = ll->runs[ri].layer;
     LLLayer& Ly = ll->layers[li];

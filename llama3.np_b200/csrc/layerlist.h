@@ -41,6 +41,8 @@ struct LLLayer {
   float* correction = nullptr;  // [experts + identity]
   // parallel layers: convolutions ahead of the sublayers [width, taps], layer scales [width], depth-average weights [layer + 2]
   float *canon1 = nullptr, *canon2 = nullptr, *ls1 = nullptr, *ls2 = nullptr, *dwa = nullptr;
+  // residual streams (L3StackConfig::streams): in / out [S], mix [S, S] of the two sublayers (views of LayerList::one without streams)
+  float *hc_in[2] = {nullptr, nullptr}, *hc_out[2] = {nullptr, nullptr}, *hc_mix[2] = {nullptr, nullptr};
   float *canon1t = nullptr, *canon2t = nullptr;  // [taps, width] copies the kernels read (made at finalize)
   // differential attention: w_in = q | k | v rows with in_bias [n_in]; q_norm / k_norm [dim]; lam_vec = lq1 | lk1 | lq2 | lk2
   float *lam_vec = nullptr, *lambda = nullptr;
@@ -48,7 +50,7 @@ struct LLLayer {
   // sigmoid-routed gated experts: w13 = [2 (experts ff + shared_ff), width] rows interleaved (gate_j, up_j), expert by
   // expert, the shared expert last; w2 = [width, experts ff + shared_ff]
   int ff_total = 0;
-  // window attention: head_vec [heads] the sinks' logits or the sigmoid's biases; state-space mixer: conv_b [channels],
+  // window attention: head_vec [heads] the sinks' logits or the sigmoid's biases (latent attention: the sinks' logits); state-space mixer: conv_b [channels],
   // skip_d [heads] (the D of y += D x), dt_bias [heads]; gated linear attention: a2_bias [heads * dim]
   float *head_vec = nullptr, *conv_b = nullptr, *skip_d = nullptr, *a2_bias = nullptr;
   // Two mixers side by side: `pair` is the second one (its mixer fields only).  Both read ONE fused input projection -
@@ -66,6 +68,7 @@ struct LLState {
   float* S = nullptr;                 // recurrent: [maxB, heads, dim, vdim]
   float* conv_tail = nullptr;         // gated delta: [maxB, channels, taps - 1]
   void* lat = nullptr;                // latent attention: [maxB, M, kv_rank + rot_dim] of KVT
+  bool lat_shared = false;            // lat is another layer run's (L3LayerSpec::kv_source)
   float* hprev = nullptr;             // token shift: [maxB, width] the last token's normed mixer input
   // differential attention: ck [maxB, 2 kv_heads, M, dim] (head g, map m at 2 g + m), cv [maxB, kv_heads, M, vdim];
   // parallel layers with a convolution: conv_tail [maxB, width, taps - 1] the last rows of the layer's normed input
@@ -84,6 +87,9 @@ struct LayerList {
   std::vector<LLLayer> layers;
   std::vector<LLRun> runs;       // execution order
   std::vector<LLState> state;    // per run
+  int streams = 0;               // residual rows per token (0: one, the output projections add into it)
+  float* one = nullptr;          // the number 1: stream weights of a layer-scaled stack without streams
+  float* X = nullptr;            // [cap_tok, streams, width] the residual rows
   float* loop_step = nullptr;    // [loop_times, width] fp32
   void* loop_in = nullptr;       // [width, 2 width] of WT: the looped block's entry projection (loop_in)
   float* embed_norm = nullptr;   // [width]
@@ -111,7 +117,7 @@ struct LayerList {
   float* Xs = nullptr;                     // [n_layers + 1][cap_tok, width] embedding output and every layer's own result
   float *hn = nullptr, *hf = nullptr;      // normed rows ahead of the convolutions; the feed-forward's input
   void* hf16 = nullptr;
-  float *y1 = nullptr, *y2 = nullptr;      // the two sublayers' results [cap_tok, width]
+  float *y1 = nullptr, *y2 = nullptr;      // the two sublayers' results [cap_tok, width] (with streams: y1 alone)
   float* moe_gu = nullptr;                 // [cap_tok, 2 ff_total] gate | up of every expert
   float *diff_part_o = nullptr, *diff_part_ml = nullptr;  // split scratch of the differential decode attention
   int max_in = 0, max_o = 0, max_ff = 0;

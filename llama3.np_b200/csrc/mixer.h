@@ -94,10 +94,36 @@ cudaError_t launch_prenorm_shift(const float* x, const float* w, float eps, cons
 // x[r, i] = x[r, i] * mul + (vec ? vec[i] : 0)
 cudaError_t launch_scale_add_rows(float* x, float mul, const float* vec, int rows, int D, cudaStream_t s);
 
+// ---- residual streams (stream_ops.cu)
+constexpr int STREAMS_MAX = 32;
+// One pass over the S residual rows of every token: apply the pending sublayer result y (null: none),
+//   X_t <- sum_s mix[s * S + t] X_s + out_w[t] * (ls * y)            (ls null: ones; written back when `store`)
+// and form what follows: the next sublayer's input  h = n(sum_s in_w[s] X_s)  with n the RMS norm of weight norm_w (norm_w
+// null: un-normed), its bf16 mirror, and / or the sum of the streams.
+struct StreamArgs {
+  const float* x0;       // non-null: every stream is x0[r] * x_mul (X is not read): the first passes of a step
+  float x_mul;
+  float* X;              // [rows, S, D]
+  const float* y;        // [rows, D]
+  const float* ls;       // [D]
+  const float *mix, *out_w;
+  int store;
+  float* sum;            // [rows, D] or null (may be the buffer x0 points to)
+  const float* in_w;     // [S] or null: no next sublayer
+  const float* norm_w;   // [D]
+  float eps;
+  float* h;              // [rows, D] or null
+  bf16* h16;             // or null
+  int S, D;
+};
+bool streams_supported(int S, int D);
+cudaError_t launch_streams(const StreamArgs& a, int rows, cudaStream_t s);
+
 // ---- latent attention (attn_latent.cu)
+// rotary pairs: layout 0 = entries (2i, 2i + 1), 1 = entries (i, i + dims / 2)
 struct LatentPrepArgs {
   const float* proj;     // [rows, ld]: query latent at column 0 (q_rank), key latent at k_off (kv_rank), rotated key part behind it (rot_dim)
-  int ld, k_off;
+  int ld, k_off;         // k_off < 0: the queries only (the layer reads another layer's cache)
   const float *wq, *wk;  // norm weights [q_rank], [kv_rank]
   float eps;
   float* cq;             // [rows, q_rank] normed query latent (+ bf16 mirror, may be null)
@@ -105,19 +131,21 @@ struct LatentPrepArgs {
   void* cache;           // [maxB, M, kv_rank + rot_dim] of KVT
   const float* inv_freq; // [rot_dims / 2]
   const int* pos_ptr;
-  int L, M, q_rank, kv_rank, rot_dim, rot_dims;
+  int L, M, q_rank, kv_rank, rot_dim, rot_dims, rot_layout;
 };
 cudaError_t launch_latent_prep(const LatentPrepArgs& a, int rows, bool kv_bf16, cudaStream_t s);
-// rotated part of the queries: qlat[r, h, kv_rank + j] = rot(q[r, h, dim + j]) at the row's position
-cudaError_t launch_latent_q_rope(const float* q, float* qlat, const float* inv_freq, const int* pos_ptr, int rows, int L,
-                                 int H, int dim, int rot_dim, int rot_dims, int kv_rank, cudaStream_t s);
 // Batched per-head product  C[r, h, j] = sum_k A[r * lda + h * a_hs + k] * W[h * w_hs + k * w_ks + j * w_js]
-// for r < rows, h < H, j < J, k < K; C at c[r * ldc + h * c_hs + j] (+ bf16 mirror).  One of w_ks, w_js is 1.
+// for r < rows, h < H, j < J, k < K; C at c[r * ldc + h * c_hs + j] (+ bf16 mirror; either may be null).  One of w_ks, w_js is 1.
 struct HeadGemmArgs {
   const float* A; int lda, a_hs;
   const void* W; int64_t w_hs; int w_ks, w_js;
   float* C; bf16* C16; int ldc, c_hs;
   int rows, H, J, K;
+  // optional: C *= sigmoid(gate[r * ld_gate + h * c_hs + j])
+  const float* gate; int ld_gate;
+  // optional rotated query part, finished by the same launch (rot_dim > 0): C[r, h, J + i] = rot(A[r, h, K + i]) for
+  // i < rot_dim at position *pos_ptr + r % L
+  const float* inv_freq; const int* pos_ptr; int L, rot_dim, rot_dims, rot_layout;
 };
 cudaError_t launch_head_gemm(const HeadGemmArgs& a, bool w_bf16, cudaStream_t s);
 struct LatentAttnArgs {
@@ -126,6 +154,7 @@ struct LatentAttnArgs {
   float* out;            // [B * L, H, Dv]
   const float* gate;     // head h of row r is multiplied by sigmoid(gate[r * ld_gate + h]) (null: none)
   int ld_gate;
+  const float* sink;     // [H] the softmax denominator of head h also holds exp(sink[h]) (null: none)
   const int* pos_ptr;    // keys [0, *pos_ptr + t] are visible to token t
   float scale;
   int B, L, H, Dk, Dv, M;

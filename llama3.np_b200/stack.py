@@ -21,7 +21,7 @@ SOFTMAX, DECAY_LINEAR, GATED_DELTA = _cabi.MIX_SOFTMAX, _cabi.MIX_DECAY_LINEAR, 
 LATENT, MINGRU, DIFF = _cabi.MIX_LATENT, _cabi.MIX_MINGRU, _cabi.MIX_DIFF
 WINDOW, SSD, GLA = _cabi.MIX_WINDOW, _cabi.MIX_SSD, _cabi.MIX_GLA
 ATTN_SINK, ATTN_SIGMOID = _cabi.ATTN_SINK, _cabi.ATTN_SIGMOID
-FF_GLU, FF_POLYNORM = _cabi.FF_GLU, _cabi.FF_POLYNORM
+FF_GLU, FF_POLYNORM, FF_RELU2 = _cabi.FF_GLU, _cabi.FF_POLYNORM, _cabi.FF_RELU2
 ROUTE_SOFTMAX, ROUTE_SIGMOID_IN = _cabi.ROUTE_SOFTMAX, _cabi.ROUTE_SIGMOID_IN
 _DTYPES = {"float32": _cabi.DTYPE_F32, "fp32": _cabi.DTYPE_F32, "bfloat16": _cabi.DTYPE_BF16, "bf16": _cabi.DTYPE_BF16}
 
@@ -53,18 +53,21 @@ class LayerSpec:
     window: int = 0               # DIFF: keys a query sees, itself included; 0 = all
     diff: float = 0.0             # DIFF: constant of lambda and of the output multiplier 1 - diff
     rot_scaling: Optional[Tuple[float, float, float, int]] = None   # DIFF: (factor, low, high, original) or None
-    ff_kind: int = 0              # FF_GLU | FF_POLYNORM
+    ff_kind: int = 0              # FF_GLU | FF_POLYNORM | FF_RELU2
     router_kind: int = 0          # ROUTE_SOFTMAX | ROUTE_SIGMOID_IN
     shared_ff: int = 0            # ROUTE_SIGMOID_IN: width of the shared expert
     keep_first: int = 0           # WINDOW: the first tokens that stay visible behind the window
     attn_kind: int = 0            # WINDOW: ATTN_SINK (softmax with a sink per head) | ATTN_SIGMOID (sigmoid(score + bias), not normalised)
-    rot_layout: int = 0           # WINDOW: 0 = entries (2i, 2i + 1) turn together, 1 = entries (i, i + rot_dims / 2)
+    rot_layout: int = 0           # WINDOW, LATENT: 0 = entries (2i, 2i + 1) turn together, 1 = entries (i, i + rot_dims / 2)
     qk_unit: bool = False         # WINDOW: q and k over their root mean square per head, after the rotation
     out_norm_groups: int = 1      # SSD: parts of the output norm
     tau: float = 1.0              # GLA: the decay is sigmoid(.)^(1 / tau)
     pair: Optional["LayerSpec"] = None   # a second mixer on the same input (tensors mix.left.* / mix.right.*)
     mix_scale: float = 1.0        # with `pair`: result = mix_scale * mixer + pair_scale * pair mixer
     pair_scale: float = 1.0
+    kv_from: Optional[int] = None  # LATENT: the layer whose cache rows this one attends over (None: its own)
+    sink: bool = False            # LATENT: a learned logit per head in the softmax denominator
+    gate_wide: bool = False       # LATENT: the output gate has one entry per value instead of one per head
 
 
 @dataclass
@@ -84,13 +87,16 @@ class StackConfig:
     loop: Optional[Tuple[int, int, int]] = None   # (start, stop, times): layers [start, stop) run `times` times
     parallel: bool = False        # one norm per layer, the mixer and the feed-forward both read it
     norm_center: bool = False     # norms subtract the mean (layer norm with a weight, no bias)
-    layer_scale: bool = False     # per-channel multipliers l<i>.ls1 / ls2 on the sublayers' results
+    layer_scale: bool = False     # per-channel multipliers l<i>.ls1 / ls2 on the sublayers' results (parallel and pre-norm layers)
     canon_taps: int = 0           # taps of the causal convolution ahead of every sublayer; 0 = none
     depth_avg: bool = False       # the stream handed on is a weighted sum of every earlier layer's result
     norm_groups: int = 1          # pre-norm stacks: every norm cuts the vector into this many parts, each over its own RMS
     embed_norm: bool = False      # the embedding rows pass a norm (tensor embed.norm)
     loop_in: bool = False         # ahead of every pass of the loop x <- W [x ; x0] (tensor loop.in) instead of x + loop.step[pass]
     logit_softcap: float = 0.0    # c > 0: logits <- c tanh(logits / c)
+    streams: int = 0              # pre-norm stacks: residual rows per token (0: one row, plain sums), mixed by l<i>.hc1 / hc2 tensors
+    tied_head: bool = False       # the output projection is the embedding table
+    logit_scale: float = 1.0      # multiplier of the logits
     max_seq_len: int = 256
     max_batch_size: int = 1
     dtype: str = "float32"
@@ -133,7 +139,9 @@ class StackDecoder:
                                          keep_first=l.keep_first, attn_kind=l.attn_kind, rot_layout=l.rot_layout,
                                          qk_unit=int(l.qk_unit), out_norm_groups=l.out_norm_groups, tau=float(l.tau),
                                          pair=C.pointer(pair) if pair is not None else None,
-                                         mix_scale=float(l.mix_scale), pair_scale=float(l.pair_scale))
+                                         mix_scale=float(l.mix_scale), pair_scale=float(l.pair_scale),
+                                         kv_source=0 if l.kv_from is None else int(l.kv_from) + 1, sink=int(l.sink),
+                                         gate_wide=int(l.gate_wide))
 
         for i, l in enumerate(cfg.layers):
             specs[i] = c_spec(i, l)
@@ -147,7 +155,8 @@ class StackDecoder:
                                 loop_times=cfg.loop[2] if cfg.loop else 0, parallel=int(cfg.parallel),
                                 norm_center=int(cfg.norm_center), layer_scale=int(cfg.layer_scale),
                                 canon_taps=int(cfg.canon_taps), depth_avg=int(cfg.depth_avg), norm_groups=int(cfg.norm_groups),
-                                embed_norm=int(cfg.embed_norm), loop_in=int(cfg.loop_in), logit_softcap=float(cfg.logit_softcap))
+                                embed_norm=int(cfg.embed_norm), loop_in=int(cfg.loop_in), logit_softcap=float(cfg.logit_softcap),
+                                streams=int(cfg.streams), tied_head=int(cfg.tied_head), logit_scale=float(cfg.logit_scale))
         _cabi.check(self._lib.l3_create_stack(C.byref(c), specs, C.byref(self._h)))
         n = C.c_int()
         _cabi.check(self._lib.l3_stack_runs(self._h, C.byref(n)), self._h)
@@ -299,7 +308,7 @@ class StackDecoder:
 
     def read_state(self, layer: int, slot: int = 0):
         """(S [heads, dim, vdim], conv tail [channels, taps - 1] or None) of a recurrent layer run's slot; for a
-        latent-attention run S is its cache `[max_seq_len, kv_rank + rot_dim]`.  `layer` counts layer runs."""
+        latent-attention run S is the cache it reads, `[max_seq_len, kv_rank + rot_dim]`.  `layer` counts layer runs."""
         l = self.cfg.layers[self.run_layer(layer)]
         if l.pair is not None and l.mixer == WINDOW:   # two mixers side by side: the recurrent one
             l = l.pair
