@@ -740,12 +740,14 @@ static int enqueue_prefill(L3Model* m, const int32_t* d_ids, int B, int L, int s
     if (rc != L3_OK) return rc;
   }
   LAUNCH(m, launch_set_int(d_pos, start_pos, m->stream));
+  if (m->ll) m->ll->keys_end = start_pos + L;
   if (d_rows || d_resid)  // chosen rows / the residual trace index the whole block: one chunk (checked by the caller)
     return enqueue_chunk(m, d_ids, L, 0, B, L, want_logits, want_argmax, os, nullptr, d_rows, n_rows, d_resid);
   const int lc_max = std::max(1, m->cap_tok / B);
   for (int l0 = 0; l0 < L; l0 += lc_max) {
     const int lc = std::min(lc_max, L - l0);
     const bool last = l0 + lc >= L;
+    if (m->ll) m->ll->keys_end = start_pos + l0 + lc;
     int rc = enqueue_chunk(m, d_ids, L, l0, B, lc, last && want_logits, last && want_argmax, os);
     if (rc != L3_OK) return rc;
     if (!last) LAUNCH(m, launch_add_int(d_pos, lc, m->stream));
@@ -793,7 +795,7 @@ extern "C" int l3_forward(L3Model* m, const int32_t* ids, int B, int L, int star
   if (argmax_out)
     CK(m, cudaMemcpyAsync(argmax_out, m->d_fwd_arg, (size_t)B * 8, cudaMemcpyDeviceToHost, m->stream));
   CK(m, cudaStreamSynchronize(m->stream));
-  return L3_OK;
+  return ll_check(m);
 }
 
 extern "C" int l3_forward_rows(L3Model* m, const int32_t* ids, int B, int L, int start_pos, const int32_t* rows, int n_rows,
@@ -829,7 +831,7 @@ extern "C" int l3_forward_rows(L3Model* m, const int32_t* ids, int B, int L, int
   if (rc != L3_OK) return rc;
   CK(m, e);
   CK(m, e2);
-  return L3_OK;
+  return ll_check(m);
 }
 
 // ------------------------------------------------------------------------------ greedy loop
@@ -999,10 +1001,10 @@ extern "C" int l3_generate_greedy(L3Model* m, const int32_t* ids, int B, int L, 
   CK(m, cudaMemcpy2DAsync(out, (size_t)n_out * 8, m->d_tokens, (size_t)m->M * 8, (size_t)n_out * 8, B,
                           cudaMemcpyDeviceToHost, m->stream));
   CK(m, cudaStreamSynchronize(m->stream));
-  return L3_OK;
+  return ll_check(m);
 }
 
-// Greedy generation for prompts of DIFFERENT lengths (SURVEY.md 8(f)-2; the reference handles equal
+// Greedy generation for prompts of DIFFERENT lengths (the reference handles equal
 // lengths only and checks EOS for row 0 in the caller, llama3.py:341-343).  Each sequence behaves exactly
 // as if it ran alone through Llama.generate (pos_offset 0) or llama_generate (pos_offset -1): the
 // right-padded prompt rows are prefilled together, padding leaves the KV cache untouched, the LM head
@@ -1086,7 +1088,7 @@ extern "C" int l3_generate_next(L3Model* m, int64_t* out_B) {
   CK(m, cudaMemcpyAsync(m->h_next, m->d_next, (size_t)m->gen_B * 4, cudaMemcpyDeviceToHost, m->stream));
   CK(m, cudaStreamSynchronize(m->stream));
   for (int b = 0; b < m->gen_B; ++b) out_B[b] = m->h_next[b];
-  return L3_OK;
+  return ll_check(m);
 }
 
 // ------------------------------------------------------------------------------ measurement helpers
@@ -1094,7 +1096,7 @@ extern "C" int l3_sync(L3Model* m) {
   if (!m) return L3_EINVAL;
   CK(m, cudaSetDevice(m->cfg.device));
   CK(m, cudaStreamSynchronize(m->stream));
-  return L3_OK;
+  return ll_check(m);
 }
 extern "C" int l3_timer_start(L3Model* m) {
   if (!m) return L3_EINVAL;

@@ -24,6 +24,9 @@
 //                 the same rows (attn_latent.cu), gate per head -> values out of the latent per head (Wuv o)
 //                 Variants: a layer may read ANOTHER layer's rows (kv_source: no dkv rows in its projection), the softmax may
 //                 have a sink per head, the gate may be one value per output (then applied where the values are expanded)
+//                 Prompts in bf16 mode (sizes in multiples of 8): the sequence's cache rows are expanded to per-head keys and
+//                 values by one GEMM, queries packed as an operand, attention on the tensor cores (attn_latent_tc.cu), both
+//                 kinds of gate in its epilogue
 //   minGRU        fused z|x|g projection -> element-wise gated recurrence (prenorm_ops.cu)
 //   and a feed-forward that is a mixture of experts (moe.cu): fp32 router -> few rows: only the chosen experts' weights
 //   are read; many rows: ONE up-projection over all experts, relu^2 times the routing weight (zero where not chosen),
@@ -295,8 +298,9 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
       if (!s.kv_source) AL(L.k_norm, (size_t)s.kv_rank * 4);
       if (s.sink) AL(L.head_vec, (size_t)H * 4);
       AL(L.w_uq, (size_t)H * (DK + s.rot_dim) * s.q_rank * w);
-      AL(L.w_uk, (size_t)H * DK * s.kv_rank * w);
-      AL(L.w_uv, (size_t)H * DV * s.kv_rank * w);
+      const size_t ukv = (size_t)H * (DK + DV) * (s.kv_rank + s.rot_dim) * w;
+      AL(L.w_ukv, ukv);
+      cudaMemset(L.w_ukv, 0, ukv);
       AL(L.inv_freq, (size_t)std::max(1, s.rot_dims / 2) * 4);
       std::vector<float> f(std::max(1, s.rot_dims / 2), 0.f);
       for (int j = 0; j < s.rot_dims / 2; ++j) f[j] = (float)pow(s.rot_base, -2.0 * j / s.rot_dims);
@@ -643,8 +647,8 @@ static bool ll_place(L3Model* m, const std::string& name, LLPlace* p) {
     if (r == "mix.dq.norm") return vec(L.q_norm, s.q_rank, 1.f, 0.1f);
     if (r == "mix.dkv.norm") return vec(L.k_norm, s.kv_rank, 1.f, 0.1f);
     if (r == "mix.uq") { const bool ok = mat(L.w_uq, (int64_t)H * (DK + s.rot_dim), s.q_rank); p->scale *= 2.f; return ok; }
-    if (r == "mix.uk") { const bool ok = mat(L.w_uk, (int64_t)H * DK, s.kv_rank); p->scale *= 2.f; return ok; }
-    if (r == "mix.uv") return mat(L.w_uv, (int64_t)H * DV, s.kv_rank);
+    if (r == "mix.uk") { const bool ok = mat(L.w_ukv, (int64_t)H * DK, s.kv_rank); p->ld = s.kv_rank + s.rot_dim; p->scale *= 2.f; return ok; }
+    if (r == "mix.uv") { const bool ok = mat(L.w_ukv, (int64_t)H * DV, s.kv_rank, H * DK); p->ld = s.kv_rank + s.rot_dim; return ok; }
     return false;
   }
   if (s.mixer == L3_MIX_DIFF) {
@@ -866,6 +870,13 @@ static int ll_reset_unit_state(L3Model* m, const L3LayerSpec& s, LLState& St, in
   return L3_OK;
 }
 
+// do prompts of this latent-attention layer run on the tensor cores?
+static bool ll_latent_on_tc(const L3Model* m, const L3LayerSpec& s) {
+  static const bool off = getenv("L3_LATENT_TC") && atoi(getenv("L3_LATENT_TC")) == 0;
+  return !off && m->tc_ok && s.mixer == L3_MIX_LATENT && s.scale > 0.f && s.kv_rank + s.rot_dim >= 64 && s.heads * (s.dim + s.vdim) >= 64 &&
+         latent_tc_supported(s.dim, s.rot_dim, s.vdim, s.kv_rank);
+}
+
 int ll_finalize(L3Model* m) {
   LayerList* ll = m->ll;
   for (const auto& name : ll_expected(m))
@@ -1035,6 +1046,21 @@ int ll_finalize(L3Model* m) {
     if (ll->hf) CK(m, cudaMalloc(&ll->hf16, ct * W * 2));
     if (ll->cat) CK(m, cudaMalloc(&ll->cat16, ct * 2 * W * 2));
   }
+  CK(m, cudaHostAlloc((void**)&ll->h_err, sizeof(int), cudaHostAllocMapped));
+  *ll->h_err = 0;
+  size_t q_ld = 0, e_ld = 0;
+  for (auto& L : ll->layers)
+    if (ll_latent_on_tc(m, L.spec)) {
+      q_ld = std::max(q_ld, (size_t)L.spec.heads * latent_tc_q_ld(L.spec.dim, L.spec.rot_dim));
+      e_ld = std::max(e_ld, (size_t)L.spec.heads * (L.spec.dim + L.spec.vdim));
+    }
+  if (e_ld && ct > 8) {
+    const size_t per = (size_t)m->M * e_ld * 2;  // one sequence's keys and values; sequences share the workspace in turns
+    ll->exp_seqs = (int)std::max<size_t>(1, std::min<size_t>(m->maxB, ((size_t)1 << 30) / per));
+    CK(m, cudaMalloc(&ll->lat_q16, ct * q_ld * 2));
+    CK(m, cudaMalloc(&ll->lat_exp, ll->exp_seqs * per));
+    CK(m, cudaMemsetAsync(ll->lat_exp, 0, ll->exp_seqs * per, m->stream));  // never anything but finite numbers
+  }
   m->max_split = 32;
   int max_hn = 1, max_hd = 1;
   for (auto& L : ll->layers)
@@ -1076,7 +1102,7 @@ void ll_destroy(L3Model* m) {
     fr(L.w_in); fr(L.w_o); fr(L.w_a2); fr(L.w_g2); fr(L.w13); fr(L.w2); fr(L.side_gate); fr(L.side_proj);
     fr(L.norm1); fr(L.norm2); fr(L.side_norm); fr(L.mix_norm); fr(L.q_norm); fr(L.k_norm); fr(L.conv_w);
     fr(L.A_log); fr(L.dt_bias); fr(L.decay);
-    fr(L.w_uq); fr(L.w_uk); fr(L.w_uv); fr(L.inv_freq); fr(L.in_bias); fr(L.shift); fr(L.router); fr(L.correction);
+    fr(L.w_uq); fr(L.w_ukv); fr(L.inv_freq); fr(L.in_bias); fr(L.shift); fr(L.router); fr(L.correction);
     fr(L.canon1); fr(L.canon2); fr(L.canon1t); fr(L.canon2t); fr(L.ls1); fr(L.ls2); fr(L.dwa); fr(L.lam_vec); fr(L.lambda); fr(L.poly);
     fr(L.head_vec); fr(L.conv_b); fr(L.skip_d); fr(L.a2_bias);
     for (int q = 0; q < 2 && ll->cfg.streams > 0; ++q) { fr(L.hc_in[q]); fr(L.hc_out[q]); fr(L.hc_mix[q]); }
@@ -1094,6 +1120,8 @@ void ll_destroy(L3Model* m) {
   fr(ll->loop_in); fr(ll->embed_norm); fr(ll->x0); fr(ll->cat); fr(ll->cat16); fr(ll->win_part_o); fr(ll->win_part_ml); fr(ll->xs);
   fr(ll->diff_part_o); fr(ll->diff_part_ml);
   fr(ll->Xs); fr(ll->hn); fr(ll->hf); fr(ll->hf16); fr(ll->y1); fr(ll->y2); fr(ll->moe_gu);
+  fr(ll->lat_q16); fr(ll->lat_exp);
+  if (ll->h_err) cudaFreeHost(ll->h_err);
   fr(ll->loop_step); fr(ll->qlat); fr(ll->aux16); fr(ll->moe_sel); fr(ll->moe_w); fr(ll->moe_dense); fr(ll->moe_idw);
   fr(ll->pin); fr(ll->aux); fr(ll->rk); fr(ll->rv); fr(ll->rg); fr(ll->rbeta); fr(ll->o); fr(ll->sg); fr(ll->sg16); fr(ll->x2); fr(ll->chunk_ws);
   delete ll;
@@ -1144,6 +1172,13 @@ int ll_reset_slots(L3Model* m, int slot0, int n, bool kv_too) {
   }
   for (int b = slot0; b < slot0 + n; ++b) ll->slot_pos[b] = 0;
   return L3_OK;
+}
+
+int ll_check(L3Model* m) {
+  if (!m->ll || !m->ll->h_err || !*(volatile int*)m->ll->h_err) return L3_OK;
+  *m->ll->h_err = 0;
+  set_err(m, "a kernel gave up waiting for its own pipeline; the results of this call are not valid");
+  return L3_ESTATE;
 }
 
 int ll_begin_call(L3Model* m, int B, int L, int start_pos) {
@@ -1369,6 +1404,43 @@ static int ll_mix_unit(L3Model* m, LLLayer& Ly, LLState& St, const float* pin, i
   return L3_OK;
 }
 
+// Attention of a prompt (portion) on the tensor cores, from the query up-projection's output (m->q) to the output
+// projection's input: pack the queries, then - sequences in groups that fit the workspace - expand every cached row so far to
+// keys and values and attend.
+static int ll_latent_prompt(L3Model* m, LLLayer& Ly, LLState& St, int B, int L) {
+  LayerList* ll = m->ll;
+  const L3LayerSpec& s = Ly.spec;
+  const int ntok = B * L, H = s.heads, DK = s.dim, DV = s.vdim, Dk = s.kv_rank + s.rot_dim, n_exp = H * (DK + DV);
+  int* d_pos = m->d_scal + 0;
+  LatentQPackArgs qa{};
+  qa.q = m->q; qa.q16 = (bf16*)ll->lat_q16; qa.inv_freq = Ly.inv_freq; qa.pos_ptr = d_pos;
+  qa.L = L; qa.H = H; qa.dim = DK; qa.rot_dim = s.rot_dim; qa.rot_dims = s.rot_dims; qa.rot_layout = s.rot_layout;
+  LAUNCH(m, launch_latent_q_pack(qa, ntok, m->stream));
+  LatentTcArgs at{};
+  at.q16 = qa.q16; at.expand = (const bf16*)ll->lat_exp; at.cache = (const bf16*)St.lat; at.out16 = (bf16*)m->ctx16;
+  at.out = ll_takes_mirror(m, ntok, m->D, H * DV) ? nullptr : m->ctx;
+  at.gate = ll->pin + Ly.off_g; at.ld_gate = Ly.n_in; at.gate_wide = s.gate_wide; at.sink = s.sink ? Ly.head_vec : nullptr;
+  at.pos_ptr = d_pos; at.scale = s.scale; at.err = ll->h_err;
+  at.n_rows = ntok; at.L = L; at.H = H; at.dim = DK; at.rot_dim = s.rot_dim; at.vdim = DV; at.kv_rank = s.kv_rank; at.M = m->M;
+  at.c_seqs = m->maxB; at.e_rows = m->M; at.e_seqs = ll->exp_seqs;
+  // rows to expand: up to the chunk's last token, in steps of 128 (few distinct tensor maps; the surplus rows are stale but finite)
+  const int T = std::min(m->M, (ll->keys_end + 127) / 128 * 128);
+  for (int b0 = 0; b0 < B; b0 += ll->exp_seqs) {
+    const int n = std::min(ll->exp_seqs, B - b0);
+    for (int i = 0; i < n; ++i) {
+      const bf16* rows = (const bf16*)St.lat + (size_t)(b0 + i) * m->M * Dk;
+      TcGemmArgs t{};
+      t.kind = TC_BF16; t.A[0] = rows; t.W[0] = Ly.w_ukv; t.rows = T; t.N = n_exp; t.K = Dk; t.epi = EPI_STORE;
+      t.e = store_to(nullptr, (bf16*)ll->lat_exp + (size_t)i * m->M * n_exp, n_exp);
+      t.part = m->gemm_part; t.part_bytes = (size_t)32 << 20; t.tile_cnt = m->gemm_cnt; t.tile_cnt_len = 1024;
+      LAUNCH(m, launch_gemm_tc(t, m->stream));
+    }
+    at.b0 = b0;
+    LAUNCH(m, launch_attn_latent_tc(at, n, m->stream));
+  }
+  return L3_OK;
+}
+
 static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
   LayerList* ll = m->ll;
   const int ntok = B * L, W = m->D;
@@ -1442,34 +1514,38 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
       pa.rot_layout = s.rot_layout;
       LAUNCH(m, launch_latent_prep(pa, ntok, m->bf16, m->stream));
       if ((rc = ll_linear(m, Ly.w_uq, ll->aux, ll->aux16, 0, ntok, nq, s.q_rank, EPI_STORE, store_to(m->q, nullptr, nq))) != L3_OK) return rc;
-      // queries onto the latent: qlat[r, h] = [Wuk_h^T q_c | rot(q_r)]
-      HeadGemmArgs ga{};
-      ga.A = m->q; ga.lda = nq; ga.a_hs = DK + s.rot_dim;
-      ga.W = Ly.w_uk; ga.w_hs = (int64_t)DK * s.kv_rank; ga.w_ks = s.kv_rank; ga.w_js = 1;
-      ga.C = ll->qlat; ga.C16 = nullptr; ga.ldc = H * Dk; ga.c_hs = Dk;
-      ga.rows = ntok; ga.H = H; ga.J = s.kv_rank; ga.K = DK;
-      ga.inv_freq = Ly.inv_freq; ga.pos_ptr = d_pos; ga.L = L; ga.rot_dim = s.rot_dim; ga.rot_dims = s.rot_dims; ga.rot_layout = s.rot_layout;
-      LAUNCH(m, launch_head_gemm(ga, m->bf16, m->stream));
-      LatentAttnArgs at{};
-      at.q = ll->qlat; at.cache = St.lat; at.out = ll->o; at.gate = s.gate_wide ? nullptr : ll->pin + Ly.off_g; at.ld_gate = Ly.n_in;
-      at.sink = s.sink ? Ly.head_vec : nullptr;
-      at.pos_ptr = d_pos; at.scale = s.scale; at.B = B; at.L = L; at.H = H; at.Dk = Dk; at.Dv = s.kv_rank; at.M = m->M;
-      at.part_o = m->part_o; at.part_ml = m->part_ml;
-      at.nsplit = 1;
-      if (L == 1) {  // decode: the keys of a sequence spread over CTAs
-        const int ctas = B * ((H + 31) / 32);
-        at.nsplit = std::max(1, std::min(std::min(m->max_split, m->M / 64), (2 * 148) / std::max(1, ctas)));
+      if (L > 8 && ll->lat_exp && ll_latent_on_tc(m, s)) {
+        if ((rc = ll_latent_prompt(m, Ly, St, B, L)) != L3_OK) return rc;
+      } else {
+        // queries onto the latent: qlat[r, h] = [Wuk_h^T q_c | rot(q_r)]
+        HeadGemmArgs ga{};
+        ga.A = m->q; ga.lda = nq; ga.a_hs = DK + s.rot_dim;
+        ga.W = Ly.w_ukv; ga.w_hs = (int64_t)DK * Dk; ga.w_ks = Dk; ga.w_js = 1;
+        ga.C = ll->qlat; ga.C16 = nullptr; ga.ldc = H * Dk; ga.c_hs = Dk;
+        ga.rows = ntok; ga.H = H; ga.J = s.kv_rank; ga.K = DK;
+        ga.inv_freq = Ly.inv_freq; ga.pos_ptr = d_pos; ga.L = L; ga.rot_dim = s.rot_dim; ga.rot_dims = s.rot_dims; ga.rot_layout = s.rot_layout;
+        LAUNCH(m, launch_head_gemm(ga, m->bf16, m->stream));
+        LatentAttnArgs at{};
+        at.q = ll->qlat; at.cache = St.lat; at.out = ll->o; at.gate = s.gate_wide ? nullptr : ll->pin + Ly.off_g; at.ld_gate = Ly.n_in;
+        at.sink = s.sink ? Ly.head_vec : nullptr;
+        at.pos_ptr = d_pos; at.scale = s.scale; at.B = B; at.L = L; at.H = H; at.Dk = Dk; at.Dv = s.kv_rank; at.M = m->M;
+        at.part_o = m->part_o; at.part_ml = m->part_ml;
+        at.nsplit = 1;
+        if (L == 1) {  // decode: the keys of a sequence spread over CTAs
+          const int ctas = B * ((H + 31) / 32);
+          at.nsplit = std::max(1, std::min(std::min(m->max_split, m->M / 64), (2 * 148) / std::max(1, ctas)));
+        }
+        LAUNCH(m, launch_latent_attn(at, m->bf16, m->stream));
+        if (at.nsplit > 1) m->launch_acc += 1;
+        // values out of the latent: ctx[r, h] = Wuv_h o[r, h]
+        HeadGemmArgs gv{};
+        gv.A = ll->o; gv.lda = H * s.kv_rank; gv.a_hs = s.kv_rank;
+        gv.W = (char*)Ly.w_ukv + (size_t)H * DK * Dk * wb(m); gv.w_hs = (int64_t)DV * Dk; gv.w_ks = 1; gv.w_js = Dk;
+        gv.C = m->ctx16 && ll_takes_mirror(m, ntok, W, H * DV) ? nullptr : m->ctx; gv.C16 = (bf16*)m->ctx16; gv.ldc = H * DV; gv.c_hs = DV;
+        if (s.gate_wide) { gv.gate = ll->pin + Ly.off_g; gv.ld_gate = Ly.n_in; }
+        gv.rows = ntok; gv.H = H; gv.J = DV; gv.K = s.kv_rank;
+        LAUNCH(m, launch_head_gemm(gv, m->bf16, m->stream));
       }
-      LAUNCH(m, launch_latent_attn(at, m->bf16, m->stream));
-      if (at.nsplit > 1) m->launch_acc += 1;
-      // values out of the latent: ctx[r, h] = Wuv_h o[r, h]
-      HeadGemmArgs gv{};
-      gv.A = ll->o; gv.lda = H * s.kv_rank; gv.a_hs = s.kv_rank;
-      gv.W = Ly.w_uv; gv.w_hs = (int64_t)DV * s.kv_rank; gv.w_ks = 1; gv.w_js = s.kv_rank;
-      gv.C = m->ctx16 && ll_takes_mirror(m, ntok, W, H * DV) ? nullptr : m->ctx; gv.C16 = (bf16*)m->ctx16; gv.ldc = H * DV; gv.c_hs = DV;
-      if (s.gate_wide) { gv.gate = ll->pin + Ly.off_g; gv.ld_gate = Ly.n_in; }
-      gv.rows = ntok; gv.H = H; gv.J = DV; gv.K = s.kv_rank;
-      LAUNCH(m, launch_head_gemm(gv, m->bf16, m->stream));
     } else if (s.mixer == L3_MIX_MINGRU) {
       n_ctx = DK;
       LAUNCH(m, launch_mingru_scan(ll->pin, Ly.n_in, Ly.off_b, Ly.off_v, Ly.off_g, Ly.in_bias, St.S, B, L, DK, m->ctx, (bf16*)m->ctx16, m->stream));

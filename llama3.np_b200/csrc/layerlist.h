@@ -31,8 +31,9 @@ struct LLLayer {
   float* decay = nullptr;     // decay-linear: [heads]
   // latent attention: w_in = dq | dkv | g rows; q_norm / k_norm hold the two latent norms' weights
   void* w_uq = nullptr;       // [heads * (dim + rot_dim), q_rank]
-  void* w_uk = nullptr;       // [heads * dim, kv_rank]
-  void* w_uv = nullptr;       // [heads * vdim, kv_rank]
+  // [heads * dim | heads * vdim, kv_rank + rot_dim]: key, then value expansion, zero in the last rot_dim columns, so that ONE
+  // GEMM over whole cache rows expands both (prompts) while decode reads the first kv_rank columns
+  void* w_ukv = nullptr;
   float* inv_freq = nullptr;  // [rot_dims / 2] rot_base^(-2 i / rot_dims), rounded from double
   float* in_bias = nullptr;   // minGRU: [2 dim] biases of the z and x segments of w_in
   float* shift = nullptr;     // token shift: [width]
@@ -111,6 +112,11 @@ struct LayerList {
   // pre-norm / latent / mixture-of-experts workspace
   float* qlat = nullptr;                   // [rows, heads, kv_rank + rot_dim] queries folded onto the latent
   void* aux16 = nullptr;                   // bf16 mirror of aux (the query latent)
+  // latent attention of prompts on the tensor cores: packed queries, expanded keys | values of exp_seqs sequences
+  void *lat_q16 = nullptr, *lat_exp = nullptr;
+  int exp_seqs = 0;
+  int* h_err = nullptr;                    // pinned: a kernel sets it when one of its bounded waits ran out
+  int keys_end = 0;                        // position behind the last token of the chunk being enqueued
   float *moe_w = nullptr, *moe_dense = nullptr, *moe_idw = nullptr;  // [rows, top] | [rows, experts] | [rows]
   int32_t* moe_sel = nullptr;              // [rows, top]
   // parallel layers
@@ -135,6 +141,8 @@ void ll_destroy(L3Model* m);
 int ll_reset_slots(L3Model* m, int slot0, int n, bool kv_too);
 // position bookkeeping of a call that feeds L tokens to slots [0, B) at start_pos; start_pos 0 zeroes their state
 int ll_begin_call(L3Model* m, int B, int L, int start_pos);
+// after a synchronise: did a kernel of this handle give up waiting?
+int ll_check(L3Model* m);
 // all layers of one chunk; x in m->x (and its bf16 mirror) on entry and exit.  d_resid: null, or
 // [n_layers, B * L, width] receiving the residual stream after every layer
 int ll_enqueue_layers(L3Model* m, const int32_t* d_ids, int ids_ld, int ids_off, int B, int L, float* d_resid);

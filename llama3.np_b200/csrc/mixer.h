@@ -95,7 +95,7 @@ cudaError_t launch_prenorm_shift(const float* x, const float* w, float eps, cons
 cudaError_t launch_scale_add_rows(float* x, float mul, const float* vec, int rows, int D, cudaStream_t s);
 
 // ---- residual streams (stream_ops.cu)
-constexpr int STREAMS_MAX = 32;
+constexpr int STREAMS_MAX = 16;
 // One pass over the S residual rows of every token: apply the pending sublayer result y (null: none),
 //   X_t <- sum_s mix[s * S + t] X_s + out_w[t] * (ls * y)            (ls null: ones; written back when `store`)
 // and form what follows: the next sublayer's input  h = n(sum_s in_w[s] X_s)  with n the RMS norm of weight norm_w (norm_w
@@ -161,6 +161,34 @@ struct LatentAttnArgs {
   int nsplit;            // > 1 (L == 1 only): every split writes (o, m, l) to part_o / part_ml, the combine kernel merges
   float *part_o, *part_ml;
 };
+// Prompts in bf16 mode: attention over expanded keys and values on the tensor cores (attn_latent_tc.cu)
+struct LatentQPackArgs {
+  const float* q;        // [rows, H, dim + rot_dim]
+  bf16* q16;             // [rows, H, latent_tc_q_ld]: q_c, zeros to a multiple of 64, rot(q_r), zeros
+  const float* inv_freq;
+  const int* pos_ptr;
+  int L, H, dim, rot_dim, rot_dims, rot_layout;
+};
+struct LatentTcArgs {
+  const bf16* q16;       // [n_rows = B * L, H, latent_tc_q_ld]
+  const bf16* expand;    // [e_seqs * e_rows, H * dim | H * vdim]: keys and values of sequences b0 .., e_rows rows each (finite
+                         // values everywhere: what lies behind a sequence's last row meets weights of zero)
+  const bf16* cache;     // [c_seqs * M, kv_rank + rot_dim]
+  bf16* out16;           // [B * L, H * vdim], and / or fp32
+  float* out;
+  const float* gate;     // sigmoid(gate[r * ld_gate + h]), or with gate_wide + h * vdim + d, multiplies the output (null: none)
+  int ld_gate, gate_wide;
+  const float* sink;     // [H] or null
+  const int* pos_ptr;
+  float scale;           // > 0
+  int* err;              // set to 1 when a wait inside the kernel ran out
+  int n_rows, L, H, dim, rot_dim, vdim, kv_rank, M, c_seqs, b0, e_rows, e_seqs;
+};
+int latent_tc_q_ld(int dim, int rot_dim);  // entries of a packed query head
+bool latent_tc_supported(int dim, int rot_dim, int vdim, int kv_rank);
+cudaError_t launch_latent_q_pack(const LatentQPackArgs& a, int rows, cudaStream_t s);
+cudaError_t launch_attn_latent_tc(const LatentTcArgs& a, int n_seq, cudaStream_t s);
+
 size_t latent_attn_smem(int Dk);
 bool latent_attn_supported(int Dk, int Dv);
 cudaError_t launch_latent_attn(const LatentAttnArgs& a, bool kv_bf16, cudaStream_t s);

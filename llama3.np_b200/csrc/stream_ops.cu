@@ -76,22 +76,28 @@ __device__ __forceinline__ Row<VEC> advance(const StreamArgs& a, const StreamWei
       for (int k = 0; k < VEC; ++k) y.v[k] *= l.v[k];
     }
   }
+  if (!a.y) {
 #pragma unroll
-  for (int t = 0; t < NS; ++t) {
-    if (!EXACT && t >= S) break;
-    Row<VEC> n = x[t];
-    if (a.y) {
+    for (int s = 0; s < NS; ++s) {
+      if (!EXACT && s >= S) break;
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) n.v[k] = w.out[t] * y.v[k];
-#pragma unroll
-      for (int s = 0; s < NS; ++s) {
-        if (!EXACT && s >= S) break;
-        const float c = w.mix[s * S + t];
-#pragma unroll
-        for (int k = 0; k < VEC; ++k) n.v[k] = fmaf(c, x[s].v[k], n.v[k]);
-      }
-      if (a.store) n.store(Xr + (size_t)t * D);
+      for (int k = 0; k < VEC; ++k) { u.v[k] = fmaf(w.in[s], x[s].v[k], u.v[k]); total.v[k] += x[s].v[k]; }
     }
+    return u;
+  }
+#pragma unroll (EXACT ? NS : 1)
+  for (int t = 0; t < S; ++t) {
+    Row<VEC> n;
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) n.v[k] = w.out[t] * y.v[k];
+#pragma unroll
+    for (int s = 0; s < NS; ++s) {
+      if (!EXACT && s >= S) break;
+      const float c = w.mix[s * S + t];
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) n.v[k] = fmaf(c, x[s].v[k], n.v[k]);
+    }
+    if (a.store) n.store(Xr + (size_t)t * D);
     const float in = w.in[t];
 #pragma unroll
     for (int k = 0; k < VEC; ++k) { u.v[k] = fmaf(in, n.v[k], u.v[k]); total.v[k] += n.v[k]; }
