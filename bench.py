@@ -779,10 +779,45 @@ def debuzen_layer_params(cfg):
     return held, read
 
 
+# ------------------------------------------------------------------------------ --arch gifudra
+# Eight layers of latent attention over four residual streams (heads of 128 + 64 rotated, values 128, latent of 512, a gate
+# per value), the last four attending over layer 3's cache; relu^2 feed-forward of 4 x width.  Beside it the closest family at
+# equal size: Rakelorn with eight latent-attention layers of the same head sizes and 4 relu^2 experts of `width`, all of them
+# chosen (the same parameters held and read per token in the feed-forward).
+def gifudra_bench_config(width, vocab=32000):
+    heads = max(1, width // 128)
+    mixer = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": 3 * width // 4, "kv_rank": 512,
+             "scale": 192 ** -0.5, "rot": {"base": 10000.0, "dims": 64}}
+    layers = [{"type": "latent_attention", "mixer": dict(mixer, **({"kv_from": 3} if i >= 4 else {})),
+               "mlp": {"kind": "dense", "ff": 4 * width}} for i in range(8)]
+    return {"architecture": "Gifudra", "layers": layers, "norm": {"eps": 1e-5}, "streams": 4, "embedding": {"scale": 1.0},
+            "logit_scale": 1.0, "vocab": vocab, "width": width}
+
+
+def gifudra_layer_params(cfg):
+    W, tot = cfg["width"], 0
+    for lc in cfg["layers"]:
+        mc = lc["mixer"]
+        H, dn, dr, dv = mc["heads"], mc["dim"], mc["rot_dim"], mc["vdim"]
+        own = 0 if "kv_from" in mc else mc["kv_rank"] + dr
+        tot += W * (mc["q_rank"] + own + H * dv) + mc["q_rank"] * H * (dn + dr) + mc["kv_rank"] * H * (dn + dv) + W * H * dv
+        tot += 2 * W * lc["mlp"]["ff"]
+    return tot
+
+
+def rakelorn_like_gifudra(width, vocab=32000):
+    cfg = rakelorn_bench_config(width, vocab)
+    mlp = {"kind": "moe", "expert": {"ff": width}, "router": {"experts": 4, "top": 4, "identity": 0, "scale": 2.0}}
+    out = dict(cfg, layers=[dict(cfg["layers"][0], mlp=mlp)] * 8)
+    del out["loop"]
+    return out
+
+
 def run_arch_compare(a):
     import llama3_np_b200  # noqa: F401
     from llama3_np_b200 import Llama, ModelArgs, _cabi
     from llama3_np_b200.debuzen import Debuzen
+    from llama3_np_b200.gifudra import Gifudra
     from llama3_np_b200.mabedra import Mabedra
     from llama3_np_b200.rakelorn import Rakelorn
     from llama3_np_b200.risalix import Risalix
@@ -835,6 +870,9 @@ def run_arch_compare(a):
         elif a.arch == "debuzen":
             cfg = debuzen_bench_config(W)
             rp, rp_read = debuzen_layer_params(cfg)
+        elif a.arch == "gifudra":
+            cfg = gifudra_bench_config(W)
+            rp = rp_read = gifudra_layer_params(cfg)
         else:
             cfg = risalix_bench_config(W)
             rp = rp_read = risalix_layer_params(cfg)
@@ -844,7 +882,7 @@ def run_arch_compare(a):
         nl = max(1, round((rp_read if a.arch == "debuzen" else rp) / lp1))
         clock = ClockSampler(0)
         clock.start()
-        r = {"rakelorn": Rakelorn, "mabedra": Mabedra, "risalix": Risalix, "debuzen": Debuzen}[a.arch](cfg, None, dtype=dtype, max_seq_len=M, max_batch_size=8, random_seed=1)
+        r = {"rakelorn": Rakelorn, "mabedra": Mabedra, "risalix": Risalix, "debuzen": Debuzen, "gifudra": Gifudra}[a.arch](cfg, None, dtype=dtype, max_seq_len=M, max_batch_size=8, random_seed=1)
         # the decode leg streams what a token reads (chosen experts, looped layers once per pass), the prefill leg's
         # useful work is the same count per token
         rec_r = measure(r, cfg["vocab"], rp_read + cfg["vocab"] * W, True)
@@ -862,6 +900,12 @@ def run_arch_compare(a):
             rr = Risalix(rcfg, None, dtype=dtype, max_seq_len=M, max_batch_size=8, random_seed=1)
             extra["risalix"] = {"layers": n_ris, "params_in_layers": risalix_layer_params(rcfg),
                                 **measure(rr, rcfg["vocab"], risalix_layer_params(rcfg) + rcfg["vocab"] * W, True)}
+            rr.close()
+        if a.arch == "gifudra":
+            rcfg = rakelorn_like_gifudra(W)
+            held, read = rakelorn_layer_params(rcfg)
+            rr = Rakelorn(rcfg, None, dtype=dtype, max_seq_len=M, max_batch_size=8, random_seed=1)
+            extra["rakelorn"] = {"layers": len(rcfg["layers"]), "params_in_layers": held, **measure(rr, rcfg["vocab"], read + rcfg["vocab"] * W, True)}
             rr.close()
         clk = clock.stop()
         out.append({"size": name, "width": W, a.arch: {"layers": len(cfg["layers"]), "params_in_layers": rp, "params_read_per_token": rp_read, **rec_r},
@@ -882,7 +926,7 @@ def main():
     ap.add_argument("--total-len", type=int, default=256, help="profiling only: shorter generate")
     ap.add_argument("--no-cpu-baseline", action="store_true", help="profiling only: skip the CPU legs")
     ap.add_argument("--no-extra", action="store_true", help="headline only: skip the `extra` / `tp` sub-records")
-    ap.add_argument("--arch", default="", choices=["", "risalix", "rakelorn", "mabedra", "debuzen"],
+    ap.add_argument("--arch", default="", choices=["", "risalix", "rakelorn", "mabedra", "debuzen", "gifudra"],
                     help="instead of the headline: prefill / decode throughput of this decoder family beside Llama at equal size")
     ap.add_argument("--arch-sizes", default="w1024,w2048", help="comma list of " + ",".join(ARCH_SIZES))
     ap.add_argument("--arch-prefill", type=int, default=2048)
