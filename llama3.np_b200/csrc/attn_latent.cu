@@ -9,10 +9,11 @@
 //  * head_gemm_kernel          batched per-head product (Wuk_j^T q_c and Wuv_j ctx): 64 x 64 FFMA tiles, 4 x 4 per thread;
 //                              head_gemv_kernel for up to 8 rows (decode).  The launch that folds the queries also turns
 //                              their rotated part; the one that expands the values also applies an element-wise gate
-//  * attn_latent_kernel        flash-style exact attention: a CTA holds 32 (token, head) query rows in shared memory
-//                              and walks the visible cache rows 32 at a time; a lane scores one key for its warp's
-//                              four query rows, then the lanes own output columns.  Scores, weights and sums fp32.
-//                              Decode splits the keys over CTAs; attn_latent_combine_kernel merges the parts.  A sink
+//  * attn_latent_kernel        flash-style exact attention: a CTA holds up to 32 (token, head) query rows in shared
+//                              memory and walks the visible cache rows 32 at a time; a lane scores one key for its warp's
+//                              query rows, then the lanes own output columns.  Scores, weights and sums fp32.
+//                              Calls with few rows spread them over all warps and split the keys over CTAs;
+//                              attn_latent_combine_kernel merges the parts.  A sink
 //                              (one logit per head without a value) joins the denominator once, at the very end.
 #include <algorithm>
 
@@ -159,7 +160,8 @@ __global__ void __launch_bounds__(256) head_gemm_kernel(HeadGemmArgs a) {
 }
 
 // ---------------------------------------------------------------- attention over the latent cache
-constexpr int LA_ROWS = 32, LA_KT = 32, LA_RW = 4, LA_WARPS = 8, LA_PF = 10;
+constexpr int LA_KT = 32, LA_RW_MAX = 4, LA_WARPS = 8, LA_PF = 10;
+constexpr int LA_CTAS = 2 * 148;  // splits stop at two CTAs per SM
 
 __host__ __device__ inline int la_kstride(int Dk) {
   // 16-byte loads by 8 lanes at a time want an odd stride in 16-byte units; scalar loads an odd stride in words
@@ -178,10 +180,11 @@ __device__ __forceinline__ float latent_out_scale(const LatentAttnArgs& a, size_
   return g * c / fmaf(l, c, 1.0f);
 }
 
-// ND: output columns per lane (Dv <= 32 * ND)
-template <typename KVT, int ND>
+// ND: output columns per lane (Dv <= 32 * ND); RW: query rows per warp
+template <typename KVT, int ND, int LA_RW>
 __global__ void __launch_bounds__(256) attn_latent_kernel(LatentAttnArgs a) {
   extern __shared__ __align__(16) float sm[];
+  constexpr int LA_ROWS = LA_WARPS * LA_RW;
   const int Dk = a.Dk, Dv = a.Dv, KS = la_kstride(Dk), QS = (Dk + 3) & ~3;
   float* Qs = sm;                                    // [LA_ROWS][QS]
   float* Ks = Qs + LA_ROWS * QS;                     // [LA_KT][KS]
@@ -200,6 +203,13 @@ __global__ void __launch_bounds__(256) attn_latent_kernel(LatentAttnArgs a) {
     const int per = ((k_end + a.nsplit - 1) / a.nsplit + LA_KT - 1) / LA_KT * LA_KT;
     k_begin = split * per;
     k_end = min(k_end, k_begin + per);
+    if (k_begin >= k_end) {  // no keys for this split: weight zero, and the merge does not read the partial outputs
+      for (int rr = threadIdx.x; rr < rows_here; rr += blockDim.x) {
+        float* ml = a.part_ml + (((size_t)b * nrow + row0 + rr) * a.nsplit + split) * 2;
+        ml[0] = -INFINITY; ml[1] = 0.f;
+      }
+      return;
+    }
   }
   const float* qg = a.q + ((size_t)b * nrow + row0) * Dk;
   if (Dk % 4 == 0) {
@@ -285,7 +295,7 @@ __global__ void __launch_bounds__(256) attn_latent_kernel(LatentAttnArgs a) {
     __syncthreads();
     if (kvec && k0 + LA_KT < k_end) issue(k0 + LA_KT);
     // scores: lane = key
-    float s[LA_RW] = {0.f, 0.f, 0.f, 0.f};
+    float s[LA_RW] = {};
     if (lane < nk) {
       const float* kr = Ks + lane * KS;
       const float* q0 = Qs + (warp * LA_RW) * QS;
@@ -321,17 +331,22 @@ __global__ void __launch_bounds__(256) attn_latent_kernel(LatentAttnArgs a) {
 #pragma unroll
       for (int c = 0; c < ND; ++c) acc[i][c] *= alpha;
     }
-    *reinterpret_cast<float4*>(Pw + lane * LA_RW) = make_float4(p[0], p[1], p[2], p[3]);
+    if constexpr (LA_RW == 4) *reinterpret_cast<float4*>(Pw + lane * LA_RW) = make_float4(p[0], p[1], p[2], p[3]);
+    else if constexpr (LA_RW == 2) *reinterpret_cast<float2*>(Pw + lane * LA_RW) = make_float2(p[0], p[1]);
+    else Pw[lane] = p[0];
     __syncwarp();
     for (int j = 0; j < nk; ++j) {
-      const float4 pj = *reinterpret_cast<const float4*>(Pw + j * LA_RW);
+      float pj[LA_RW];
+      if constexpr (LA_RW == 4) { const float4 t = *reinterpret_cast<const float4*>(Pw + j * LA_RW); pj[0] = t.x; pj[1] = t.y; pj[2] = t.z; pj[3] = t.w; }
+      else if constexpr (LA_RW == 2) { const float2 t = *reinterpret_cast<const float2*>(Pw + j * LA_RW); pj[0] = t.x; pj[1] = t.y; }
+      else pj[0] = Pw[j];
       const float* vr = Ks + j * KS;
 #pragma unroll
       for (int c = 0; c < ND; ++c) {
         const int d = lane + 32 * c;
         const float v = d < Dv ? vr[d] : 0.f;
-        acc[0][c] = fmaf(pj.x, v, acc[0][c]); acc[1][c] = fmaf(pj.y, v, acc[1][c]);
-        acc[2][c] = fmaf(pj.z, v, acc[2][c]); acc[3][c] = fmaf(pj.w, v, acc[3][c]);
+#pragma unroll
+        for (int i = 0; i < LA_RW; ++i) acc[i][c] = fmaf(pj[i], v, acc[i][c]);
       }
     }
     __syncwarp();
@@ -356,28 +371,41 @@ __global__ void __launch_bounds__(256) attn_latent_kernel(LatentAttnArgs a) {
   }
 }
 
+// merge of the splits: a CTA per (query row, 128 output columns)
 __global__ void __launch_bounds__(128) attn_latent_combine_kernel(LatentAttnArgs a) {
-  __shared__ float wsplit[64];
+  __shared__ float wsplit[LA_CTAS], red[8];
   pdl_launch();
   pdl_wait();
   const size_t row = blockIdx.x;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const float* ml = a.part_ml + row * a.nsplit * 2;
   float mx = -INFINITY;
-  for (int s = 0; s < a.nsplit; ++s) mx = fmaxf(mx, ml[2 * s]);
-  if (threadIdx.x < a.nsplit) wsplit[threadIdx.x] = ml[2 * threadIdx.x] == -INFINITY ? 0.f : expf(ml[2 * threadIdx.x] - mx);
+  for (int s = threadIdx.x; s < a.nsplit; s += 128) mx = fmaxf(mx, ml[2 * s]);
+  mx = warp_max(mx);
+  if (lane == 0) red[warp] = mx;
   __syncthreads();
+  mx = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
   float l = 0.f;
-  for (int s = 0; s < a.nsplit; ++s) l = fmaf(wsplit[s], ml[2 * s + 1], l);
-  const size_t tok = row / a.H;
-  const int head = (int)(row - tok * a.H);
-  const float inv = latent_out_scale(a, tok, head, mx, l);
-  const float* po = a.part_o + row * a.nsplit * a.Dv;
-  for (int d = threadIdx.x; d < a.Dv; d += blockDim.x) {
-    float o = 0.f;
-#pragma unroll 8
-    for (int s = 0; s < a.nsplit; ++s) o = fmaf(wsplit[s], po[(size_t)s * a.Dv + d], o);
-    a.out[row * a.Dv + d] = o * inv;
+  for (int s = threadIdx.x; s < a.nsplit; s += 128) {
+    const float w = ml[2 * s] == -INFINITY ? 0.f : expf(ml[2 * s] - mx);
+    wsplit[s] = w;
+    l = fmaf(w, ml[2 * s + 1], l);
   }
+  l = warp_sum(l);
+  if (lane == 0) red[4 + warp] = l;
+  __syncthreads();
+  l = (red[4] + red[5]) + (red[6] + red[7]);
+  const int d = blockIdx.y * 128 + threadIdx.x;
+  if (d >= a.Dv) return;
+  const size_t tok = row / a.H;
+  const float* po = a.part_o + row * a.nsplit * a.Dv + d;
+  float o = 0.f;
+#pragma unroll 8
+  for (int s = 0; s < a.nsplit; ++s) {
+    const float w = wsplit[s];
+    if (w != 0.f) o = fmaf(w, po[(size_t)s * a.Dv], o);
+  }
+  a.out[row * a.Dv + d] = o * latent_out_scale(a, tok, (int)(row - tok * a.H), mx, l);
 }
 
 // Few rows (decode): the per-head product as matrix-vector products that stream the head's weights once.
@@ -415,38 +443,64 @@ __global__ void __launch_bounds__(256) head_gemv_kernel(HeadGemmArgs a) {
   if (a.C16) a.C16[o] = __float2bfloat16_rn(v);
 }
 
+// query rows per warp: few rows spread over all warps of a CTA
+int la_rw(int L, int H) { return L * H <= LA_WARPS ? 1 : L * H <= 2 * LA_WARPS ? 2 : LA_RW_MAX; }
+
+size_t la_smem(int Dk, int rw) {
+  return ((size_t)LA_WARPS * rw * ((Dk + 3) & ~3) + (size_t)LA_KT * la_kstride(Dk) + LA_WARPS * LA_KT * rw) * sizeof(float);
+}
+
+template <typename KVT, int ND, int RW>
+cudaError_t launch_la_t(const LatentAttnArgs& a, cudaStream_t s) {
+  static bool set = false;
+  if (!set) {
+    const cudaError_t e = cudaFuncSetAttribute(attn_latent_kernel<KVT, ND, RW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+    if (e != cudaSuccess) return e;
+    set = true;
+  }
+  const int rows = LA_WARPS * RW;
+  const dim3 grid((a.L * a.H + rows - 1) / rows, a.B, std::max(1, a.nsplit));
+  return launch_k(attn_latent_kernel<KVT, ND, RW>, grid, dim3(256), la_smem(a.Dk, RW), s, a);
+}
+
+template <typename KVT, int ND>
+cudaError_t launch_la_n(const LatentAttnArgs& a, cudaStream_t s) {
+  switch (la_rw(a.L, a.H)) {
+    case 1: return launch_la_t<KVT, ND, 1>(a, s);
+    case 2: return launch_la_t<KVT, ND, 2>(a, s);
+    default: return launch_la_t<KVT, ND, 4>(a, s);
+  }
+}
+
 template <typename KVT>
 cudaError_t launch_la(const LatentAttnArgs& a, cudaStream_t s) {
-  const int nrow = a.L * a.H;
-  const dim3 grid((nrow + LA_ROWS - 1) / LA_ROWS, a.B, std::max(1, a.nsplit));
-  const size_t smem = latent_attn_smem(a.Dk);
   const int nd = (a.Dv + 31) / 32;
-#define LA_CASE(N)                                                                                                        \
-  if (nd <= N) {                                                                                                          \
-    static bool set = false;                                                                                              \
-    if (!set) {                                                                                                           \
-      cudaFuncSetAttribute(attn_latent_kernel<KVT, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);          \
-      set = true;                                                                                                         \
-    }                                                                                                                     \
-    return launch_k(attn_latent_kernel<KVT, N>, grid, dim3(256), smem, s, a);                                             \
-  }
-  LA_CASE(1) LA_CASE(2) LA_CASE(4) LA_CASE(8) LA_CASE(16) LA_CASE(32)
-#undef LA_CASE
+  if (nd <= 1) return launch_la_n<KVT, 1>(a, s);
+  if (nd <= 2) return launch_la_n<KVT, 2>(a, s);
+  if (nd <= 4) return launch_la_n<KVT, 4>(a, s);
+  if (nd <= 8) return launch_la_n<KVT, 8>(a, s);
+  if (nd <= 16) return launch_la_n<KVT, 16>(a, s);
+  if (nd <= 32) return launch_la_n<KVT, 32>(a, s);
   return cudaErrorInvalidValue;
 }
 
 }  // namespace
 
-size_t latent_attn_smem(int Dk) {
-  return ((size_t)LA_ROWS * ((Dk + 3) & ~3) + (size_t)LA_KT * la_kstride(Dk) + LA_WARPS * LA_KT * LA_RW) * sizeof(float);
+size_t latent_attn_smem(int Dk) { return la_smem(Dk, LA_RW_MAX); }
+
+int latent_attn_splits(int B, int L, int H, int max_keys) {
+  const int rows = LA_WARPS * la_rw(L, H), ctas = B * ((L * H + rows - 1) / rows);
+  return std::max(1, std::min((max_keys + LA_KT - 1) / LA_KT, LA_CTAS / ctas));
 }
+
+size_t latent_attn_part_rows() { return (size_t)LA_CTAS * LA_WARPS * LA_RW_MAX; }
 
 bool latent_attn_supported(int Dk, int Dv) { return Dv >= 1 && Dv <= Dk && Dv <= 1024 && latent_attn_smem(Dk) <= 220 * 1024; }
 
 cudaError_t launch_latent_attn(const LatentAttnArgs& a, bool kv_bf16, cudaStream_t s) {
   cudaError_t e = kv_bf16 ? launch_la<bf16>(a, s) : launch_la<float>(a, s);
   if (e != cudaSuccess || a.nsplit <= 1) return e;
-  return launch_k(attn_latent_combine_kernel, dim3(a.B * a.L * a.H), dim3(128), 0, s, a);
+  return launch_k(attn_latent_combine_kernel, dim3(a.B * a.L * a.H, (a.Dv + 127) / 128), dim3(128), 0, s, a);
 }
 
 cudaError_t launch_latent_prep(const LatentPrepArgs& a, int rows, bool kv_bf16, cudaStream_t s) {

@@ -206,8 +206,8 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   float2* ml = reinterpret_cast<float2*>(smem_raw + (bars + 512 - raw));  // [group][row] (maximum, sum)
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int qt = gridDim.x - 1 - blockIdx.x;  // longest tiles (latest queries) first
-  const int head = blockIdx.y, bl = blockIdx.z, b = a.b0 + bl;
+  const int qt = gridDim.y - 1 - blockIdx.y;  // longest tiles (latest queries) of every head first
+  const int head = blockIdx.x, bl = blockIdx.z, b = a.b0 + bl;
   const int q0 = qt * BQ;
   pdl_launch();
 
@@ -478,6 +478,6 @@ cudaError_t launch_attn_latent_tc(const LatentTcArgs& a, int n_seq, cudaStream_t
   const CUtensorMap* me = tc_get_map(a.expand, true, a.e_seqs * a.e_rows, a.H * (a.dim + a.vdim), BKV);
   const CUtensorMap* mc = tc_get_map(a.cache, true, a.c_seqs * a.M, a.kv_rank + a.rot_dim, BKV);
   if (!mq || !me || !mc) return cudaErrorInvalidValue;
-  const dim3 grid((a.L + BQ - 1) / BQ, a.H, n_seq);
+  const dim3 grid(a.H, (a.L + BQ - 1) / BQ, n_seq);
   return launch_k(attn_latent_tc_kernel, grid, dim3(THREADS), (size_t)make_shape(a.dim, a.rot_dim, a.vdim).smem(), s, *mq, *me, *mc, a);
 }

@@ -883,7 +883,7 @@ int ll_finalize(L3Model* m) {
     if (!ll->loaded.count(name)) { set_err(m, "tensor '%s' was never loaded", name.c_str()); return L3_ESTATE; }
   if (m->stage) { cudaFree(m->stage); m->stage = nullptr; }
   const size_t kvb = m->bf16 ? 2 : 4;
-  int max_rq = 1, max_rk = 1, max_rv = 1, max_rg = 1, max_h = 1, max_aux = 1, max_qlat = 0, max_top = 0, max_exp = 0, max_hid = 1, max_gu = 0;
+  int max_rq = 1, max_rk = 1, max_rv = 1, max_rg = 1, max_h = 1, max_aux = 1, max_qlat = 0, max_lat = 0, max_top = 0, max_exp = 0, max_hid = 1, max_gu = 0;
   for (size_t ri = 0; ri < ll->runs.size(); ++ri) {
     const LLLayer& L = ll->layers[ll->runs[ri].layer];
     LLState& St = ll->state[ri];
@@ -957,6 +957,7 @@ int ll_finalize(L3Model* m) {
       max_rq = std::max(max_rq, H * (DK + s.rot_dim));
       max_aux = std::max(max_aux, s.q_rank);
       max_qlat = std::max(max_qlat, H * (s.kv_rank + s.rot_dim));
+      max_lat = std::max(max_lat, s.kv_rank);
     }
     if (s.experts > 0) { max_top = std::max(max_top, s.top); max_exp = std::max(max_exp, s.experts); max_hid = std::max(max_hid, (s.top + 1) * std::max(s.ff, s.shared_ff)); }
     max_gu = std::max(max_gu, 2 * L.ff_total);
@@ -981,7 +982,11 @@ int ll_finalize(L3Model* m) {
   CK(m, cudaMalloc((void**)&ll->rbeta, ct * max_h * 4));
   CK(m, cudaMalloc((void**)&ll->o, ct * ll->max_o * 4));
   CK(m, cudaMalloc((void**)&ll->sg, ct * std::max(1, sd) * 4));
-  if (max_qlat) CK(m, cudaMalloc((void**)&ll->qlat, ct * max_qlat * 4));
+  if (max_qlat) {
+    CK(m, cudaMalloc((void**)&ll->qlat, ct * max_qlat * 4));
+    CK(m, cudaMalloc((void**)&ll->lat_part_o, latent_attn_part_rows() * max_lat * 4));
+    CK(m, cudaMalloc((void**)&ll->lat_part_ml, latent_attn_part_rows() * 2 * 4));
+  }
   if (ll->streams) {
     CK(m, cudaMalloc((void**)&ll->X, ct * ll->streams * W * 4));
     CK(m, cudaMalloc((void**)&ll->y1, ct * W * 4));
@@ -1065,7 +1070,6 @@ int ll_finalize(L3Model* m) {
   int max_hn = 1, max_hd = 1;
   for (auto& L : ll->layers)
     if (L.spec.mixer == L3_MIX_SOFTMAX || L.spec.mixer == L3_MIX_DIFF) { max_hn = std::max(max_hn, L.spec.heads); max_hd = std::max(max_hd, L.spec.dim); }
-    else if (L.spec.mixer == L3_MIX_LATENT) { max_hn = std::max(max_hn, L.spec.heads); max_hd = std::max(max_hd, L.spec.kv_rank); }
   CK(m, cudaMalloc((void**)&m->part_o, (size_t)m->maxB * max_hn * m->max_split * max_hd * 4));
   CK(m, cudaMalloc((void**)&m->part_ml, (size_t)m->maxB * max_hn * m->max_split * 2 * 4));
   CK(m, cudaMalloc((void**)&m->attn_cnt, (size_t)m->maxB * max_hn * 4));
@@ -1120,7 +1124,7 @@ void ll_destroy(L3Model* m) {
   fr(ll->loop_in); fr(ll->embed_norm); fr(ll->x0); fr(ll->cat); fr(ll->cat16); fr(ll->win_part_o); fr(ll->win_part_ml); fr(ll->xs);
   fr(ll->diff_part_o); fr(ll->diff_part_ml);
   fr(ll->Xs); fr(ll->hn); fr(ll->hf); fr(ll->hf16); fr(ll->y1); fr(ll->y2); fr(ll->moe_gu);
-  fr(ll->lat_q16); fr(ll->lat_exp);
+  fr(ll->lat_q16); fr(ll->lat_exp); fr(ll->lat_part_o); fr(ll->lat_part_ml);
   if (ll->h_err) cudaFreeHost(ll->h_err);
   fr(ll->loop_step); fr(ll->qlat); fr(ll->aux16); fr(ll->moe_sel); fr(ll->moe_w); fr(ll->moe_dense); fr(ll->moe_idw);
   fr(ll->pin); fr(ll->aux); fr(ll->rk); fr(ll->rv); fr(ll->rg); fr(ll->rbeta); fr(ll->o); fr(ll->sg); fr(ll->sg16); fr(ll->x2); fr(ll->chunk_ws);
@@ -1258,21 +1262,30 @@ static int ll_settle(L3Model* m, LLPending& pd, int rows) {
   return L3_OK;
 }
 
+// Few rows stream the weights through the GEMV, which holds the rows in fp32 shared memory.  From five rows on every CTA of
+// it stages 8 K floats first, and the swapped-role GEMM on the tensor cores is faster; pre-norm stacks write the bf16
+// mirrors it reads for any number of rows.
+static bool ll_gemv(const L3Model* m, int rows, int N, int K) {
+  if (!linear_rows_supported(rows, K)) return false;
+  return !(rows > 4 && m->tc_ok && m->ll->cfg.norm_input && !m->ll->cfg.parallel && K >= 64 && N >= 128);
+}
+
 // does a projection of contiguous rows with a bf16 mirror run on the tensor cores (and so read the mirror alone)?
 static bool ll_takes_mirror(const L3Model* m, int rows, int N, int K) {
-  return m->tc_ok && !linear_rows_supported(rows, K) && K % 8 == 0 && K >= 64 && N >= 64;
+  return m->tc_ok && !ll_gemv(m, rows, N, K) && K % 8 == 0 && K >= 64 && N >= 64;
 }
 
 // y = x W^T (+ epilogue).  x32: fp32 rows with stride lda (0 = K); x16: bf16 mirror with stride K, or null.
 // pd: non-null when x32 is the residual stream (ll->xcur) - a deferred step is applied on the way.
-// norm_w: the row-streaming GEMV norms the rows while staging them (only where linear_rows_supported says it runs).
+// norm_w: the row-streaming GEMV norms the rows while staging them (only where ll_gemv says it runs).
 static int ll_linear(L3Model* m, const void* W, const float* x32, const void* x16, int lda, int rows, int N, int K, int epi,
                      const EpiArgs& e, LLPending* pd = nullptr, const float* norm_w = nullptr) {
   LayerList* ll = m->ll;
   LinearArgs a{};
   a.W = W; a.x = x32; a.lda = lda; a.rows = rows; a.N = N; a.K = K; a.src_mul = 1; a.src_add = 0; a.epi = epi; a.e = e;
   const int ld = lda ? lda : K;
-  if (linear_rows_supported(rows, K) && ld % 4 == 0) {
+  const bool mirror = x16 && ld == K && ll_takes_mirror(m, rows, N, K);
+  if (!mirror && linear_rows_supported(rows, K) && ld % 4 == 0) {
     // the fused form costs every CTA a pass over x, y and w per row: it wins for one or two rows (0.85 -> 0.75 ms per
     // decode step of a 12-layer width-2048 model) and loses from four rows on (8 rows: 1.87 -> 2.08 ms)
     if (pd && pd->y && rows > 2) {
@@ -1294,7 +1307,7 @@ static int ll_linear(L3Model* m, const void* W, const float* x32, const void* x1
     if (rc != L3_OK) return rc;
     a.x = ll->xcur;
   }
-  if (x16 && ld == K && ll_takes_mirror(m, rows, N, K)) {
+  if (mirror) {
     TcGemmArgs t{};
     t.kind = TC_BF16; t.A[0] = x16; t.W[0] = W;
     t.rows = rows; t.N = N; t.K = K; t.epi = epi; t.e = e; t.bn = 0;
@@ -1454,7 +1467,6 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
   if (embed_mul != 1.f && !ll->streams) LAUNCH(m, launch_scale_add_rows(m->x, embed_mul, nullptr, ntok, W, m->stream));
   StreamArgs sa{};  // the streams' side of the step: sa.y is the sublayer result they have not taken yet
   sa.x0 = m->x; sa.x_mul = embed_mul; sa.X = ll->X; sa.eps = eps; sa.S = ll->streams; sa.D = W;
-  const bool gemv = linear_rows_supported(ntok, W);  // few rows: the GEMV norms what the stream launch leaves un-normed
   // the normed input of sublayer q into hn / hn16 (or, for few rows of a streamed stack, its un-normed form: *in_norm)
   auto sublayer_in = [&](LLLayer& Ly, int q, const float* norm, const float* shift, float* hprev, int n_out, const float** in_norm) -> int {
     *in_norm = nullptr;
@@ -1464,7 +1476,7 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
     }
     StreamArgs a = sa;
     a.store = 1; a.in_w = Ly.hc_in[q];
-    if (gemv) { a.h = hn; *in_norm = norm; }
+    if (ll_gemv(m, ntok, n_out, W)) { a.h = hn; *in_norm = norm; }  // the GEMV norms what the stream launch leaves un-normed
     else { a.norm_w = norm; a.h16 = hn16; a.h = hn16 && ll_takes_mirror(m, ntok, n_out, W) ? nullptr : hn; }
     LAUNCH(m, launch_streams(a, ntok, m->stream));
     if (sa.y) sa.x0 = nullptr;  // from here on X holds the streams
@@ -1529,12 +1541,8 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
         at.q = ll->qlat; at.cache = St.lat; at.out = ll->o; at.gate = s.gate_wide ? nullptr : ll->pin + Ly.off_g; at.ld_gate = Ly.n_in;
         at.sink = s.sink ? Ly.head_vec : nullptr;
         at.pos_ptr = d_pos; at.scale = s.scale; at.B = B; at.L = L; at.H = H; at.Dk = Dk; at.Dv = s.kv_rank; at.M = m->M;
-        at.part_o = m->part_o; at.part_ml = m->part_ml;
-        at.nsplit = 1;
-        if (L == 1) {  // decode: the keys of a sequence spread over CTAs
-          const int ctas = B * ((H + 31) / 32);
-          at.nsplit = std::max(1, std::min(std::min(m->max_split, m->M / 64), (2 * 148) / std::max(1, ctas)));
-        }
+        at.part_o = ll->lat_part_o; at.part_ml = ll->lat_part_ml;
+        at.nsplit = latent_attn_splits(B, L, H, m->M);  // few rows: the keys of a sequence spread over CTAs
         LAUNCH(m, launch_latent_attn(at, m->bf16, m->stream));
         if (at.nsplit > 1) m->launch_acc += 1;
         // values out of the latent: ctx[r, h] = Wuv_h o[r, h]

@@ -117,6 +117,7 @@ struct LayerList {
   int exp_seqs = 0;
   int* h_err = nullptr;                    // pinned: a kernel sets it when one of its bounded waits ran out
   int keys_end = 0;                        // position behind the last token of the chunk being enqueued
+  float *lat_part_o = nullptr, *lat_part_ml = nullptr;  // split scratch of the latent attention
   float *moe_w = nullptr, *moe_dense = nullptr, *moe_idw = nullptr;  // [rows, top] | [rows, experts] | [rows]
   int32_t* moe_sel = nullptr;              // [rows, top]
   // parallel layers

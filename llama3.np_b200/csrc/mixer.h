@@ -158,7 +158,7 @@ struct LatentAttnArgs {
   const int* pos_ptr;    // keys [0, *pos_ptr + t] are visible to token t
   float scale;
   int B, L, H, Dk, Dv, M;
-  int nsplit;            // > 1 (L == 1 only): every split writes (o, m, l) to part_o / part_ml, the combine kernel merges
+  int nsplit;            // > 1: every split of a row's keys writes (o, m, l) to part_o / part_ml, the combine kernel merges
   float *part_o, *part_ml;
 };
 // Prompts in bf16 mode: attention over expanded keys and values on the tensor cores (attn_latent_tc.cu)
@@ -191,6 +191,8 @@ cudaError_t launch_attn_latent_tc(const LatentTcArgs& a, int n_seq, cudaStream_t
 
 size_t latent_attn_smem(int Dk);
 bool latent_attn_supported(int Dk, int Dv);
+int latent_attn_splits(int B, int L, int H, int max_keys);
+size_t latent_attn_part_rows();  // rows of split scratch (part_o: Dv floats each, part_ml: 2) that any such number of splits needs
 cudaError_t launch_latent_attn(const LatentAttnArgs& a, bool kv_bf16, cudaStream_t s);
 
 // ---- minGRU (mingru.cu): proj [rows, ld] = z | x | g logits of width n each at z_off, x_off, g_off; bias [2 n] (z, x)
