@@ -4,8 +4,8 @@
 // q~_j . [c | k_r] and the output Wuv_j (sum_i p_i c_i): attention runs on the cache rows themselves, all heads
 // of a token against the same rows, the value of a row being its first kv_rank entries.
 //
-//  * latent_prep_kernel        norms of the two latents, rotation of k_r, cache append (one CTA per token); the query latent
-//                              alone for a layer that reads another layer's cache
+//  * latent_prep_kernel        norms of the two latents, rotation of k_r, cache append (a CTA per token and latent); the
+//                              query latent alone for a layer that reads another layer's cache
 //  * head_gemm_kernel          batched per-head product (Wuk_j^T q_c and Wuv_j ctx): 64 x 64 FFMA tiles, 4 x 4 per thread;
 //                              head_gemv_kernel for up to 8 rows (decode).  The launch that folds the queries also turns
 //                              their rotated part; the one that expands the values also applies an element-wise gate
@@ -48,33 +48,33 @@ __device__ __forceinline__ void rotate_item(const float* src, T* dst, int i, int
   dst[iv] = from_f32<T>(v * cs + u * sn);
 }
 
+// blockIdx.y 0: the query latent of a token; 1: its cache row
 template <typename KVT>
 __global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrepArgs a) {
   __shared__ float red[32];
   pdl_launch();
   pdl_wait();
   const int r = blockIdx.x;
-  const int b = r / a.L, t = r - b * a.L;
-  const int pos = *a.pos_ptr + t;
-  const float* row = a.proj + (size_t)r * a.ld;
+  const bool query = blockIdx.y == 0;
+  const int n = query ? a.q_rank : a.kv_rank;
+  const float* row = a.proj + (size_t)r * a.ld + (query ? 0 : a.k_off);
+  const float* w = query ? a.wq : a.wk;
   float ss = 0.f;
-  for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) { const float v = row[i]; ss = fmaf(v, v, ss); }
-  const float rq = 1.0f / sqrtf(block_sum(ss, red) / (float)a.q_rank + a.eps);
-  for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) {
-    const float v = row[i] * rq * a.wq[i];
-    a.cq[(size_t)r * a.q_rank + i] = v;
-    if (a.cq16) a.cq16[(size_t)r * a.q_rank + i] = __float2bfloat16_rn(v);
+  for (int i = threadIdx.x; i < n; i += blockDim.x) { const float v = row[i]; ss = fmaf(v, v, ss); }
+  const float rinv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + a.eps);
+  if (query) {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+      const float v = row[i] * rinv * w[i];
+      if (a.cq) a.cq[(size_t)r * n + i] = v;
+      if (a.cq16) a.cq16[(size_t)r * n + i] = __float2bfloat16_rn(v);
+    }
+    return;
   }
-  if (a.k_off < 0) return;
-  const float* kv = row + a.k_off;
-  ss = 0.f;
-  for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) { const float v = kv[i]; ss = fmaf(v, v, ss); }
-  const float rk = 1.0f / sqrtf(block_sum(ss, red) / (float)a.kv_rank + a.eps);
+  const int b = r / a.L, pos = *a.pos_ptr + r - b * a.L;
   KVT* dst = (KVT*)a.cache + ((size_t)b * a.M + pos) * (a.kv_rank + a.rot_dim);
-  for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) dst[i] = from_f32<KVT>(kv[i] * rk * a.wk[i]);
-  const float* kr = kv + a.kv_rank;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = from_f32<KVT>(row[i] * rinv * w[i]);
   for (int i = threadIdx.x; i < a.rot_dim - a.rot_dims / 2; i += blockDim.x)
-    rotate_item(kr, dst + a.kv_rank, i, a.rot_dims, a.rot_layout, pos, a.inv_freq);
+    rotate_item(row + n, dst + n, i, a.rot_dims, a.rot_layout, pos, a.inv_freq);
 }
 
 // ---------------------------------------------------------------- batched per-head product
@@ -400,18 +400,22 @@ __global__ void __launch_bounds__(128) attn_latent_combine_kernel(LatentAttnArgs
   const size_t tok = row / a.H;
   const float* po = a.part_o + row * a.nsplit * a.Dv + d;
   float o = 0.f;
-#pragma unroll 8
+#pragma unroll 16
   for (int s = 0; s < a.nsplit; ++s) {
     const float w = wsplit[s];
-    if (w != 0.f) o = fmaf(w, po[(size_t)s * a.Dv], o);
+    const float v = w != 0.f ? __ldg(po + (size_t)s * a.Dv) : 0.f;  // a split without keys left nothing here
+    o = fmaf(w, v, o);
   }
   a.out[row * a.Dv + d] = o * latent_out_scale(a, tok, (int)(row - tok * a.H), mx, l);
 }
 
 // Few rows (decode): the per-head product as matrix-vector products that stream the head's weights once.
-// w_ks == 1 (an output's weights are contiguous): a warp per output; w_js == 1: a thread per output, the k loop unrolled.
+// w_ks == 1 (an output's weights are contiguous): a warp per output; w_js == 1: a CTA per 64 outputs, two to a lane, its
+// warps each taking an eighth of the k range.
+constexpr int HV_OUT = 64;
 template <typename WT>
 __global__ void __launch_bounds__(256) head_gemv_kernel(HeadGemmArgs a) {
+  __shared__ float part[8][HV_OUT];
   pdl_launch();
   pdl_wait();
   const int h = blockIdx.y, r = blockIdx.z, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -430,12 +434,26 @@ __global__ void __launch_bounds__(256) head_gemv_kernel(HeadGemmArgs a) {
     v = warp_sum(acc);
     if (lane != 0) return;
   } else {
-    j = blockIdx.x * 256 + threadIdx.x;
+    const int per = (a.K + 7) / 8, k0 = warp * per, k1 = min(a.K, k0 + per);
+    const int j0 = blockIdx.x * HV_OUT + lane, j1 = j0 + 32;
+    const int c0 = min(j0, a.J - 1), c1 = min(j1, a.J - 1);  // lanes past the last output repeat it
+    float acc0 = 0.f, acc1 = 0.f;
+#pragma unroll 16
+    for (int k = k0; k < k1; ++k) {
+      const WT* wk = W + (size_t)k * a.w_ks;
+      const float x = A[k];
+      acc0 = fmaf(to_f32(wk[c0]), x, acc0);
+      acc1 = fmaf(to_f32(wk[c1]), x, acc1);
+    }
+    part[warp][lane] = acc0;
+    part[warp][lane + 32] = acc1;
+    __syncthreads();
+    if (threadIdx.x >= HV_OUT) return;
+    j = blockIdx.x * HV_OUT + threadIdx.x;
     if (j >= a.J) return;
-    float acc = 0.f;
-#pragma unroll 8
-    for (int k = 0; k < a.K; ++k) acc = fmaf(to_f32(W[(size_t)k * a.w_ks + j]), A[k], acc);
-    v = acc;
+    v = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) v += part[w][threadIdx.x];
   }
   const size_t o = (size_t)r * a.ldc + (size_t)h * a.c_hs + j;
   v *= head_gate(a, r, h, j);
@@ -504,13 +522,14 @@ cudaError_t launch_latent_attn(const LatentAttnArgs& a, bool kv_bf16, cudaStream
 }
 
 cudaError_t launch_latent_prep(const LatentPrepArgs& a, int rows, bool kv_bf16, cudaStream_t s) {
-  if (kv_bf16) return launch_k(latent_prep_kernel<bf16>, dim3(rows), dim3(256), 0, s, a);
-  return launch_k(latent_prep_kernel<float>, dim3(rows), dim3(256), 0, s, a);
+  const dim3 grid(rows, a.k_off < 0 ? 1 : 2);
+  if (kv_bf16) return launch_k(latent_prep_kernel<bf16>, grid, dim3(256), 0, s, a);
+  return launch_k(latent_prep_kernel<float>, grid, dim3(256), 0, s, a);
 }
 
 cudaError_t launch_head_gemm(const HeadGemmArgs& a, bool w_bf16, cudaStream_t s) {
   if (a.rows <= 8) {
-    const dim3 g(a.w_ks == 1 ? (a.J + 7) / 8 : (a.J + 255) / 256, a.H, a.rows);
+    const dim3 g(a.w_ks == 1 ? (a.J + 7) / 8 : (a.J + HV_OUT - 1) / HV_OUT, a.H, a.rows);
     if (w_bf16) return launch_k(head_gemv_kernel<bf16>, g, dim3(256), 0, s, a);
     return launch_k(head_gemv_kernel<float>, g, dim3(256), 0, s, a);
   }

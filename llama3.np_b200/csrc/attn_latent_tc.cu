@@ -149,17 +149,20 @@ __global__ void __launch_bounds__(256) latent_q_pack_kernel(LatentQPackArgs a) {
   for (int g = threadIdx.x; g < n8; g += blockDim.x) {
     const int h = g * 8 / DQ, d0 = g * 8 - h * DQ;
     const float* qh = src + (size_t)h * hd;
-    float v[8];
-    if (d0 < dpad) {
-#pragma unroll
-      for (int k = 0; k < 8; ++k) v[k] = d0 + k < a.dim ? qh[d0 + k] : 0.f;
-    } else {
-      const float* qr = qh + a.dim;
+    __align__(16) float v[8];
+    const int i0 = d0 - dpad;  // sizes are multiples of 8: a group of 8 lies wholly inside a part or wholly in its padding
+    if (d0 < dpad ? d0 >= a.dim : i0 >= a.rot_dim) {
+      *reinterpret_cast<uint4*>(dst + (size_t)g * 8) = make_uint4(0, 0, 0, 0);
+      continue;
+    }
+    const float* qr = qh + a.dim;
+    const float* s8 = d0 < dpad ? qh + d0 : qr + i0;
+    *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(s8);
+    *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(s8 + 4);
+    if (d0 >= dpad) {
 #pragma unroll
       for (int k = 0; k < 8; ++k) {
-        const int i = d0 - dpad + k;
-        if (i >= a.rot_dim) { v[k] = 0.f; continue; }
-        v[k] = qr[i];
+        const int i = i0 + k;
         if (i >= a.rot_dims) continue;
         const int p = a.rot_layout ? (i < half ? i : i - half) : i >> 1;           // pair
         const bool second = a.rot_layout ? i >= half : i & 1;

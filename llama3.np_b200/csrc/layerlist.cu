@@ -1521,7 +1521,7 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
       const int Dk = s.kv_rank + s.rot_dim, nq = H * (DK + s.rot_dim);
       LatentPrepArgs pa{};
       pa.proj = ll->pin; pa.ld = Ly.n_in; pa.k_off = s.kv_source ? -1 : Ly.off_k; pa.wq = Ly.q_norm; pa.wk = Ly.k_norm; pa.eps = eps;
-      pa.cq = ll->aux; pa.cq16 = (bf16*)ll->aux16; pa.cache = St.lat; pa.inv_freq = Ly.inv_freq; pa.pos_ptr = d_pos;
+      pa.cq = ll->aux16 && ll_takes_mirror(m, ntok, nq, s.q_rank) ? nullptr : ll->aux; pa.cq16 = (bf16*)ll->aux16; pa.cache = St.lat; pa.inv_freq = Ly.inv_freq; pa.pos_ptr = d_pos;
       pa.L = L; pa.M = m->M; pa.q_rank = s.q_rank; pa.kv_rank = s.kv_rank; pa.rot_dim = s.rot_dim; pa.rot_dims = s.rot_dims;
       pa.rot_layout = s.rot_layout;
       LAUNCH(m, launch_latent_prep(pa, ntok, m->bf16, m->stream));

@@ -126,7 +126,7 @@ struct LatentPrepArgs {
   int ld, k_off;         // k_off < 0: the queries only (the layer reads another layer's cache)
   const float *wq, *wk;  // norm weights [q_rank], [kv_rank]
   float eps;
-  float* cq;             // [rows, q_rank] normed query latent (+ bf16 mirror, may be null)
+  float* cq;             // [rows, q_rank] normed query latent, and its bf16 mirror (either may be null)
   bf16* cq16;
   void* cache;           // [maxB, M, kv_rank + rot_dim] of KVT
   const float* inv_freq; // [rot_dims / 2]

@@ -11,7 +11,7 @@ per-sequence state of one layer (the states of all layers are at hand for layers
     sublayer q:  u = a_q . X;  y = ls_q * F_q(n_q * u / rms(u));  X_t <- sum_s M_q[s, t] X_s + b_q[t] y
     logits = s_l * E (n_f * x / rms(x)),  x = sum_t X_t
 with a_q, b_q [s] and M_q [s, s] (indexed [from, to]) the layer's stream weights, F_1 the mixer and F_2
-the feed-forward.
+the feed-forward.  A configuration without streams has one row and plain sums.
 """
 from __future__ import annotations
 
@@ -51,11 +51,13 @@ def sink_softmax(z, sink):
 # ------------------------------------------------------------------ residual streams
 def streams_in(X, P, q):
     """What sublayer q reads, ahead of its norm: a weighted sum of the streams."""
-    return P[f"hc{q}.in"] @ X
+    return P[f"hc{q}.in"] @ X if f"hc{q}.in" in P else X[0]
 
 
 def streams_out(X, y, P, q):
     """All streams at once from the old ones: new_t = sum_s mix[s, t] X_s + out[t] y."""
+    if f"hc{q}.mix" not in P:
+        return X + y[None]
     return P[f"hc{q}.mix"].T @ X + np.outer(P[f"hc{q}.out"], y)
 
 
@@ -126,7 +128,7 @@ class OracleGifudra:
         """One token -> logits (and the sum of the streams after every layer)."""
         cfg, T, eps = self.cfg, self.T, self.eps
         x = T["embed"][int(token)] * float(cfg["embedding"]["scale"])
-        X = np.tile(x, (int(cfg["streams"]), 1))
+        X = np.tile(x, (int(cfg.get("streams") or 1), 1))
         trace = []
         for lc, P, st in zip(cfg["layers"], self.per_layer, self.state):
             mc = lc["mixer"]
@@ -164,7 +166,7 @@ def to_bf16_grid(tensors):
 def random_model(config, seed, bf16_round=True):
     """Random tensors for a configuration (names and shapes as a checkpoint has them)."""
     rng = np.random.default_rng(seed)
-    W, V, S = config["width"], config["vocab"], config["streams"]
+    W, V, S = config["width"], config["vocab"], config.get("streams") or 0
 
     def mat(o, i, gain=1.0):
         return rng.standard_normal((o, i)) * gain / np.sqrt(i)
@@ -180,20 +182,22 @@ def random_model(config, seed, bf16_round=True):
         t[p + "norm1"] = vec(W, 1.0, 0.1)
         t[p + "mix.dq"] = mat(mc["q_rank"], W)
         t[p + "mix.dq.norm"] = vec(mc["q_rank"], 1.0, 0.1)
-        t[p + "mix.uq"] = mat(H * (dn + dr), mc["q_rank"], 2.0)
+        t[p + "mix.uq"] = mat(H * (dn + dr), mc["q_rank"], 1.2)
         if mc.get("kv_from") is None:
-            t[p + "mix.dkv"] = mat(mc["kv_rank"] + dr, W, 2.0)
+            t[p + "mix.dkv"] = mat(mc["kv_rank"] + dr, W, 1.2)
             t[p + "mix.dkv.norm"] = vec(mc["kv_rank"], 1.0, 0.1)
-        t[p + "mix.uk"] = mat(H * dn, mc["kv_rank"], 2.0)
+        t[p + "mix.uk"] = mat(H * dn, mc["kv_rank"], 1.2)
         t[p + "mix.uv"] = mat(H * dv, mc["kv_rank"])
         t[p + "mix.sink"] = vec(H, 0.5, 1.0)
         t[p + "mix.g"] = mat(H * dv, W)
         t[p + "mix.o"] = mat(W, H * dv)
         for q in (1, 2) if has_ff else (1,):
             t[p + f"ls{q}"] = vec(W, 0.7, 0.2)
-            t[p + f"hc{q}.in"] = vec(S, 1.0 / S, 0.3)
+            if not S:
+                continue
+            t[p + f"hc{q}.in"] = vec(S, 1.0 / S, 0.3 / S)
             t[p + f"hc{q}.out"] = vec(S, 1.0, 0.4)
-            t[p + f"hc{q}.mix"] = np.eye(S) * 0.8 + 0.15 * rng.standard_normal((S, S))
+            t[p + f"hc{q}.mix"] = np.eye(S) * 0.8 + (0.3 / S) * rng.standard_normal((S, S))
         if has_ff:
             ff = lc["mlp"]["ff"]
             t[p + "norm2"] = vec(W, 1.0, 0.1)
