@@ -28,6 +28,9 @@ def __getattr__(name):  # lazy: importing the package must not require the built
     if name == "Debuzen":
         from .debuzen import Debuzen
         return Debuzen
+    if name == "Gifudra":
+        from .gifudra import Gifudra
+        return Gifudra
     if name in ("StackDecoder", "StackConfig", "LayerSpec"):
         from . import stack as _s
         return getattr(_s, name)
