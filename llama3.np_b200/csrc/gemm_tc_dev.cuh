@@ -512,7 +512,36 @@ __device__ __forceinline__ void tc_gemm_run(TcPipe& p, const CUtensorMap* tmA0p,
               if (e.out_bf16) e.out_bf16[o] = __float2bfloat16_rn(hv);
             }
           }
-        } else {  // EPI_STORE
+        } else if (!e.out_lo && !(e.ld_out & 1) && !(N & 1)) {
+          // EPI_STORE, whole column pairs: groups of 16 rows are read from Cs before the first of their stores, row
+          // pointers advance by the leading dimension, and what does not depend on the row is decided once per chunk
+          const int mb = m0 + quarter * 32;
+          const int live = min(32, rows - mb);
+          if (col_ok) {
+            float* po = e.out ? e.out + (size_t)mb * e.ld_out + col : nullptr;
+            bf16* pb = e.out_bf16 ? e.out_bf16 + (size_t)mb * e.ld_out + col : nullptr;
+#pragma unroll
+            for (int rb = 0; rb < 32; rb += 16) {
+              float2 tt[16];
+#pragma unroll
+              for (int i = 0; i < 16; ++i) tt[i] = *reinterpret_cast<const float2*>(Cs + (rb + i) * LDC + cp);
+              if (e.unary) {
+#pragma unroll
+                for (int i = 0; i < 16; ++i) { tt[i].x = unary_act(e.unary, tt[i].x); tt[i].y = unary_act(e.unary, tt[i].y); }
+              }
+              if (po) {
+#pragma unroll
+                for (int i = 0; i < 16; ++i, po += e.ld_out)
+                  if (rb + i < live) *reinterpret_cast<float2*>(po) = tt[i];
+              }
+              if (pb) {
+#pragma unroll
+                for (int i = 0; i < 16; ++i, pb += e.ld_out)
+                  if (rb + i < live) *reinterpret_cast<__nv_bfloat162*>(pb) = __floats2bfloat162_rn(tt[i].x, tt[i].y);
+              }
+            }
+          }
+        } else {  // EPI_STORE, any strides
 #pragma unroll 1
           for (int rb = 0; rb < 32; rb += 4) {
             if (m0 + quarter * 32 + rb >= rows) break;
