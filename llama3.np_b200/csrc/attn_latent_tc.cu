@@ -9,7 +9,9 @@
 //  * attn_latent_tc_kernel   one CTA = 128 queries of one (sequence, head), keys in blocks of 64:
 //      warp 0     TMA: the query tile, then the key blocks - the head's slice of the expansion, and the rotated part straight
 //                 from the cache rows (shared by all heads)
-//      warp 1     MMA issuer: S_j = Q K_j^T into one of two TMEM score buffers; O_w += P_j V_j, V as an MN-major operand
+//      warp 1     issues S_j = Q K_j^T into one of two TMEM score buffers
+//      warp 11    issues O_w += P_j V_j, V as an MN-major operand (a thread of its own: the waits and the operand descriptors of
+//                 the two products would otherwise queue behind one another in one instruction stream)
 //      warps 2-9  two groups of four softmax warps taking alternate key blocks (w = j & 1), each with its own running
 //                 maximum, sum and TMEM output; a thread is a query row.  The weights leave as TWO bf16 tiles, p = hi + lo
 //                 (16 significant bits), and O takes both: scores, weights and sums are fp32 in effect.  The outputs are
@@ -31,7 +33,7 @@ constexpr int BQ = 128, BKV = 64;
 constexpr int SLICE_Q = BQ * 128, SLICE_K = BKV * 128;   // bytes of one 64-entry slice of a query tile / key or value block
 constexpr int P_TILE = BQ * BKV * 2;                     // one bf16 weight tile; a group owns two (hi, lo)
 constexpr int STAGES_MAX = 3;
-constexpr int THREADS = 352;
+constexpr int THREADS = 384;
 constexpr int TMEM_COLS = 512;                           // 2 score buffers of 64 columns, 2 outputs of up to 192
 constexpr int TAIL = 512 + 2 * BQ * 8;                   // barriers, TMEM slot, flag; (maximum, sum) of both groups' rows
 constexpr float LOG2E = 1.4426950408889634f;
@@ -271,46 +273,54 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       }
     }
   } else if (warp == 1) {
-    if (lane == 0) {  // ---------------- MMA issuer
-      const uint32_t idesc_pv = IDESC_PV | ((uint32_t)(((a.vdim + 15) & ~15) >> 3) << 17);
+    if (lane == 0) {  // ---------------- scores
+      uint32_t steps = 0;  // 16-entry steps of every slice, four bits each
+      for (int s = 0; s < sh.nqs; ++s) {
+        const int n = s < sh.nks ? a.dim - s * 64 : a.rot_dim - (s - sh.nks) * 64;
+        steps |= (uint32_t)((min(n, 64) + 15) >> 4) << (4 * s);
+      }
+      const uint64_t dq = desc_k_sw128(sQ), dk0 = desc_k_sw128(sK);
       bool ok = mbar_wait(q_full, 0, fail);
-      auto issue_pv = [&](int j) {  // O_w += P_j V_j, high part then low part
-        const int st = j % STAGES, w = j & 1;
-        if (!mbar_wait(v_full + 8 * st, (j / STAGES) & 1, fail) || !mbar_wait(p_full + 8 * w, (j >> 1) & 1, fail)) return false;
-        tc_fence_after();
-        const uint32_t vb = sV + st * sh.v_bytes();
-        for (int part = 0; part < 2; ++part) {
-          const uint32_t pb = sP + (2 * w + part) * P_TILE;
-#pragma unroll
-          for (int kk = 0; kk < BKV / 16; ++kk)  // 16 keys per MMA
-            mma_bf16(tO + w * o_cols, desc_k_sw128(pb) + (uint64_t)(kk * 2), desc_mn_sw128(vb + kk * 2048, SLICE_K), idesc_pv,
-                     (j < 2 && part == 0 && kk == 0) ? 0u : 1u);
-        }
-        tc_commit(v_empty + 8 * st);
-        tc_commit(p_empty + 8 * w);
-        return true;
-      };
+      int st = 0, ph = 0;
       for (int j = 0; j < nb && ok; ++j) {
-        const int st = j % STAGES, w = j & 1;
-        ok = mbar_wait(k_full + 8 * st, (j / STAGES) & 1, fail) && (j < 2 || mbar_wait(s_empty + 8 * w, ((j >> 1) - 1) & 1, fail));
+        const int w = j & 1;
+        ok = mbar_wait(k_full + 8 * st, ph, fail) && (j < 2 || mbar_wait(s_empty + 8 * w, ((j >> 1) - 1) & 1, fail));
         if (!ok) break;
         tc_fence_after();
-        const uint32_t kb = sK + st * sh.k_bytes();
-        uint32_t acc = 0u;
+        const uint64_t dk = dk0 + (uint64_t)((st * sh.k_bytes()) >> 4);
+        const uint32_t td = tS + w * BKV;
         for (int s = 0; s < sh.nqs; ++s) {
-          const int n = s < sh.nks ? a.dim - s * 64 : a.rot_dim - (s - sh.nks) * 64;  // entries of this slice
-          const int nk = (min(n, 64) + 15) >> 4;
-          for (int kk = 0; kk < nk; ++kk) {
-            mma_bf16(tS + w * BKV, desc_k_sw128(sQ + s * SLICE_Q) + (uint64_t)(kk * 2), desc_k_sw128(kb + s * SLICE_K) + (uint64_t)(kk * 2), IDESC_S, acc);
-            acc = 1u;
-          }
+          const uint64_t ad = dq + (uint64_t)(s * (SLICE_Q >> 4)), bd = dk + (uint64_t)(s * (SLICE_K >> 4));
+          const int n = (steps >> (4 * s)) & 15;
+#pragma unroll
+          for (int kk = 0; kk < 4; ++kk)
+            if (kk < n) mma_bf16(td, ad + kk * 2, bd + kk * 2, IDESC_S, (s | kk) ? 1u : 0u);
         }
         tc_commit(k_empty + 8 * st);
         tc_commit(s_full + 8 * w);
-        if (j >= 2) ok = issue_pv(j - 2);
+        if (++st == STAGES) { st = 0; ph ^= 1; }
       }
-      if (ok && nb >= 2) ok = issue_pv(nb - 2);
-      if (ok) issue_pv(nb - 1);
+    }
+  } else if (warp == 11) {
+    if (lane == 0) {  // ---------------- outputs
+      const uint32_t idesc_pv = IDESC_PV | ((uint32_t)(((a.vdim + 15) & ~15) >> 3) << 17);
+      const uint64_t dp0 = desc_k_sw128(sP), dv0 = desc_mn_sw128(sV, SLICE_K);
+      int st = 0, ph = 0;
+      for (int j = 0; j < nb; ++j) {
+        const int w = j & 1;
+        if (!mbar_wait(v_full + 8 * st, ph, fail) || !mbar_wait(p_full + 8 * w, (j >> 1) & 1, fail)) break;
+        tc_fence_after();
+        const uint64_t dv = dv0 + (uint64_t)((st * sh.v_bytes()) >> 4), dp = dp0 + (uint64_t)(w * (2 * P_TILE >> 4));
+        const uint32_t td = tO + w * o_cols;
+#pragma unroll
+        for (int part = 0; part < 2; ++part)  // high part, then low part
+#pragma unroll
+          for (int kk = 0; kk < BKV / 16; ++kk)  // 16 keys per MMA
+            mma_bf16(td, dp + part * (P_TILE >> 4) + kk * 2, dv + kk * (2048 >> 4), idesc_pv, (part | kk) ? 1u : (j < 2 ? 0u : 1u));
+        tc_commit(v_empty + 8 * st);
+        tc_commit(p_empty + 8 * w);
+        if (++st == STAGES) { st = 0; ph ^= 1; }
+      }
     }
   } else {  // ---------------- softmax and output: thread = query row
     const int w = (warp - 2) >> 2, quarter = warp & 3;       // group; TMEM lanes this warp may read
