@@ -178,17 +178,20 @@ __global__ void __launch_bounds__(256) latent_q_pack_kernel(LatentQPackArgs a) {
 
 // ---------------------------------------------------------------- attention
 struct Shape {
-  int nks, nrs, nqs, nvs, stages;  // 64-entry slices of the un-rotated keys, the rotated part, both, the values; ring depth
+  int nks, nrs, nqs, nvs;  // 64-entry slices of the un-rotated keys, the rotated part, both, the values
+  int kst, vst;            // depths of the key and value rings
   __host__ __device__ int q_bytes() const { return nqs * SLICE_Q; }
   __host__ __device__ int k_bytes() const { return nqs * SLICE_K; }
   __host__ __device__ int v_bytes() const { return nvs * SLICE_K; }
-  __host__ __device__ int smem() const { return 1024 + q_bytes() + stages * (k_bytes() + v_bytes()) + 4 * P_TILE + TAIL; }
+  __host__ __device__ int smem() const { return 1024 + q_bytes() + kst * k_bytes() + vst * v_bytes() + 4 * P_TILE + TAIL; }
 };
 
 __host__ __device__ inline Shape make_shape(int dim, int rot_dim, int vdim) {
   Shape s;
   s.nks = (dim + 63) / 64; s.nrs = (rot_dim + 63) / 64; s.nqs = s.nks + s.nrs; s.nvs = (vdim + 63) / 64;
-  for (s.stages = STAGES_MAX; s.stages > 1 && s.smem() > 227 * 1024; --s.stages) {}
+  // a key block is refilled from L2 while the other ones of the ring are used: the keys, needed first, get the spare stage
+  s.kst = s.vst = STAGES_MAX;
+  while (s.smem() > 227 * 1024 && s.kst + s.vst > 2) { if (s.vst >= s.kst) --s.vst; else --s.kst; }
   return s;
 }
 
@@ -197,10 +200,9 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
                       const __grid_constant__ CUtensorMap tmC, LatentTcArgs a) {
   extern __shared__ uint8_t smem_raw[];
   const Shape sh = make_shape(a.dim, a.rot_dim, a.vdim);
-  const int STAGES = sh.stages;
   const uint32_t raw = smem_u32(smem_raw);
   const uint32_t sQ = (raw + 1023u) & ~1023u;
-  const uint32_t sK = sQ + sh.q_bytes(), sV = sK + STAGES * sh.k_bytes(), sP = sV + STAGES * sh.v_bytes();
+  const uint32_t sK = sQ + sh.q_bytes(), sV = sK + sh.kst * sh.k_bytes(), sP = sV + sh.vst * sh.v_bytes();
   const uint32_t bars = sP + 4 * P_TILE;
   const uint32_t q_full = bars, k_full = bars + 8, k_empty = k_full + 8 * STAGES_MAX, v_full = k_empty + 8 * STAGES_MAX,
                  v_empty = v_full + 8 * STAGES_MAX, s_full = v_empty + 8 * STAGES_MAX, s_empty = s_full + 16,
@@ -222,7 +224,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     asm volatile("prefetch.tensormap [%0];" ::"l"(&tmC));
     *fail = 0;
     mbar_init(q_full, 1);
-    for (int s = 0; s < STAGES; ++s) {
+    for (int s = 0; s < STAGES_MAX; ++s) {
       mbar_init(k_full + 8 * s, 1); mbar_init(k_empty + 8 * s, 1);
       mbar_init(v_full + 8 * s, 1); mbar_init(v_empty + 8 * s, 1);
     }
@@ -254,7 +256,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       mbar_expect_tx(q_full, sh.q_bytes());
       for (int s = 0; s < sh.nqs; ++s) tma_load_2d(sQ + s * SLICE_Q, &tmQ, head * DQ + s * 64, b * a.L + q0, q_full);
       for (int j = 0; j < nb; ++j) {
-        const int st = j % STAGES, use = j / STAGES;
+        const int st = j % sh.kst, use = j / sh.kst;
         if (use > 0 && !mbar_wait(k_empty + 8 * st, (use - 1) & 1, fail)) break;
         const uint32_t kb = sK + st * sh.k_bytes(), bar = k_full + 8 * st;
         mbar_expect_tx(bar, sh.k_bytes());
@@ -265,7 +267,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   } else if (warp == 10) {
     if (lane == 0) {  // ---------------- values
       for (int j = 0; j < nb; ++j) {
-        const int st = j % STAGES, use = j / STAGES;
+        const int st = j % sh.vst, use = j / sh.vst;
         if (use > 0 && !mbar_wait(v_empty + 8 * st, (use - 1) & 1, fail)) break;
         mbar_expect_tx(v_full + 8 * st, sh.v_bytes());
         for (int s = 0; s < sh.nvs; ++s)
@@ -298,7 +300,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         }
         tc_commit(k_empty + 8 * st);
         tc_commit(s_full + 8 * w);
-        if (++st == STAGES) { st = 0; ph ^= 1; }
+        if (++st == sh.kst) { st = 0; ph ^= 1; }
       }
     }
   } else if (warp == 11) {
@@ -319,7 +321,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
             mma_bf16(td, dp + part * (P_TILE >> 4) + kk * 2, dv + kk * (2048 >> 4), idesc_pv, (part | kk) ? 1u : (j < 2 ? 0u : 1u));
         tc_commit(v_empty + 8 * st);
         tc_commit(p_empty + 8 * w);
-        if (++st == STAGES) { st = 0; ph ^= 1; }
+        if (++st == sh.vst) { st = 0; ph ^= 1; }
       }
     }
   } else {  // ---------------- softmax and output: thread = query row
