@@ -31,6 +31,9 @@ def stack_config(config: Mapping, *, max_seq_len: int = 256, max_batch_size: int
         if lc["type"] != "latent_attention":
             raise ValueError(f"layer {i}: unknown mixer type {lc['type']!r}")
         mc = lc["mixer"]
+        if mc.get("kv_from") is not None:  # what a shared cache fixes comes from its owner where the layer does not repeat it
+            owner = config["layers"][int(mc["kv_from"])]["mixer"]
+            mc = {**{k: owner[k] for k in ("kv_rank", "rot_dim", "rot") if k in owner}, **mc}
         rot, rot_dim = mc.get("rot") or {}, int(mc.get("rot_dim", 0))
         kv_from = mc.get("kv_from")
         spec = LayerSpec(mixer=LATENT, heads=int(mc["heads"]), dim=int(mc["dim"]), vdim=int(mc["vdim"]),
@@ -64,7 +67,9 @@ class Gifudra(StackDecoder):
         super().__init__(stack_config(config, max_seq_len=max_seq_len, max_batch_size=max_batch_size, dtype=dtype),
                          device=device, flags=flags)
         if tensors is not None:
-            self.load_tensors(tensors)
+            # a layer without a feed-forward reads none of these, whether or not the checkpoint holds them
+            unused = tuple(f"l{i}.{n}" for i, lc in enumerate(config["layers"]) if lc.get("mlp") is None for n in ("norm2", "ls2", "hc2."))
+            self.load_tensors({k: v for k, v in tensors.items() if not k.startswith(unused)} if unused else tensors)
         else:
             self.fill_random(random_seed)
 

@@ -38,6 +38,11 @@ def test_config_reader_takes_every_size_from_the_config():
     assert (a.scale, a.rot_base, a.rot_layout, a.sink, a.gate_wide, a.kv_from) == (0.25, 777.0, 1, True, True, None)
     assert (a.ff, a.ff_kind, a.experts) == (28, FF_RELU2, 0)
     assert (b.heads, b.dim, b.vdim, b.q_rank, b.scale, b.kv_from, b.ff) == (2, 5, 7, 9, 0.5, 0, 0)
+    brief = json.loads(json.dumps(CFG))
+    for k in ("kv_rank", "rot_dim", "rot"):
+        del brief["layers"][1]["mixer"][k]
+    b = stack_config(brief).layers[1]
+    assert (b.kv_rank, b.rot_dim, b.rot_dims, b.rot_base, b.dim) == (20, 4, 4, 777.0, 5)
     plain = json.loads(json.dumps(CFG))
     del plain["streams"], plain["embedding"], plain["logit_scale"]
     sc = stack_config(plain)

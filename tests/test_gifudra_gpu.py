@@ -420,9 +420,11 @@ def test_missing_and_unknown_tensors_are_errors():
     for drop in ("l0.hc2.mix", "l1.mix.sink", "l0.ls2", "l0.mix.dkv"):
         with pytest.raises(RuntimeError):
             Gifudra(cfg, {k: v for k, v in t.items() if k != drop})
-    for name, like in (("head", "embed"), ("l1.mix.dkv", "l0.mix.dkv"), ("l1.norm2", "l0.norm2"), ("l0.mlp.gate", "l0.mlp.up")):
+    for name, like in (("head", "embed"), ("l1.mix.dkv", "l0.mix.dkv"), ("l1.mlp.up", "l0.mlp.up"), ("l0.mlp.gate", "l0.mlp.up")):
         with pytest.raises(ValueError):
             Gifudra(cfg, {**t, name: t[like]})
+    # the feed-forward's norm, scale and stream weights of a layer that has none are ignored
+    Gifudra(cfg, {**t, **{"l1." + n: t["l0." + n] for n in ("norm2", "ls2", "hc2.in", "hc2.out", "hc2.mix")}}).close()
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
