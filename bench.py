@@ -328,7 +328,7 @@ def shape_record(name, shape, dtype, B, L, n_decode, device=0, ids=None, iters=2
 
 def cpu_shape_baseline(shape, B, L, n_decode_sample):
     """The oracle port at the SAME widths with 1 and 2 layers (+ LM head), timed on the host cores: per-layer and
-    head costs follow from the two runs; the full-depth figure is their linear extrapolation (BASELINE.md 5: the
+    head costs follow from the two runs; the full-depth figure is their linear extrapolation (the
     reference re-casts every fp32 weight to fp64 per call - a full-depth 8B-shaped run needs 30 GB and minutes)."""
     from dataclasses import replace
     import llama3_np_b200  # noqa: F401
@@ -549,7 +549,7 @@ def run_b200(a):
         step_ms = dev_ms / a.steps / N_OUT  # one decode step of the whole batch (the prefill is 1 of 248 steps)
         # Dominant kernel of a decode step: decode_stack_kernel (every layer of the step, one launch), ~88 % of the
         # step's device time (profiles/r02_launches_decode_step.csv); the LM head + finalize are the rest.
-        # Its algorithmic bytes per launch (DESIGN.md 4.0): the layers' weights once (each of the ceil(B / 12) clusters
+        # Its algorithmic bytes per launch: the layers' weights once (each of the ceil(B / 12) clusters
         # streams them, but from L2) + K and V of every cached position of every sequence and layer.
         stack_ms, lm_ms = C.c_float(), C.c_float()
         _cabi.check(lib.l3_bench_kernel(h, 4, B, pos_mid, 30, C.byref(stack_ms)), h)
@@ -573,7 +573,7 @@ def run_b200(a):
                     "traffic_note": traffic_note, "peak_source": how, "algorithmic_work_per_launch": stack_bytes,
                     "launch_ms": stack_ms.value, "at": f"B={B}, position {pos_mid}",
                     "note": "timed alone with CUDA events on the library stream, L2 flushed between launches; the kernel is bound by "
-                            "FFMA issue + cluster exchanges, not by HBM (DESIGN.md 4.0): the fraction says how far the step is from "
+                            "FFMA issue + cluster exchanges, not by HBM: the fraction says how far the step is from "
                             "the data-movement floor",
                     "per_decode_step_ms": {"decode_stack_kernel": stack_ms.value, "lm_head (gemm_tc_kernel, 256-wide tiles, fused argmax)": lm_ms.value},
                     "decode_step_ms_measured": step_ms,

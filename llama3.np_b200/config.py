@@ -1,6 +1,6 @@
 """Model hyper-parameters: the config surface of the reference, kept field for field.
 
-Mirrors `/root/reference/config.py:5-19` (`ModelArgs`): same field names, order and
+Mirrors `config.py:5-19` (`ModelArgs`): same field names, order and
 defaults, so code written against the reference (`ModelArgs(); args.dim = ...`) runs
 unchanged.  As in the reference there is no `hidden_dim` field: the FFN width is
 inferred from the `up_proj` weight shape at load time.
@@ -29,7 +29,7 @@ class ModelArgs:
     dtype: str = "float32"
 
 
-# Named shapes of BASELINE.json's configs (SURVEY.md §8 legend).  `hidden_dim` is not a
+# Named shapes of BASELINE.json's configs.  `hidden_dim` is not a
 # ModelArgs field (see above); it is returned beside the args.
 def named_config(name: str, **overrides):
     table = {

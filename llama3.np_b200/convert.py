@@ -1,5 +1,5 @@
-"""Weight ingestion (SURVEY.md 8(f)-3): Hugging Face `safetensors` Llama checkpoints -> the reference's
-`.npz` key layout (`/root/reference/llama3.py:219-235, 269, 280-281`: HF-style names, float32, `[out, in]`).
+"""Weight ingestion: Hugging Face `safetensors` Llama checkpoints -> the reference's
+`.npz` key layout (`llama3.py:219-235, 269, 280-281`: HF-style names, float32, `[out, in]`).
 
 The key names already coincide.  What differs is the ROW ORDER of q_proj / k_proj: HF checkpoints are
 permuted for the half-split (`rotate_half`) RoPE, the reference rotates INTERLEAVED pairs

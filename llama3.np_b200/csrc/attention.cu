@@ -76,7 +76,7 @@ __global__ void __launch_bounds__(128) attn_decode_warp_kernel(AttnArgs a, int n
 // chain of dependent DRAM round trips per warp (two key batches in flight, then math, then the next two).  Here ONE
 // thread requests the CTA's whole key range up front - the rows of a (sequence, kv head) are contiguous in the
 // head-major cache, so a stage of SK keys is one cp.async.bulk for K and one for V - into NST shared-memory stages
-// guarded by mbarriers; the warps then run the same lane-group math on staged rows (LDS.128, conflict-free: a lane
+// guarded by mbarriers; the warps then run the same lane-group math on staged rows (16-byte shared loads, conflict-free: a lane
 // group reads one contiguous row).  Ranges longer than NST * SK keys refill stages as they are consumed.
 __device__ __forceinline__ uint32_t attn_smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void attn_bulk_g2s(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {

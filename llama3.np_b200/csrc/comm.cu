@@ -1,4 +1,4 @@
-// Tensor-parallel communication for the 8B-shaped configs (SURVEY.md 8(e)): one process per GPU,
+// Tensor-parallel communication for the 8B-shaped configs: one process per GPU,
 // heads / FFN columns / vocabulary rows sharded at load time (place_of, l3_api.cu), and one
 // sum over ranks after the attention output projection and after the FFN down projection
 // (the two row-parallel matrices).  The reference has no counterpart (single process, NumPy).

@@ -575,7 +575,7 @@ template <typename WT, int HD, int NREP>
 __global__ void __launch_bounds__(MG_THREADS, 1) decode_mega_kernel(const __grid_constant__ MegaArgs a) {
   using KVT = WT;
   // plain pointer arithmetic on the extern array (no integer round-trip), so that the compiler keeps the shared
-  // address space and the consumers' loads are LDS.128, not generic LD.E.128; no static shared memory in this
+  // address space (16-byte shared loads by the consumers, not generic ones); no static shared memory in this
   // kernel, so the dynamic window starts at offset 0
   extern __shared__ __align__(128) uint8_t smem_raw[];
   uint8_t* base = smem_raw;

@@ -5,7 +5,7 @@
 //
 // Why: sequences are independent across the whole layer stack (only attention looks back, and only within a
 // sequence), so a step needs no grid-wide barrier at all.  The kernel-per-projection graph spent 83 % of the
-// stories15M B = 256 step in 41 launches that each moved ~1 us of data (VERDICT r01); here a cluster of C CTAs
+// stories15M B = 256 step in 41 launches that each moved ~1 us of data; here a cluster of C CTAs
 // (C = n_heads) owns S sequences for the whole step, split Megatron-style INSIDE the cluster:
 //   CTA j:  q/k/v rows of head j  ->  attention of head j (all S sequences)  ->  Wo restricted to head j's
 //           columns (partial sums)  -> reduce-scatter + all-gather over DSMEM ->  gate/up rows of FFN slice j
@@ -269,7 +269,7 @@ template <class Cf> struct XBars {
 
 // Where a compute thread sits in a projection with G k-groups: a warp holds 32 / G thread tiles (4 output features
 // each, ALL S sequences), the k-group is the HIGH part of the lane index - so the eight lanes of a quarter warp read
-// 128 contiguous bytes of a weight row (conflict-free LDS.128) and the k-groups are summed with shuffles.
+// 128 contiguous bytes of a weight row (conflict-free 16-byte shared loads) and the k-groups are summed with shuffles.
 template <int F, int G> struct Tile {
   static constexpr int FPW = 32 / G, NFG = F / 4;
   int kg, fg;

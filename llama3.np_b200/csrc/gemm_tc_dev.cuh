@@ -301,10 +301,9 @@ __device__ __forceinline__ void tc_gemm_run(TcPipe& p, const CUtensorMap* tmA0p,
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(accempty0 + 8 * buf);
-        // Variant for the next round (the pattern gemm_swap.cu already runs on hardware): the CTA barrier orders
-        // the four warps' partial stores before thread 64's acq_rel atomic (cumulative release), whose acquire
-        // side + the next barrier order the last arriver's reads - instead of two __threadfence() per thread
-        // (MEMBAR + CCTL.IVALL: 12 % of this kernel's stall samples in the ncu source view).
+        // As in gemm_swap.cu: the CTA barrier orders the four warps' partial stores before thread 64's acq_rel atomic
+        // (cumulative release), whose acquire side + the next barrier order the last arriver's reads - instead of two
+        // __threadfence() per thread.
         asm volatile("bar.sync 2, 128;" ::: "memory");  // the four epilogue warps
         int* flag = reinterpret_cast<int*>(smem_raw + (tmem_slot - raw)) + 1;
         if (threadIdx.x == 64) {
@@ -323,7 +322,7 @@ __device__ __forceinline__ void tc_gemm_run(TcPipe& p, const CUtensorMap* tmA0p,
           // Greedy argmax fused into the LM head (llama3.py:320) without leaving the registers: a thread IS an
           // accumulator row, so it walks its row's columns in increasing order keeping (max, first index) and
           // merges into best[m] with ONE 64-bit atomicMax per tile.  (The shared-memory pass + per-row shuffle
-          // tree this replaces took as long as the tile's 108-MMA main loop: VERDICT r01.)
+          // tree this replaces took as long as the tile's 108-MMA main loop.)
           float bv = -INFINITY;
           int bi = 0x7fffffff;
 #pragma unroll 1
@@ -365,7 +364,7 @@ __device__ __forceinline__ void tc_gemm_run(TcPipe& p, const CUtensorMap* tmA0p,
             const float* src = part + ((size_t)(m0 + quarter * 32 + lane)) * Np + n0 + c0 + cc;
 #pragma unroll
             for (int j = 0; j < 32; ++j) v[j] = 0.f;
-            // Variant for the next round (not yet measured; same additions in the same order, so bit-identical):
+            // Same additions in the same order as a plain loop, so bit-identical:
             // slice k2 + 1 is in flight while slice k2 is added - the loop below pays one L2 round trip per slice
             // (3-8 per tile at the stories15M shapes), this one about one per tile.
             float4 nxt[8];

@@ -1,6 +1,6 @@
 // Micro-benchmark, not on any product path: what does one tcgen05.mma (M = 128, K = 32 bytes) cost as a function
 // of its kind (bf16 / tf32), its width N and the number of TMEM accumulators the issuing thread rotates over?
-// The GEMM designs of DESIGN.md 4.2 / 4.2b / 6 rest on this number (an M = 128 MMA costs about the same for
+// The GEMM designs (gemm_tc.cu, gemm_swap.cu) rest on this number (an M = 128 MMA costs about the same for
 // N = 32 as for N = 256, so narrow tiles buy parallelism, not time); scripts/mma_cost.py sweeps it.
 //
 // One warp allocates the whole TMEM, one thread issues `iters` groups of four MMAs on zero-filled, 128-byte

@@ -1,4 +1,4 @@
-// Packed device-layout weight cache (SURVEY.md 8(f)-3): the weight matrices exactly as l3_load_weight leaves them
+// Packed device-layout weight cache: the weight matrices exactly as l3_load_weight leaves them
 // on the device - fused q|k|v rows, interleaved gate/up rows, this rank's heads / FFN columns / vocabulary rows,
 // already in the model's dtype - written to one file, so that the next start streams the file straight into the
 // device buffers instead of parsing the reference's .npz (llama3.py:269, utils.py:4-5), slicing, transposing and

@@ -1,4 +1,4 @@
-"""Data-parallel plumbing for independent prompts (stories15M configs): one
+"""Data-parallel plumbing for independent prompts: one
 process per GPU, full weights on each, prompts split in contiguous row blocks, NO data-path
 collective.  torch.distributed is used only to synchronise and to combine timings / results."""
 from __future__ import annotations
@@ -54,7 +54,7 @@ def tp_unique_id(dist=None, src: int = 0) -> bytes:
 
 
 def tp_shard_shapes(dim, n_heads, n_kv_heads, hidden_dim, vocab_size, world):
-    """Per-rank shapes of the packed matrices under tensor parallelism (SURVEY.md 8(e)): heads and
+    """Per-rank shapes of the packed matrices under tensor parallelism: heads and
     FFN columns split for the column-parallel Wqkv / Wgate|Wup, input columns split for the
     row-parallel Wo / Wdown, vocabulary rows split for the LM head."""
     if n_kv_heads % world or hidden_dim % (8 * world) or vocab_size % world:

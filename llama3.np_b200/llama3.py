@@ -1,9 +1,9 @@
 """The reference's model surface on a B200: `Llama(model_path, args)`, `__call__(input_ids,
 start_pos)`, `generate(input_ids, max_new_tokens)` - same names, argument meaning and state
-semantics as `/root/reference/llama3.py:264-321`, with every numerical step running in the
+semantics as `llama3.py:264-321`, with every numerical step running in the
 sm_100a kernels behind `include/llama3_b200.h`.
 
-Kept behaviours (SURVEY.md section 0): logits come back float64 `[B, 1, VS]`; the KV cache is
+Kept behaviours: logits come back float64 `[B, 1, VS]`; the KV cache is
 per-instance state, zero at construction, never reset, addressed by the caller's
 `start_pos`; `generate` is a lazy generator yielding `[B, 1]` int64 arrays, runs prefill at
 position 0 and decode step i >= 1 at `pos = L + i` (slot L is skipped), and

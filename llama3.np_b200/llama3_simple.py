@@ -1,6 +1,6 @@
-"""The reference's FUNCTIONAL surface on a B200 (SURVEY.md 8(f)-1): `llama_init`, `llama_forward`,
+"""The reference's FUNCTIONAL surface on a B200: `llama_init`, `llama_forward`,
 `llama_generate` with the names, argument meaning and schedule of
-`/root/reference/llama3_simple.py:168-285`, over the same sm_100a kernels as `Llama`.
+`llama3_simple.py:168-285`, over the same sm_100a kernels as `Llama`.
 
 Differences from `llama3.py` that this module keeps, as the reference's functional file does:
 decode step i runs at `pos = L + i - 1` (no skipped cache slot, llama3_simple.py:279), at most

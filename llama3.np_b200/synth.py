@@ -1,10 +1,10 @@
 """Random-init weights in the reference's `.npz` key layout.
 
 The stories15M checkpoint is absent from the reference checkout
-(`/root/reference/.MISSING_LARGE_BLOBS:1`) and no Llama-3 checkpoint is reachable, so every
+(`.MISSING_LARGE_BLOBS:1`) and no Llama-3 checkpoint is reachable, so every
 parity test and benchmark runs on seeded synthetic weights written with exactly the keys
 and `[out, in]` float32 shapes the reference reads (`llama3.py:219-235, 269, 280-281`).
-Scales follow SURVEY.md §8(d): embeddings sigma 0.5, linears ~0.85/sqrt(fan_in), norm
+Scales: embeddings sigma 0.5, linears ~0.85/sqrt(fan_in), norm
 weights 1 + 0.1*N(0,1) - logits stay O(1) and top-1/top-2 gaps stay well above fp32 noise.
 """
 from __future__ import annotations

@@ -1,6 +1,6 @@
-"""Host tokenizer with the reference's interface and IDENTICAL ids (SURVEY.md 8(f)-4).
+"""Host tokenizer with the reference's interface and IDENTICAL ids.
 
-`/root/reference/tokenizer.py:5-66` looks every candidate piece up with `list.index` - O(vocabulary)
+`tokenizer.py:5-66` looks every candidate piece up with `list.index` - O(vocabulary)
 per lookup, O(V * len^2) per prompt - which becomes the visible cost of a request once the forward
 pass runs on a B200.  This class keeps the surface (`Tokenizer(model_path)`, `encode(text, add_bos=True,
 add_eos=False)`, `decode(ids)`, `bos_id = 1`, `eos_id = 2`) and the greedy highest-score merge rule, with

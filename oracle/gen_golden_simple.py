@@ -1,8 +1,8 @@
-"""Golden fixtures for the functional surface (SURVEY.md 8(f)-1).  Run in the AUTHORING container:
+"""Golden fixtures for the functional surface.  Run in the AUTHORING container:
 
     python oracle/gen_golden_simple.py
 
-Imports the unmodified `/root/reference/llama3_simple.py` (fp32, MHA only, CORRECT decode
+Imports the unmodified `llama3_simple.py` (fp32, MHA only, CORRECT decode
 positions pos = L + i - 1, stops at max_seq_len), runs `llama_forward` / `llama_generate` on seeded
 weights and stores its outputs in tests/golden/simple_*.npz.  It also checks that stepping the
 pinned oracle (`oracle/ref_llama3.py`, float64 activations) through the same position schedule

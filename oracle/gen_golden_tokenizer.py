@@ -3,7 +3,7 @@
     python oracle/gen_golden_tokenizer.py
 
 Builds a small SYNTHETIC vocabulary in the reference's file format (the real `tokenizer.model.np` is
-the reference's asset and is not copied), runs the unmodified `/root/reference/tokenizer.py` on it and
+the reference's asset and is not copied), runs the unmodified `tokenizer.py` on it and
 stores (text, ids, decoded) triples - including duplicate pieces, equal scores, unknown characters and
 the `strip` quirk of `decode` - in tests/golden/tokenizer_cases.json.
 """

@@ -1,7 +1,7 @@
 """ORACLE - test infrastructure, not product code.
 
 A CPU (NumPy) restatement of the algorithm of the reference's Llama-3 forward pass and
-greedy generate loop (`/root/reference/llama3.py:22-321`).  Only `tests/`,
+greedy generate loop (`llama3.py:22-321`).  Only `tests/`,
 `__graft_entry__.smoke()` and `bench.py`'s `cpu_baseline` / `--impl reference` legs may
 import this module; the product path (`llama3.np_b200/`) never does and has no CPU fallback.
 
@@ -9,10 +9,10 @@ Pinning: this restatement is checked bit-for-bit against the *unmodified* refere
 imported from `/root/reference` in the authoring container, by `oracle/gen_golden.py`;
 that script also writes the golden fixtures under `tests/golden/` that the CPU test-suite
 replays (the reference itself holds no absolute golden vectors - its tests are
-implementation-vs-implementation only, SURVEY.md section 4 - and its stories15M checkpoint
+implementation-vs-implementation only - and its stories15M checkpoint
 is absent, so fixtures are reference outputs on seeded random weights).
 
-Behaviours of the reference reproduced on purpose (SURVEY.md section 0):
+Behaviours of the reference reproduced on purpose:
   * float64 activations: the KV caches (`np.zeros`, llama3.py:138-153) and RoPE tables
     (llama3.py:31-38) are float64, weights stay float32; everything downstream of the
     first RoPE / first residual add is float64, logits are returned as float64.
@@ -79,8 +79,8 @@ class OracleLlama:
 
     def __init__(self, weights, args, precast: bool = False):
         """`precast=True` (large test shapes only) converts to float64 ONCE every weight that the reference
-        multiplies with float64 activations - NumPy would otherwise re-cast it on every call (the 83 % of
-        SURVEY.md section 0).  The copy is C-contiguous like the temporary NumPy makes itself, so BLAS sees the same operands and the results are bit-identical
+        multiplies with float64 activations - NumPy would otherwise re-cast it on every call (83 % of
+        its time).  The copy is C-contiguous like the temporary NumPy makes itself, so BLAS sees the same operands and the results are bit-identical
         (tests/test_oracle_cpu.py); layer 0's q / k / v projections keep float32 weights: their input
         is still float32 there (llama3.py:166-168 before the first RoPE)."""
         if isinstance(weights, str):

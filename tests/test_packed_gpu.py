@@ -1,4 +1,4 @@
-"""Packed device-layout weight cache (SURVEY.md 8(f)-3): a cached load must be bit-identical to a fresh pack,
+"""Packed device-layout weight cache: a cached load must be bit-identical to a fresh pack,
 and a pack that does not belong to the checkpoint / dtype / placement must never be served."""
 import ctypes as C
 import os

@@ -1,4 +1,4 @@
-"""Parity cases added in round 2 ('close the parity holes'): the lazy-rescale branch of the tcgen05
+"""Parity cases: the lazy-rescale branch of the tcgen05
 flash prefill, attention at an 8192-token context, end-to-end runs at the TRUE Llama-3.2-1B / Llama-3-8B widths
 (2 layers, full vocabulary), and a numeric top-1 agreement rate of the bf16 mode over 256 teacher-forced steps."""
 import numpy as np
@@ -73,7 +73,7 @@ def test_op_attention_long_context_8192():
 
 
 TRUE_WIDTHS = {
-    # name: (dim, heads, kv_heads, hidden, vocab)  -  SURVEY.md 8: the real widths, 2 layers
+    # name: (dim, heads, kv_heads, hidden, vocab)  -  the real widths, 2 layers
     "llama3.2-1b": (2048, 32, 8, 8192, 128256),
     "llama3-8b": (4096, 32, 8, 14336, 128256),
 }
@@ -81,7 +81,7 @@ TRUE_WIDTHS = {
 
 @pytest.mark.parametrize("name", list(TRUE_WIDTHS))
 def test_true_width_two_layers_end_to_end(name):
-    """D / HN / KVHN / FD / VS of the Llama-3 shapes, 2 layers (SURVEY.md 8c): fp32 mode gives the oracle's tokens
+    """D / HN / KVHN / FD / VS of the Llama-3 shapes, 2 layers: fp32 mode gives the oracle's tokens
     through the persistent batch-1 kernel (501-tile LM head, chunked rows) and through the batched path (B = 32:
     swapped-role tcgen05 GEMMs, vocabulary-wide fused argmax); bf16 mode holds the 3e-2 logit bar."""
     d, hn, kv, hid, vs = TRUE_WIDTHS[name]

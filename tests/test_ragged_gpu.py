@@ -1,4 +1,4 @@
-"""Ragged batches (extension, SURVEY.md 8(f)-2): prompts of different lengths generated in one
+"""Ragged batches (extension): prompts of different lengths generated in one
 batch must yield, sequence by sequence, exactly what each prompt yields ALONE through the oracle -
 `generate` of llama3.py (pos = L + i, slot L skipped) or the llama3_simple schedule (pos = L + i - 1).
 Covers the row-streaming path (B <= 8), the tensor-core paths (B > 8: swapped-role GEMM epilogues with

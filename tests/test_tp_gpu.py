@@ -1,6 +1,6 @@
-"""Tensor-parallel parity on two GPUs (SURVEY.md 8(e), 8B-shaped configs): one process per GPU
+"""Tensor-parallel parity on two GPUs: one process per GPU
 under torchrun; each rank's logits and greedy tokens against the single-device oracle.  Skipped
-on a single-GPU box (run with `gpurun --gpus 2`)."""
+on a single-GPU box."""
 import ctypes as C
 import json
 import os
