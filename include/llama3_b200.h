@@ -179,19 +179,28 @@ int l3_generate_ragged(L3Model* m, const int32_t* ids, const int32_t* lens, int 
 #define L3_MIX_GLA 8           /* gated linear attention: q dim^(-1/2), k (heads x dim), v (heads x vdim); a decay per key channel
                                   alpha = sigmoid(a2 (a1 h) + a2.b)^(1 / tau); S <- diag(alpha) S + k v^T, o = S^T q; RMS norm per
                                   head with weight mix.norm [vdim], times silu(g h), mix.o                                    */
+#define L3_MIX_MLSTM 9         /* matrix memory with exponential gates (xLSTM): q dim^(-1/2), k (heads x dim), v (heads x vdim), per head
+                                  i = c tanh((mix.i h + mix.i.b) / c), f = logsigmoid(c tanh((mix.f h + mix.f.b) / c)), c = gate_cap;
+                                  m <- max(f + m, i) (0 at first), S <- e^(f + m_old - m) S + e^(i - m) k v^T, n likewise with k alone,
+                                  o = S^T q / (max(|n . q|, e^(-m)) + 1e-6); RMS norm per head, weight mix.norm [heads * vdim], times
+                                  sigmoid(mix.g h), mix.o                                                                        */
 /* weights of L3_MIX_WINDOW (L3LayerSpec::attn_kind) */
 #define L3_ATTN_SINK 0
 #define L3_ATTN_SIGMOID 1
+#define L3_ATTN_SOFTMAX 2      /* ordinary softmax over the visible keys */
 /* feed-forward kinds (L3LayerSpec::ff_kind) */
 #define L3_FF_GLU 0            /* down(act(gate x) * (up x)), act = L3StackConfig::glu_act; experts: down relu(up x)^2 */
 #define L3_FF_RELU2 2          /* down(relu(up x)^2), no gate matrix */
 #define L3_FF_POLYNORM 1       /* down(P(up x)),  P(z) = a N(z) + b N(z^2) + c N(z^3) + e with element-wise powers and
                                   N(v) = v / sqrt(mean(v^2) + eps) over the ff values of a token; tensor l<i>.mlp.act = (a, b, c, e) */
+#define L3_FF_CLAMP 3          /* gated unit with clamped gate and up values (ff_limit, ff_slope) */
 /* router kinds (L3LayerSpec::router_kind) */
 #define L3_ROUTE_SOFTMAX 0     /* softmax scores, correction, groups, identity slots; the weight multiplies the expert's output */
 #define L3_ROUTE_SIGMOID_IN 1  /* scores = sigmoid(logits); the `top` largest are chosen (ties: lower slot), their weights are
                                   the scores themselves; the weight multiplies the expert's INPUT; experts are gated units
                                   down(silu(gate x) * (up x)); a shared expert of width shared_ff (0: none) runs for every token */
+#define L3_ROUTE_SOFTMAX_GLU 2 /* softmax scores, the `top` largest are chosen, weights = scores / (sum of the chosen + 1e-20), on the
+                                  expert's OUTPUT; the same gated experts and shared expert (shared_gate) */
 typedef struct L3LayerSpec {
   int32_t mixer;        /* L3_MIX_* */
   int32_t heads;        /* value heads (query heads for L3_MIX_SOFTMAX) */
@@ -224,7 +233,7 @@ typedef struct L3LayerSpec {
   int32_t rot_scale_original;
   int32_t ff_kind;           /* L3_FF_* of the dense feed-forward */
   int32_t router_kind;       /* L3_ROUTE_* of the mixture of experts */
-  int32_t shared_ff;         /* L3_ROUTE_SIGMOID_IN: width of the shared expert; 0 = none */
+  int32_t shared_ff;         /* L3_ROUTE_SIGMOID_IN, L3_ROUTE_SOFTMAX_GLU: width of the shared expert; 0 = none */
   /* L3_MIX_WINDOW (also uses heads, kv_heads, dim, vdim, scale, window, rot_dims, rot_base); rot_layout: L3_MIX_LATENT, too */
   int32_t keep_first;        /* the first keep_first tokens stay visible behind the window */
   int32_t attn_kind;         /* L3_ATTN_* */
@@ -242,6 +251,16 @@ typedef struct L3LayerSpec {
                                 kv_rank, rot_dim, rot_dims, rot_base and rot_layout must be this layer's (no mix.dkv here) */
   int32_t sink;              /* 1: a learned logit per head in the softmax denominator (tensor mix.sink) */
   int32_t gate_wide;         /* 1: mix.g has heads * vdim rows and gates value by value; 0: heads rows */
+  /* L3_MIX_WINDOW */
+  int32_t chunked;           /* 1: position i sees j <= i only where i / window == j / window (chunks counted from position 0) */
+  int32_t qk_norm;           /* 1: RMS norm per head with a weight (mix.q.norm, mix.k.norm [dim]) ahead of the rotation */
+  int32_t proj_bias;         /* 1: mix.q.b, mix.k.b, mix.v.b are added in the projections, mix.o.b in the output projection */
+  int32_t head_gate;         /* 1: head h's output times sigmoid(W_g h)_h (mix.g [heads, width]) */
+  /* L3_MIX_MLSTM (also uses heads, dim, vdim) */
+  float gate_cap;            /* soft cap of the gates' logits */
+  /* L3_FF_CLAMP: g = min(gate x, ff_limit), u = clamp(up x, -ff_limit, ff_limit); down (g sigmoid(ff_slope g) (u + 1)) */
+  float ff_limit, ff_slope;
+  int32_t shared_gate;       /* L3_ROUTE_SOFTMAX_GLU: 1: the shared expert's result times sigmoid(mlp.shared.sg . x) */
 } L3LayerSpec;
 
 typedef struct L3StackConfig {
@@ -290,6 +309,11 @@ typedef struct L3StackConfig {
    * logit_scale: multiplier of the logits, ahead of the soft cap; 0 = 1. */
   int32_t streams, tied_head;
   float logit_scale;
+  /* pre-norm stacks without streams, layer scales, token shift or grouped norms:
+   * norm_tanh 1: every norm is element-wise, tanh(alpha x) w + b (tensors <norm>, <norm>.b [width], <norm>.alpha [1]);
+   * dual_norm 1: both sublayers read the SAME stream, each through its own norm: x <- x + (mixer(n1(x)) + ff(n2(x)));
+   * loop_x0 1: ahead of every pass of the looped block but the first the embedding output joins the stream, too. */
+  int32_t norm_tanh, dual_norm, loop_x0;
 } L3StackConfig;
 
 int l3_create_stack(const L3StackConfig* cfg, const L3LayerSpec* layers, L3Model** out);
@@ -305,7 +329,8 @@ int l3_forward_rows(L3Model* m, const int32_t* ids, int B, int L, int start_pos,
 int l3_stack_runs(L3Model* m, int* n_runs_out);
 /* Recurrent state of one layer run and slot (tests): S [heads, dim, vdim] float32; conv_out (may be NULL)
  * [channels, taps - 1] float32, the convolution's tail, oldest input first.  L3_MIX_LATENT: S receives the
- * slot's latent cache [max_seq_len, kv_rank + rot_dim].  `layer` counts layer runs. */
+ * slot's latent cache [max_seq_len, kv_rank + rot_dim].  L3_MIX_MLSTM: conv_out receives the normalisers
+ * [heads, dim], then the running maxima [heads].  `layer` counts layer runs. */
 int l3_read_state(L3Model* m, int layer, int slot, float* S_out, float* conv_out);
 
 /* -- state inspection (tests): the layer's caches in the reference's layout

@@ -31,6 +31,9 @@ def __getattr__(name):  # lazy: importing the package must not require the built
     if name == "Gifudra":
         from .gifudra import Gifudra
         return Gifudra
+    if name == "Vupitar":
+        from .vupitar import Vupitar
+        return Vupitar
     if name in ("StackDecoder", "StackConfig", "LayerSpec"):
         from . import stack as _s
         return getattr(_s, name)

@@ -25,10 +25,10 @@ class L3Config(C.Structure):
 
 
 MIX_SOFTMAX, MIX_DECAY_LINEAR, MIX_GATED_DELTA, MIX_LATENT, MIX_MINGRU, MIX_DIFF = 0, 1, 2, 3, 4, 5
-MIX_WINDOW, MIX_SSD, MIX_GLA = 6, 7, 8
-ATTN_SINK, ATTN_SIGMOID = 0, 1
-FF_GLU, FF_POLYNORM, FF_RELU2 = 0, 1, 2
-ROUTE_SOFTMAX, ROUTE_SIGMOID_IN = 0, 1
+MIX_WINDOW, MIX_SSD, MIX_GLA, MIX_MLSTM = 6, 7, 8, 9
+ATTN_SINK, ATTN_SIGMOID, ATTN_SOFTMAX = 0, 1, 2
+FF_GLU, FF_POLYNORM, FF_RELU2, FF_CLAMP = 0, 1, 2, 3
+ROUTE_SOFTMAX, ROUTE_SIGMOID_IN, ROUTE_SOFTMAX_GLU = 0, 1, 2
 GLU_SILU, GLU_GELU_TANH = 0, 1
 
 
@@ -49,7 +49,9 @@ L3LayerSpec._fields_ = [("mixer", C.c_int32), ("heads", C.c_int32), ("kv_heads",
                 ("keep_first", C.c_int32), ("attn_kind", C.c_int32), ("rot_layout", C.c_int32), ("qk_unit", C.c_int32),
                 ("out_norm_groups", C.c_int32), ("tau", C.c_float), ("pair", C.POINTER(L3LayerSpec)),
                 ("mix_scale", C.c_float), ("pair_scale", C.c_float),
-                ("kv_source", C.c_int32), ("sink", C.c_int32), ("gate_wide", C.c_int32)]
+                ("kv_source", C.c_int32), ("sink", C.c_int32), ("gate_wide", C.c_int32),
+                ("chunked", C.c_int32), ("qk_norm", C.c_int32), ("proj_bias", C.c_int32), ("head_gate", C.c_int32),
+                ("gate_cap", C.c_float), ("ff_limit", C.c_float), ("ff_slope", C.c_float), ("shared_gate", C.c_int32)]
 
 
 class L3StackConfig(C.Structure):
@@ -61,7 +63,8 @@ class L3StackConfig(C.Structure):
                 ("embed_scale", C.c_float), ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32),
                 ("parallel", C.c_int32), ("norm_center", C.c_int32), ("layer_scale", C.c_int32), ("canon_taps", C.c_int32),
                 ("depth_avg", C.c_int32), ("norm_groups", C.c_int32), ("embed_norm", C.c_int32), ("loop_in", C.c_int32),
-                ("logit_softcap", C.c_float), ("streams", C.c_int32), ("tied_head", C.c_int32), ("logit_scale", C.c_float)]
+                ("logit_softcap", C.c_float), ("streams", C.c_int32), ("tied_head", C.c_int32), ("logit_scale", C.c_float),
+                ("norm_tanh", C.c_int32), ("dual_norm", C.c_int32), ("loop_x0", C.c_int32)]
 
 
 _P = C.c_void_p

@@ -1,11 +1,12 @@
-// Sliding-window attention that may keep the first tokens (L3_MIX_WINDOW): GQA with key size DK and value size DV,
-// the weight of a visible key either a softmax term whose denominator also holds a per-head sink, or sigmoid(score +
-// per-head bias) without any normalisation over keys.  Everything fp32 (FFMA): scores, weights, accumulation.
+// Attention over a sliding window or inside chunks of the sequence, which may keep the first tokens (L3_MIX_WINDOW): GQA
+// with key size DK and value size DV, the weight of a visible key either a softmax term - plain, or with a per-head sink
+// in the denominator - or sigmoid(score + per-head bias) without any normalisation over keys; an optional sigmoid gate per
+// head on the output.  Everything fp32 (FFMA): scores, weights, accumulation.
 //
-//  * win_prep_kernel     a warp per head vector of a token: rotary turn of the leading rot_dims entries at the token's
-//                        position (pairs (2i, 2i + 1) or (i, i + rot_dims / 2); angle = position * frequency in fp32,
-//                        sincosf), optional division by the vector's root mean square, q to the query buffer, k and the
-//                        value row to the caches
+//  * win_prep_kernel     a warp per head vector of a token: biases, optional RMS norm per head with a weight, rotary turn
+//                        of the leading rot_dims entries at the token's position (pairs (2i, 2i + 1) or (i, i + rot_dims / 2); angle = position * frequency in fp32,
+//                        sincosf), optional division by the turned vector's root mean square, q to the query buffer, k and
+//                        the value row to the caches
 //  * win_attn_kernel     a CTA holds 32 query rows of ONE key head - row = (token, query head of the group), token-major,
 //                        so the heads of a group share every key / value tile - and walks the keys the tile can see, 64 at
 //                        a time: first the kept tokens that lie ahead of the window, then the window.  A
@@ -42,14 +43,29 @@ __global__ void __launch_bounds__(256) win_prep_kernel(WinPrepArgs a) {
   __syncthreads();
   for (int v = warp; v < a.H + a.G; v += nw) {
     const bool is_q = v < a.H;
-    const float* src = row + (is_q ? a.q_off + (size_t)v * a.DK : a.k_off + (size_t)(v - a.H) * a.DK);
+    const size_t col = is_q ? a.q_off + (size_t)v * a.DK : a.k_off + (size_t)(v - a.H) * a.DK;
+    const float* src = row + col;
+    const float* bias = a.bias ? a.bias + col : nullptr;
+    const float* nw_ = is_q ? a.wq : a.wk;
+    float rinv = 1.0f;
+    if (nw_) {  // norm ahead of the rotation
+      float ss = 0.f;
+      for (int i = lane; i < a.DK; i += 32) { const float t = src[i] + (bias ? bias[i] : 0.f); ss = fmaf(t, t, ss); }
+      rinv = 1.0f / sqrtf(warp_sum(ss) / (float)a.DK + a.eps);
+    }
+    auto in = [&](int i) {
+      float t = src[i];
+      if (bias) t += bias[i];
+      if (nw_) t *= rinv * nw_[i];
+      return t;
+    };
     for (int i = lane; i < half; i += 32) {
       const int i0 = a.rot_layout ? i : 2 * i, i1 = a.rot_layout ? i + half : 2 * i + 1;
-      const float u = src[i0], w = src[i1];
+      const float u = in(i0), w = in(i1);
       buf[i0] = u * cs[i] - w * sn[i];
       buf[i1] = w * cs[i] + u * sn[i];
     }
-    for (int i = a.rot_dims + lane; i < a.DK; i += 32) buf[i] = src[i];
+    for (int i = a.rot_dims + lane; i < a.DK; i += 32) buf[i] = in(i);
     __syncwarp();
     float mul = 1.0f;
     if (a.unit_norm) {
@@ -68,7 +84,7 @@ __global__ void __launch_bounds__(256) win_prep_kernel(WinPrepArgs a) {
   }
   for (int i = threadIdx.x; i < a.G * a.DV; i += blockDim.x) {
     const int g = i / a.DV, d = i - g * a.DV;
-    ((KVT*)a.cache_v)[(((size_t)b * a.G + g) * a.M + pos) * a.DV + d] = from_f32<KVT>(row[a.v_off + i]);
+    ((KVT*)a.cache_v)[(((size_t)b * a.G + g) * a.M + pos) * a.DV + d] = from_f32<KVT>(row[a.v_off + i] + (a.bias ? a.bias[a.v_off + i] : 0.f));
   }
 }
 
@@ -119,7 +135,8 @@ __global__ void __launch_bounds__(256) win_attn_kernel(WinAttnArgs a) {
   const int t_lo = row0 / rep, t_hi = min(a.L - 1, (row0 + WA_ROWS - 1) / rep);
   const int p_lo = pos0 + t_lo, p_hi = pos0 + t_hi;
   // keys the tile can see: [0, ka) kept tokens ahead of the window, then [w_lo, p_hi]
-  const int w_lo = a.window > 0 ? max(0, p_lo - a.window + 1) : 0;
+  auto first_key = [&](int p) { return a.window <= 0 ? 0 : a.chunked ? p - p % a.window : max(0, p - a.window + 1); };
+  const int w_lo = first_key(p_lo);
   const int ka = min(a.keep_first, w_lo);
   const int nkeys = ka + (p_hi + 1 - w_lo);
   const int ntiles = (nkeys + WA_KEYS - 1) / WA_KEYS;
@@ -138,13 +155,14 @@ __global__ void __launch_bounds__(256) win_attn_kernel(WinAttnArgs a) {
   }
   // per-row state: rows warp, warp + 8, warp + 16, warp + 24 of the tile
   float o[WA_QW][NJ], mx[WA_QW], sum[WA_QW], hv[WA_QW];
-  int rpos[WA_QW];
+  int rpos[WA_QW], rlo[WA_QW];  // a row's position and the first key of its window / chunk
 #pragma unroll
   for (int qi = 0; qi < WA_QW; ++qi) {
     const int row = row0 + warp + qi * WA_WARPS;
     const bool live = row < nrows;
     const int t = live ? row / rep : 0, h = g * rep + (live ? row - t * rep : 0);
     rpos[qi] = live ? pos0 + t : -1;
+    rlo[qi] = live ? first_key(pos0 + t) : 0;
     hv[qi] = a.head_vec ? a.head_vec[h] : 0.f;
     const bool sink_here = a.kind == L3_ATTN_SINK && a.head_vec && split == 0;
     mx[qi] = sink_here ? hv[qi] : -INFINITY;
@@ -197,7 +215,7 @@ __global__ void __launch_bounds__(256) win_attn_kernel(WinAttnArgs a) {
       float s2[2], w[2];
 #pragma unroll
       for (int u = 0; u < 2; ++u) {
-        vis[u] = kj[u] >= 0 && kj[u] <= p && ((a.window <= 0 || p - kj[u] < a.window) || kj[u] < a.keep_first);
+        vis[u] = kj[u] >= 0 && kj[u] <= p && (kj[u] >= rlo[qi] || kj[u] < a.keep_first);
         s2[u] = sc[qi][u] * a.scale;
       }
       if (a.kind == L3_ATTN_SIGMOID) {
@@ -261,14 +279,15 @@ __global__ void __launch_bounds__(256) win_attn_kernel(WinAttnArgs a) {
       if (lane == 0) { a.part_ml[pi * 2] = mx[qi]; a.part_ml[pi * 2 + 1] = sum[qi]; }
       continue;
     }
-    const float mul = a.out_scale * (a.kind == L3_ATTN_SIGMOID ? 1.f : (sum[qi] > 0.f ? 1.0f / sum[qi] : 0.f));
+    float mul = a.out_scale * (a.kind == L3_ATTN_SIGMOID ? 1.f : (sum[qi] > 0.f ? 1.0f / sum[qi] : 0.f));
+    if (a.gate) mul *= sigmoid_f(a.gate[r * a.ld_gate + h]);
 #pragma unroll
     for (int j = 0; j < NJ; ++j) {
       const int d = win_col<NJ>(lane, j);
       if (d < a.DV) {
         const float v = o[qi][j] * mul;
         const size_t oi = r * a.ld_out + (size_t)h * a.DV + d;
-        a.out[oi] = v;
+        if (a.out) a.out[oi] = v;
         if (a.out16) a.out16[oi] = __float2bfloat16_rn(v);
       }
     }
@@ -300,10 +319,11 @@ __global__ void __launch_bounds__(128) win_attn_combine_kernel(WinAttnArgs a) {
     }
     acc = fmaf(a.part_o[pi * a.DV + d], f, acc);
   }
-  const float mul = a.out_scale * (a.kind == L3_ATTN_SIGMOID ? 1.f : (den > 0.f ? 1.0f / den : 0.f));
+  float mul = a.out_scale * (a.kind == L3_ATTN_SIGMOID ? 1.f : (den > 0.f ? 1.0f / den : 0.f));
+  if (a.gate) mul *= sigmoid_f(a.gate[r * a.ld_gate + h]);
   const float v = acc * mul;
   const size_t oi = r * a.ld_out + (size_t)h * a.DV + d;
-  a.out[oi] = v;
+  if (a.out) a.out[oi] = v;
   if (a.out16) a.out16[oi] = __float2bfloat16_rn(v);
 }
 

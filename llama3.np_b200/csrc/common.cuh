@@ -67,7 +67,7 @@ __device__ __forceinline__ float gelu_tanh_ref(float z) {
   return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 // activation of a gated linear unit's gate column (EpiArgs::act)
-enum GluAct : int { GLU_SILU = 0, GLU_GELU_TANH = 1 };
+enum GluAct : int { GLU_SILU = 0, GLU_GELU_TANH = 1, GLU_CLAMP = 2 };
 __device__ __forceinline__ float glu_act(int act, float z) { return act == GLU_GELU_TANH ? gelu_tanh_ref(z) : silu_ref(z); }
 
 __device__ __forceinline__ float warp_sum(float v) {
@@ -187,12 +187,24 @@ struct EpiArgs {
   int L;                 // tokens per sequence in this call: row m -> (b = m / L, t = m % L)
   int HD, HN, KVHN, M;   // head_dim, local heads, local kv heads, max_seq_len
   int act;               // SWIGLU: GluAct of the gate column (0 = silu)
+  float act_limit, act_slope;  // GLU_CLAMP: g = min(gate, limit), u = clamp(up, -limit, limit); g sigmoid(slope g) (u + 1)
   int unary;             // STORE: UnaryAct applied to every output value
   // SWIGLU with a routing weight on the unit's INPUT: output j of row m is act(w g) * (w u) with
   // w = glu_w[m * glu_w_ld + j / glu_group] for j < glu_groups * glu_group and 1 beyond (a shared expert); w = 0 gives 0.
   const float* glu_w;    // null: no weight
   int glu_w_ld, glu_group, glu_groups;
 };
+// a gated unit's output from its gate and up values (FAST: exp2-based exponential and approximate divide)
+template <bool FAST>
+__device__ __forceinline__ float glu_pair(const EpiArgs& e, float g, float u) {
+  if (e.act == GLU_CLAMP) {
+    g = fminf(g, e.act_limit);
+    u = fminf(fmaxf(u, -e.act_limit), e.act_limit);
+    const float z = -e.act_slope * g;
+    return (FAST ? __fdividef(g, 1.0f + __expf(z)) : g / (1.0f + expf(z))) * (u + 1.0f);
+  }
+  return glu_act(e.act, g) * u;
+}
 // routing weight of output j (= column pair index) of row m
 __device__ __forceinline__ float glu_in_weight(const EpiArgs& e, int m, int j) {
   if (!e.glu_w) return 1.0f;
@@ -232,7 +244,7 @@ __device__ __forceinline__ void epilogue_pair(int epi, const EpiArgs& e, int m, 
     if (has1) e.out[o + 1] = e.resid[o + 1] + v1;
   } else if (epi == EPI_SWIGLU) {
     if (e.glu_w) { const float w = glu_in_weight(e, m, col >> 1); v0 *= w; v1 *= w; }
-    float h = glu_act(e.act, v0) * v1;
+    float h = glu_pair<false>(e, v0, v1);
     size_t o = (size_t)m * e.ld_out + (col >> 1);
     if (e.out_lo) {
       float hh, hl;

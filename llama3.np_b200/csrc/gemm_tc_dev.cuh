@@ -502,7 +502,7 @@ __device__ __forceinline__ void tc_gemm_run(TcPipe& p, const CUtensorMap* tmA0p,
               float2 t = *reinterpret_cast<const float2*>(Cs + i * LDC + cp);
               if (e.glu_w) { const float w = glu_in_weight(e, m, col >> 1); t.x *= w; t.y *= w; }
               float hv;
-              if (e.act != GLU_SILU) hv = glu_act(e.act, t.x) * t.y;
+              if (e.act != GLU_SILU) hv = glu_pair<KIND == TC_BF16>(e, t.x, t.y);
               else if constexpr (KIND == TC_BF16) hv = t.x * __fdividef(1.0f, 1.0f + __expf(-t.x)) * t.y;
               else hv = silu_ref(t.x) * t.y;
               const size_t o = (size_t)m * e.ld_out + (col >> 1);

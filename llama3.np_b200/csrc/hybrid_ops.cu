@@ -5,7 +5,7 @@
 //                        the call from the slot's tail), dt = softplus(dt + bias), decay = exp(-exp(A_log) dt) per head,
 //                        and the recurrence's operands: keys B, queries C, values dt * x, plus x itself for the skip term
 //  * gla_prep_kernel     q * dim^(-1/2) and the per-channel decay sigmoid(z + b)^(1 / tau) = exp(-softplus(-(z + b)) / tau)
-//  * mix_out_kernel      skip term, gate (ahead of or behind the norm, sigmoid or silu), RMS norm in groups, weight, scale;
+//  * mix_out_kernel      normaliser of an mLSTM, skip term, gate (ahead of or behind the norm, sigmoid or silu), RMS norm in groups, weight, scale;
 //                        writes into a slice of a wider row so that two mixers side by side share one output projection
 //  * softcap_kernel      c tanh(x / c)
 //  * concat_rows_kernel  [a | b] row by row (+ bf16 mirror): the input of the looped block's entry projection
@@ -86,8 +86,13 @@ __global__ void __launch_bounds__(256) mix_out_kernel(MixOutArgs a, int wpg) {
   const float* grow = a.gate ? a.gate + r * a.ld_gate : nullptr;
   const float* xrow = a.skip_d ? a.skip_x + r * a.n : nullptr;
   auto act = [&](float z) { return a.gate_act ? z * sigmoid_f(z) : sigmoid_f(z); };
+  float dinv = 1.0f;  // mLSTM: one over the group's head's normaliser
+  if (a.nq && live) {
+    const size_t rh = r * (a.n / a.DV) + (g * a.group) / a.DV;
+    dinv = 1.0f / (fmaxf(fabsf(a.nq[rh]), a.floor[rh]) + 1e-6f);
+  }
   auto val = [&](int i) {
-    float y = orow[i];
+    float y = orow[i] * dinv;
     if (xrow) y = fmaf(a.skip_d[i / a.DV], xrow[i], y);
     if (grow && a.pre_gate) y *= act(grow[i]);
     return y;
@@ -110,7 +115,7 @@ __global__ void __launch_bounds__(256) mix_out_kernel(MixOutArgs a, int wpg) {
     float v = val(c) * rinv * a.w[c % a.wlen];
     if (grow && !a.pre_gate) v *= act(grow[c]);
     v *= a.out_scale;
-    a.out[r * a.ld_out + c] = v;
+    if (a.out) a.out[r * a.ld_out + c] = v;
     if (a.out16) a.out16[r * a.ld_out + c] = __float2bfloat16_rn(v);
   }
 }
@@ -152,7 +157,7 @@ cudaError_t launch_gla_prep(const float* q, int ld, float q_mul, const float* z,
 }
 
 cudaError_t launch_mix_out(const MixOutArgs& a, int rows, cudaStream_t s) {
-  if (a.group < 1 || a.n % a.group != 0) return cudaErrorInvalidValue;
+  if (a.group < 1 || a.n % a.group != 0 || (a.nq && a.DV % a.group != 0)) return cudaErrorInvalidValue;
   const int groups = a.n / a.group;
   const int wpg = a.group >= 1024 ? 8 : a.group >= 512 ? 4 : a.group >= 256 ? 2 : 1;  // warps per group
   const int gpc = 8 / wpg;

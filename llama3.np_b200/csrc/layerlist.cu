@@ -34,6 +34,9 @@
 //   or dense: a gated unit, or down(relu(up x)^2) with the square in the up projection's epilogue.
 // With residual streams (L3StackConfig::streams, stream_ops.cu) the sublayers' output projections store their result and one
 // launch per sublayer border re-mixes the S residual rows of a token and forms the next sublayer's normed input.
+// With dual_norm both sublayers read the same stream through norms of their own; norms can be element-wise (norm_tanh,
+// tanh_norm.cu: one launch forms both inputs, the stream's additions ahead of a layer and the output biases); a dense
+// feed-forward then shares the mixer's output projection (its hidden values are more columns of the same product's input).
 // Parallel stacks (L3StackConfig::parallel, ll_enqueue_parallel):  h = norm1(x);  X_new = x + ls1 mixer(h + conv1(h)) +
 // ls2 ff(h + conv2(h));  x <- sum_j dwa[j] X_j over the embedding output and every layer result so far.  One mixer:
 //
@@ -65,15 +68,20 @@ static int pad8(int v) { return (v + 7) & ~7; }
 
 // ------------------------------------------------------------------------------ create
 // the mixers that pre-norm stacks run through ll_mix_unit, alone or two side by side
-static bool unit_mixer(int mixer) { return mixer == L3_MIX_WINDOW || mixer == L3_MIX_SSD || mixer == L3_MIX_GLA || mixer == L3_MIX_GATED_DELTA; }
+static bool unit_mixer(int mixer) { return mixer == L3_MIX_WINDOW || mixer == L3_MIX_SSD || mixer == L3_MIX_GLA || mixer == L3_MIX_GATED_DELTA || mixer == L3_MIX_MLSTM; }
+// a mixture of gated experts (and maybe a shared one): w13 / w2 hold all of them side by side
+static bool gated_experts(const L3LayerSpec& s) { return s.experts > 0 && s.router_kind != L3_ROUTE_SOFTMAX; }
 
 static int check_unit(const L3LayerSpec& s, int i) {
   REQUIRE(nullptr, s.heads >= 1 && s.dim >= 1 && s.vdim >= 1, "layer %d: bad sizes", i);
   if (s.mixer == L3_MIX_WINDOW) {
     REQUIRE(nullptr, s.kv_heads >= 1 && s.heads % s.kv_heads == 0, "layer %d: heads %% kv_heads != 0", i);
     REQUIRE(nullptr, s.rot_dims >= 0 && s.rot_dims <= s.dim && s.rot_dims % 2 == 0 && (s.rot_dims == 0 || s.rot_base > 0), "layer %d: bad rotary sizes", i);
-    REQUIRE(nullptr, s.window >= 0 && s.keep_first >= 0 && (s.attn_kind == L3_ATTN_SINK || s.attn_kind == L3_ATTN_SIGMOID), "layer %d: bad window / kind", i);
+    REQUIRE(nullptr, s.window >= 0 && s.keep_first >= 0 && s.attn_kind >= L3_ATTN_SINK && s.attn_kind <= L3_ATTN_SOFTMAX, "layer %d: bad window / kind", i);
     REQUIRE(nullptr, win_attn_supported(s.dim, s.vdim), "layer %d: head sizes %d, %d unsupported", i, s.dim, s.vdim);
+  } else if (s.mixer == L3_MIX_MLSTM) {
+    REQUIRE(nullptr, s.gate_cap > 0.f && s.vdim <= 8192, "layer %d: bad gate cap / value size", i);
+    REQUIRE(nullptr, recur_supported(s.dim, s.vdim), "layer %d: state %d x %d unsupported", i, s.dim, s.vdim);
   } else if (s.mixer == L3_MIX_SSD) {
     REQUIRE(nullptr, s.kv_heads >= 1 && s.heads % s.kv_heads == 0, "layer %d: heads %% groups != 0", i);
     REQUIRE(nullptr, s.conv_taps >= 1 && s.conv_taps <= 64, "layer %d: bad conv size", i);
@@ -91,21 +99,24 @@ static int check_unit(const L3LayerSpec& s, int i) {
 }
 
 static int check_spec(const L3StackConfig* c, const L3LayerSpec& s, int i) {
-  REQUIRE(nullptr, s.mixer >= L3_MIX_SOFTMAX && s.mixer <= L3_MIX_GLA, "layer %d: unknown mixer %d", i, s.mixer);
+  REQUIRE(nullptr, s.mixer >= L3_MIX_SOFTMAX && s.mixer <= L3_MIX_MLSTM, "layer %d: unknown mixer %d", i, s.mixer);
   REQUIRE(nullptr, s.mixer < L3_MIX_WINDOW || (c->norm_input && !c->parallel), "layer %d: this mixer is built for pre-norm layers (norm_input)", i);
   REQUIRE(nullptr, !s.pair || (c->norm_input && !c->parallel && unit_mixer(s.mixer) && unit_mixer(s.pair->mixer) && !s.pair->pair),
-          "layer %d: two mixers side by side need a pre-norm stack and mixers of the window / state-space / gated-linear / gated-delta kinds", i);
+          "layer %d: two mixers side by side need a pre-norm stack and mixers of the window / state-space / gated-linear / gated-delta / mLSTM kinds", i);
   if (c->norm_input && !c->parallel && unit_mixer(s.mixer)) {
     int rc = check_unit(s, i);
     if (rc == L3_OK && s.pair) rc = check_unit(*s.pair, i);
     if (rc != L3_OK) return rc;
   }
   REQUIRE(nullptr, (s.mixer == L3_MIX_DIFF) == (c->parallel != 0), "layer %d: differential attention and parallel layers come together", i);
-  REQUIRE(nullptr, s.ff_kind == L3_FF_GLU || (s.ff_kind == L3_FF_POLYNORM && c->parallel) || (s.ff_kind == L3_FF_RELU2 && c->norm_input && !c->parallel),
-          "layer %d: this feed-forward kind is built for %s layers", i, s.ff_kind == L3_FF_RELU2 ? "pre-norm" : "parallel");
-  REQUIRE(nullptr, s.ff_kind != L3_FF_RELU2 || s.experts == 0, "layer %d: experts have a feed-forward kind of their own", i);
+  REQUIRE(nullptr, s.ff_kind == L3_FF_GLU || (s.ff_kind == L3_FF_POLYNORM && c->parallel) || ((s.ff_kind == L3_FF_RELU2 || s.ff_kind == L3_FF_CLAMP) && c->norm_input && !c->parallel),
+          "layer %d: this feed-forward kind is built for %s layers", i, s.ff_kind == L3_FF_POLYNORM ? "parallel" : "pre-norm");
+  REQUIRE(nullptr, s.ff_kind != L3_FF_CLAMP || s.ff == 0 || s.ff_limit > 0.f, "layer %d: bad feed-forward limit", i);
+  REQUIRE(nullptr, (s.ff_kind != L3_FF_RELU2 && s.ff_kind != L3_FF_CLAMP) || s.experts == 0, "layer %d: experts have a feed-forward kind of their own", i);
   REQUIRE(nullptr, s.mixer == L3_MIX_LATENT || (!s.kv_source && !s.sink && !s.gate_wide), "layer %d: shared caches, the sink switch and wide gates belong to latent attention", i);
-  REQUIRE(nullptr, s.router_kind == L3_ROUTE_SOFTMAX || (s.router_kind == L3_ROUTE_SIGMOID_IN && c->parallel), "layer %d: this router kind is built for parallel layers", i);
+  REQUIRE(nullptr, s.router_kind == L3_ROUTE_SOFTMAX || (s.router_kind == L3_ROUTE_SIGMOID_IN && c->parallel) || (s.router_kind == L3_ROUTE_SOFTMAX_GLU && c->norm_input && !c->parallel),
+          "layer %d: this router kind is built for %s layers", i, s.router_kind == L3_ROUTE_SIGMOID_IN ? "parallel" : "pre-norm");
+  REQUIRE(nullptr, !s.shared_gate || (s.router_kind == L3_ROUTE_SOFTMAX_GLU && s.shared_ff > 0), "layer %d: a shared expert's gate without such an expert", i);
   REQUIRE(nullptr, !(c->parallel && s.experts > 0) || s.router_kind == L3_ROUTE_SIGMOID_IN, "layer %d: parallel layers take the sigmoid router", i);
   REQUIRE(nullptr, s.heads >= 1 && s.dim >= 1 && s.vdim >= 1 && s.ff >= 0, "layer %d: bad sizes", i);
   REQUIRE(nullptr, s.mixer <= L3_MIX_GATED_DELTA || c->norm_input, "layer %d: this mixer is built for pre-norm layers (norm_input)", i);
@@ -115,7 +126,7 @@ static int check_spec(const L3StackConfig* c, const L3LayerSpec& s, int i) {
     const int n = s.experts + s.identity;
     REQUIRE(nullptr, c->norm_input, "layer %d: the mixture of experts is built for pre-norm layers (norm_input)", i);
     REQUIRE(nullptr, s.ff >= 1 && s.identity >= 0 && s.top >= 1 && s.top <= n && n <= 1024, "layer %d: bad expert counts", i);
-    REQUIRE(nullptr, s.router_kind == L3_ROUTE_SOFTMAX || (s.identity == 0 && s.top <= s.experts && s.shared_ff >= 0), "layer %d: bad sigmoid-router sizes", i);
+    REQUIRE(nullptr, s.router_kind == L3_ROUTE_SOFTMAX || (s.identity == 0 && s.top <= s.experts && s.shared_ff >= 0), "layer %d: bad router sizes", i);
     REQUIRE(nullptr, s.groups >= 1 && n % s.groups == 0 && s.groups_keep >= 1 && s.groups_keep <= s.groups, "layer %d: bad expert groups", i);
   }
   if (s.mixer == L3_MIX_LATENT) {
@@ -149,19 +160,27 @@ static int check_spec(const L3StackConfig* c, const L3LayerSpec& s, int i) {
 
 // Segment layout of a unit mixer's share of the fused input projection (offsets relative to the unit's first column),
 // the width of its share of the output projection's input, and its small fp32 tensors.
-static int ll_alloc_unit(LLLayer& L, size_t w) {
+static int ll_alloc_unit(LLLayer& L, size_t w, size_t row_bytes) {  // row_bytes: a fp32 vector of the model's width
   const L3LayerSpec& s = L.spec;
   const int H = s.heads, G = s.kv_heads, DK = s.dim, DV = s.vdim;
   cudaError_t e = cudaSuccess;
   auto al = [&](void** p, size_t bytes) { if (e == cudaSuccess) e = cudaMalloc(p, std::max<size_t>(16, bytes)); };
   L.n_ctx = H * DV;
   if (s.mixer == L3_MIX_WINDOW) {
-    L.off_q = 0; L.off_k = H * DK; L.off_v = L.off_k + G * DK; L.n_in = pad8(L.off_v + G * DV);  // q | k | v
-    al((void**)&L.head_vec, (size_t)H * 4);
+    L.off_q = 0; L.off_k = H * DK; L.off_v = L.off_k + G * DK; L.off_g = L.off_v + G * DV; L.n_in = pad8(L.off_g + (s.head_gate ? H : 0));  // q | k | v (| g)
+    if (s.attn_kind != L3_ATTN_SOFTMAX) al((void**)&L.head_vec, (size_t)H * 4);
+    if (s.qk_norm) { al((void**)&L.q_norm, (size_t)DK * 4); al((void**)&L.k_norm, (size_t)DK * 4); }
+    if (s.proj_bias) { al((void**)&L.in_bias, (size_t)L.off_g * 4); al((void**)&L.o_bias, row_bytes); }
     al((void**)&L.inv_freq, (size_t)std::max(1, s.rot_dims / 2) * 4);
     std::vector<float> f(std::max(1, s.rot_dims / 2), 0.f);
     for (int j = 0; j < s.rot_dims / 2; ++j) f[j] = (float)pow(s.rot_base, -2.0 * j / s.rot_dims);
     if (e == cudaSuccess) e = cudaMemcpy(L.inv_freq, f.data(), f.size() * 4, cudaMemcpyHostToDevice);
+  } else if (s.mixer == L3_MIX_MLSTM) {
+    // every segment starts on a multiple of 8 columns: 16-byte rows for the recurrence, which reads them in place
+    L.off_q = 0; L.off_k = pad8(H * DK); L.off_v = L.off_k + pad8(H * DK); L.off_g = L.off_v + pad8(H * DV); L.off_b = L.off_g + pad8(H * DV);
+    L.n_in = pad8(L.off_b + 2 * H);
+    al((void**)&L.in_bias, (size_t)2 * H * 4);
+    al((void**)&L.mix_norm, (size_t)H * DV * 4);
   } else if (s.mixer == L3_MIX_SSD) {
     // z | x | B | C | dt as the checkpoint lays them out: x, B, C stay contiguous (a convolution channel is a column)
     const int inner = H * DV, gn = G * DK;
@@ -232,6 +251,11 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
   REQUIRE(nullptr, (c->norm_input && !c->parallel) || (c->norm_groups <= 1 && !c->embed_norm && !c->loop_in && !(c->logit_softcap > 0.f)),
           "grouped norms, the embedding norm, the loop's entry projection and the logit cap are built for pre-norm stacks");
   REQUIRE(nullptr, !c->loop_in || c->loop_times > 0, "loop_in without a loop");
+  REQUIRE(nullptr, pre || (!c->norm_tanh && !c->dual_norm && !c->loop_x0), "element-wise norms, two norms of one stream and loop_x0 are built for pre-norm stacks");
+  if (c->norm_tanh || c->dual_norm || c->loop_x0)
+    REQUIRE(nullptr, !c->token_shift && !c->streams && !c->layer_scale && c->norm_groups <= 1 && !c->embed_norm && !(c->norm_tanh && c->norm_scalar),
+            "element-wise norms, two norms of one stream and loop_x0 exclude token shift, streams, layer scales, grouped norms and the embedding norm");
+  REQUIRE(nullptr, !c->loop_x0 || (c->loop_times > 0 && !c->loop_in), "loop_x0 without a loop, or beside loop_in");
   REQUIRE(nullptr, !(c->norm_groups > 1 && c->norm_scalar), "grouped norms have one weight per coordinate");
   L3Model* m = new L3Model();
   LayerList* ll = m->ll = new LayerList();
@@ -264,6 +288,7 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
   if (c->tied_head) m->lm_head = m->embed;
   else AL(m->lm_head, (size_t)c->vocab * W * w);
   AL(m->norm_final, (size_t)W * 4);
+  if (c->norm_tanh) { AL(ll->final_b, (size_t)W * 4); AL(ll->final_alpha, 4); }
   if (sd) AL(ll->side_embed, (size_t)c->vocab * c->n_layers * sd * w);
   ll->streams = c->streams > 0 ? c->streams : (pre && c->layer_scale) ? 1 : 0;
   if (ll->streams && !c->streams) {
@@ -287,8 +312,8 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
       L.spec.pair = nullptr;  // the caller's record is not kept
     }
     if (unit_mixer(s.mixer) && c->norm_input) {
-      int rc = ll_alloc_unit(L, w);
-      if (rc == L3_OK && L.pair) rc = ll_alloc_unit(*L.pair, w);
+      int rc = ll_alloc_unit(L, w, (size_t)W * 4);
+      if (rc == L3_OK && L.pair) rc = ll_alloc_unit(*L.pair, w, (size_t)W * 4);
       if (rc != L3_OK) { l3_destroy(m); return rc; }
     } else if (s.mixer == L3_MIX_LATENT) {
       // dq | dkv | g rows, every segment on a multiple of 8 columns of the projection's output (no dkv with a shared cache)
@@ -363,13 +388,17 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
     const int n_ctx = (s.mixer == L3_MIX_MINGRU ? DK : H * DV) + (L.pair ? L.pair->n_ctx : 0);  // columns the output projection reads
     L.n_ctx = n_ctx - (L.pair ? L.pair->n_ctx : 0);
     L.in_base = 0; L.ctx_base = 0; L.ctx_ld = n_ctx;
-    if (L.pair) { L.pair->in_base = L.n_in; L.pair->ctx_base = L.n_ctx; L.pair->ctx_ld = n_ctx; L.n_in += L.pair->n_in; L.pair->in_ld = L.n_in; }
+    if (c->dual_norm && unit_mixer(s.mixer) && s.ff > 0 && s.experts == 0) { L.h_base = pad8(n_ctx); L.ctx_ld = pad8(L.h_base + s.ff); }
+    if (L.pair) { L.pair->in_base = L.n_in; L.pair->ctx_base = L.n_ctx; L.pair->ctx_ld = L.ctx_ld; L.n_in += L.pair->n_in; L.pair->in_ld = L.n_in; }
     L.in_ld = L.n_in;  // n_in: the rows of the whole fused projection
     AL(L.w_in, (size_t)L.n_in * W * w);
     cudaMemset(L.w_in, 0, (size_t)L.n_in * W * w);  // padding rows project to zero
-    AL(L.w_o, (size_t)W * n_ctx * w);
+    AL(L.w_o, (size_t)W * L.ctx_ld * w);
+    cudaMemset(L.w_o, 0, (size_t)W * L.ctx_ld * w);  // padding columns take nothing
+    if (L.h_base) L.w2 = (char*)L.w_o + (size_t)L.h_base * w;
     if (L.pair) { L.pair->w_in = (char*)L.w_in + (size_t)L.pair->in_base * W * w; L.pair->w_o = (char*)L.w_o + (size_t)L.pair->ctx_base * w; }
     AL(L.norm1, (size_t)W * 4);
+    for (int q = 0; q < (s.ff > 0 ? 2 : 1) && c->norm_tanh; ++q) { AL(L.norm_b[q], (size_t)W * 4); AL(L.norm_alpha[q], 4); }
     if (c->token_shift) AL(L.shift, (size_t)W * 4);
     if (c->layer_scale) { AL(L.ls1, (size_t)W * 4); if (s.ff > 0) AL(L.ls2, (size_t)W * 4); }
     if (c->canon_taps > 0) { AL(L.canon1, (size_t)W * c->canon_taps * 4); if (s.ff > 0) AL(L.canon2, (size_t)W * c->canon_taps * 4); }
@@ -382,11 +411,12 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
       AL(L.hc_out[q], (size_t)S * 4);
       AL(L.hc_mix[q], (size_t)S * S * 4);
     }
-    if (s.experts > 0 && s.router_kind == L3_ROUTE_SIGMOID_IN) {
+    if (gated_experts(s)) {
       L.ff_total = s.experts * s.ff + s.shared_ff;
+      if (!c->parallel) AL(L.norm2, (size_t)W * 4);
       AL(L.w13, (size_t)2 * L.ff_total * W * w);
       AL(L.w2, (size_t)W * L.ff_total * w);
-      AL(L.router, (size_t)s.experts * W * 4);
+      AL(L.router, (size_t)(s.experts + s.shared_gate) * W * 4);  // a shared expert's gate is one more row
     } else if (s.ff > 0 && s.ff_kind == L3_FF_POLYNORM) {
       AL(L.w13, (size_t)s.ff * W * w);
       AL(L.w2, (size_t)W * s.ff * w);
@@ -399,7 +429,7 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
       AL(L.correction, (size_t)(s.experts + s.identity) * 4);
     } else if (s.ff > 0) {
       AL(L.w13, (size_t)(s.ff_kind == L3_FF_RELU2 ? 1 : 2) * s.ff * W * w);
-      AL(L.w2, (size_t)W * s.ff * w);
+      if (!L.h_base) AL(L.w2, (size_t)W * s.ff * w);
       if (!c->parallel) AL(L.norm2, (size_t)W * 4);
     }
     if (sd) {
@@ -409,6 +439,7 @@ extern "C" int l3_create_stack(const L3StackConfig* c, const L3LayerSpec* specs,
     }
     ll->max_in = std::max(ll->max_in, L.n_in);
     ll->max_o = std::max(ll->max_o, std::max(std::max(H * DV, H * DK), n_ctx));
+    ll->max_ctx = std::max(ll->max_ctx, L.ctx_ld);
     if (L.pair) ll->max_o = std::max(ll->max_o, std::max(L.pair->spec.heads * L.pair->spec.vdim, L.pair->spec.heads * L.pair->spec.dim));
     if (L.ff_total) ll->max_ff = std::max(ll->max_ff, L.ff_total);
     if (s.mixer == L3_MIX_LATENT) ll->max_o = std::max(ll->max_o, H * s.kv_rank);
@@ -475,8 +506,27 @@ static bool ll_place_unit(L3Model* m, LLLayer& L, const std::string& r, LLPlace*
     if (r == "mix.q") return seg(L.off_q, (int64_t)H * DK, 2.f);
     if (r == "mix.k") return seg(L.off_k, (int64_t)G * DK, 2.f);
     if (r == "mix.v") return seg(L.off_v, (int64_t)G * DV);
+    if (r == "mix.g") return s.head_gate && seg(L.off_g, H);
+    if (r == "mix.q.norm") return L.q_norm && vec(L.q_norm, DK, 1.f, 0.1f);
+    if (r == "mix.k.norm") return L.k_norm && vec(L.k_norm, DK, 1.f, 0.1f);
+    if (r == "mix.q.b") return L.in_bias && vec(L.in_bias + L.off_q, (int64_t)H * DK, 0.f, 0.2f);
+    if (r == "mix.k.b") return L.in_bias && vec(L.in_bias + L.off_k, (int64_t)G * DK, 0.f, 0.2f);
+    if (r == "mix.v.b") return L.in_bias && vec(L.in_bias + L.off_v, (int64_t)G * DV, 0.f, 0.2f);
+    if (r == "mix.o.b") return L.o_bias && vec(L.o_bias, W, 0.f, 0.1f);
     if (r == "mix.sink") return s.attn_kind == L3_ATTN_SINK && vec(L.head_vec, H, 0.5f, 0.5f);
     if (r == "mix.pb") return s.attn_kind == L3_ATTN_SIGMOID && vec(L.head_vec, H, -2.f, 0.5f);
+    return false;
+  }
+  if (s.mixer == L3_MIX_MLSTM) {
+    if (r == "mix.q") return seg(L.off_q, (int64_t)H * DK);
+    if (r == "mix.k") return seg(L.off_k, (int64_t)H * DK);
+    if (r == "mix.v") return seg(L.off_v, (int64_t)H * DV);
+    if (r == "mix.g") return seg(L.off_g, (int64_t)H * DV);
+    if (r == "mix.i") return seg(L.off_b, H);
+    if (r == "mix.f") return seg(L.off_b + H, H);
+    if (r == "mix.i.b") return vec(L.in_bias, H, -1.f, 0.5f);
+    if (r == "mix.f.b") return vec(L.in_bias + H, H, 3.f, 1.f);
+    if (r == "mix.norm") return vec(L.mix_norm, (int64_t)H * DV, 1.f, 0.1f);
     return false;
   }
   if (s.mixer == L3_MIX_SSD) {
@@ -520,7 +570,16 @@ static bool ll_place_unit(L3Model* m, LLLayer& L, const std::string& r, LLPlace*
 }
 
 static std::vector<const char*> ll_unit_names(const L3LayerSpec& s) {
-  if (s.mixer == L3_MIX_WINDOW) return {"q", "k", "v", s.attn_kind == L3_ATTN_SIGMOID ? "pb" : "sink", "o"};
+  if (s.mixer == L3_MIX_WINDOW) {
+    std::vector<const char*> v = {"q", "k", "v"};
+    if (s.attn_kind != L3_ATTN_SOFTMAX) v.push_back(s.attn_kind == L3_ATTN_SIGMOID ? "pb" : "sink");
+    v.push_back("o");
+    if (s.proj_bias) v.insert(v.end(), {"q.b", "k.b", "v.b", "o.b"});
+    if (s.qk_norm) v.insert(v.end(), {"q.norm", "k.norm"});
+    if (s.head_gate) v.push_back("g");
+    return v;
+  }
+  if (s.mixer == L3_MIX_MLSTM) return {"q", "k", "v", "g", "i", "i.b", "f", "f.b", "norm", "o"};
   if (s.mixer == L3_MIX_SSD) return {"in", "conv", "conv.b", "dt_bias", "A_log", "D", "norm", "o"};
   if (s.mixer == L3_MIX_GLA) return {"q", "k", "v", "g", "a1", "a2", "a2.b", "norm", "o"};
   return {"q", "k", "v", "b", "a1", "a2", "g1", "g2", "norm", "A_log", "dt_bias", "q.conv", "k.conv", "v.conv", "o"};
@@ -555,6 +614,8 @@ static bool ll_place(L3Model* m, const std::string& name, LLPlace* p) {
   if (name == "embed") { const bool ok = mat(m->embed, V, W); p->scale = pre ? 0.1f : 1.0f; return ok; }
   if (name == "head") return !ll->cfg.tied_head && mat(m->lm_head, V, W);
   if (name == "final.norm") return norm(m->norm_final);
+  if (name == "final.norm.b") return ll->final_b && vec(ll->final_b, W, 0.f, 0.1f);
+  if (name == "final.norm.alpha") return ll->final_alpha && vec(ll->final_alpha, 1, 0.7f, 0.1f);
   if (name == "loop.step") return ll->loop_step && fmat(ll->loop_step, ll->cfg.loop_times, W, 0.3f);
   if (name == "loop.in") { const bool ok = ll->loop_in && mat(ll->loop_in, W, (int64_t)2 * W); p->scale *= 1.4f; return ok; }
   if (name == "embed.norm") return ll->embed_norm && norm(ll->embed_norm);
@@ -567,6 +628,11 @@ static bool ll_place(L3Model* m, const std::string& name, LLPlace* p) {
   const int H = s.heads, G = s.kv_heads, DK = s.dim, DV = s.vdim;
   if (r == "norm1") return norm(L.norm1);
   if (r == "norm2") return s.ff > 0 && L.norm2 && norm(L.norm2);
+  for (int q = 0; q < 2; ++q) {
+    const std::string h = q ? "norm2" : "norm1";
+    if (r == h + ".b") return L.norm_b[q] && vec(L.norm_b[q], W, 0.f, 0.1f);
+    if (r == h + ".alpha") return L.norm_alpha[q] && vec(L.norm_alpha[q], 1, 0.7f, 0.1f);
+  }
   for (int q = 0; q < 2 && ll->cfg.streams > 0; ++q) {
     const int S = ll->cfg.streams;
     const std::string h = q ? "hc2." : "hc1.";
@@ -579,8 +645,9 @@ static bool ll_place(L3Model* m, const std::string& name, LLPlace* p) {
   if (r == "canon1") return L.canon1 && fmat(L.canon1, W, ll->cfg.canon_taps, 0.3f / (float)ll->cfg.canon_taps);
   if (r == "canon2") return L.canon2 && fmat(L.canon2, W, ll->cfg.canon_taps, 0.3f / (float)ll->cfg.canon_taps);
   if (r == "dwa") return L.dwa && vec(L.dwa, li + 2, 1.f / (float)(li + 2), 0.3f / (float)(li + 2));
-  if (L.ff_total) {  // sigmoid-routed gated experts + shared expert: gate / up rows interleaved, expert by expert
+  if (L.ff_total) {  // gated experts + shared expert: gate / up rows interleaved, expert by expert
     if (r == "mlp.router") return fmat(L.router, s.experts, W, 3.0f / sqrtf((float)W));
+    if (r == "mlp.shared.sg") return s.shared_gate && fmat(L.router + (size_t)s.experts * W, 1, W, 1.0f / sqrtf((float)W));
     int e = -1, n2 = 0;
     std::string part;
     int off = -1, width = 0;
@@ -621,11 +688,11 @@ static bool ll_place(L3Model* m, const std::string& name, LLPlace* p) {
     if (r.compare(0, 4, "mlp.") == 0) return false;
   } else if (s.ff_kind == L3_FF_RELU2) {
     if (r == "mlp.up") return s.ff > 0 && mat(L.w13, s.ff, W);
-    if (r == "mlp.down") return s.ff > 0 && mat(L.w2, W, s.ff);
+    if (r == "mlp.down") { const bool ok = s.ff > 0 && mat(L.w2, W, s.ff); if (L.h_base) p->ld = L.ctx_ld; return ok; }
   } else {
     if (r == "mlp.gate") return s.ff > 0 && mat(L.w13, s.ff, W, 0, 2);
     if (r == "mlp.up") return s.ff > 0 && mat(L.w13, s.ff, W, 1, 2);
-    if (r == "mlp.down") return s.ff > 0 && mat(L.w2, W, s.ff);
+    if (r == "mlp.down") { const bool ok = s.ff > 0 && mat(L.w2, W, s.ff); if (L.h_base) p->ld = L.ctx_ld; return ok; }
   }
   if (r == "side.gate") return sd && mat(L.side_gate, sd, W);
   if (r == "side.proj") return sd && mat(L.side_proj, W, sd);
@@ -722,6 +789,7 @@ static std::vector<std::string> ll_expected(const L3Model* m) {
   if (ll->loop_step) v.push_back("loop.step");
   if (ll->loop_in) v.push_back("loop.in");
   if (ll->embed_norm) v.push_back("embed.norm");
+  if (ll->final_b) v.insert(v.end(), {"final.norm.b", "final.norm.alpha"});
   for (int i = 0; i < ll->cfg.n_layers; ++i) {
     const L3LayerSpec& s = ll->layers[i].spec;
     const std::string p = "l" + std::to_string(i) + ".";
@@ -746,6 +814,8 @@ static std::vector<std::string> ll_expected(const L3Model* m) {
     else names.insert(names.end(), {"mix.q", "mix.k", "mix.v", "mix.b", "mix.a1", "mix.a2", "mix.g1", "mix.g2", "mix.norm",
                                     "mix.A_log", "mix.dt_bias", "mix.q.conv", "mix.k.conv", "mix.v.conv"});
     const LLLayer& Lx = ll->layers[i];
+    if (Lx.norm_b[0]) names.insert(names.end(), {"norm1.b", "norm1.alpha"});
+    if (Lx.norm_b[1]) names.insert(names.end(), {"norm2.b", "norm2.alpha"});
     if (Lx.ls1) names.push_back("ls1");
     if (Lx.ls2) names.push_back("ls2");
     if (ll->cfg.streams > 0) {
@@ -757,6 +827,8 @@ static std::vector<std::string> ll_expected(const L3Model* m) {
     if (Lx.dwa) names.push_back("dwa");
     if (Lx.ff_total) {
       names.push_back("mlp.router");
+      if (Lx.norm2) names.push_back("norm2");
+      if (s.shared_gate) names.push_back("mlp.shared.sg");
       for (int e = 0; e <= s.experts; ++e) {
         if (e == s.experts && s.shared_ff == 0) break;
         const std::string ep = p + (e == s.experts ? std::string("mlp.shared.") : "mlp.e" + std::to_string(e) + ".");
@@ -849,6 +921,10 @@ static int ll_alloc_unit_state(L3Model* m, const L3LayerSpec& s, LLState& St) {
     return L3_OK;
   }
   CK(m, cudaMalloc((void**)&St.S, (size_t)m->maxB * s.heads * s.dim * s.vdim * 4));
+  if (s.mixer == L3_MIX_MLSTM) {
+    CK(m, cudaMalloc((void**)&St.n, (size_t)m->maxB * s.heads * s.dim * 4));
+    CK(m, cudaMalloc((void**)&St.m, (size_t)m->maxB * s.heads * 4));
+  }
   const int C = unit_conv_channels(s);
   if (C) CK(m, cudaMalloc((void**)&St.conv_tail, std::max<size_t>(16, (size_t)m->maxB * C * (s.conv_taps - 1) * 4)));
   return L3_OK;
@@ -865,6 +941,10 @@ static int ll_reset_unit_state(L3Model* m, const L3LayerSpec& s, LLState& St, in
   }
   const size_t per = (size_t)s.heads * s.dim * s.vdim;
   CK(m, cudaMemsetAsync(St.S + slot0 * per, 0, n * per * 4, m->stream));
+  if (St.n) {  // the running maximum starts at zero, too
+    CK(m, cudaMemsetAsync(St.n + (size_t)slot0 * s.heads * s.dim, 0, (size_t)n * s.heads * s.dim * 4, m->stream));
+    CK(m, cudaMemsetAsync(St.m + (size_t)slot0 * s.heads, 0, (size_t)n * s.heads * 4, m->stream));
+  }
   const size_t pc = (size_t)unit_conv_channels(s) * (s.conv_taps - 1);
   if (pc) CK(m, cudaMemsetAsync(St.conv_tail + slot0 * pc, 0, n * pc * 4, m->stream));
   return L3_OK;
@@ -926,6 +1006,8 @@ int ll_finalize(L3Model* m) {
       } else if (s.mixer == L3_MIX_SSD) {
         max_rq = std::max(max_rq, G * DK); max_rk = std::max(max_rk, G * DK); max_rv = std::max(max_rv, H * DV);
         max_rg = std::max(max_rg, 2 * H); max_xs = std::max(max_xs, H * DV);  // decays and their logarithms
+      } else if (s.mixer == L3_MIX_MLSTM) {
+        max_rg = std::max(max_rg, 5 * H);  // decays, their logarithms, key factors, floors, normalisers
       } else if (s.mixer == L3_MIX_GLA) {
         max_rq = std::max(max_rq, H * DK); max_rg = std::max(max_rg, H * DK); max_aux = std::max(max_aux, H * DK);
       }
@@ -970,7 +1052,9 @@ int ll_finalize(L3Model* m) {
   CK(m, cudaMalloc((void**)&ll->x2, (size_t)8 * W * 4));  // second residual buffer of the fused post-norm step (<= 8 rows)
   CK(m, cudaMalloc((void**)&m->xn, ct * W * 4));  // sublayer output before its norm
   CK(m, cudaMalloc((void**)&m->q, ct * max_rq * 4));
-  CK(m, cudaMalloc((void**)&m->ctx, ct * ll->max_o * 4));
+  ll->max_ctx = std::max(ll->max_ctx, ll->max_o);
+  CK(m, cudaMalloc((void**)&m->ctx, ct * ll->max_ctx * 4));
+  CK(m, cudaMemsetAsync(m->ctx, 0, ct * ll->max_ctx * 4, m->stream));  // columns no layer writes meet weights of zero: finite
   CK(m, cudaMalloc((void**)&m->h, std::max(ct * std::max(1, ll->max_ff), (size_t)8 * max_hid) * 4));
   CK(m, cudaMalloc((void**)&m->xlast, (size_t)m->maxB * W * 4));
   CK(m, cudaMalloc((void**)&m->logits, (size_t)m->maxB * m->VS * 4));
@@ -992,16 +1076,22 @@ int ll_finalize(L3Model* m) {
     CK(m, cudaMalloc((void**)&ll->y1, ct * W * 4));
   }
   // the logit scale rides on the final norm's weight
-  if (ll->cfg.logit_scale != 0.f && ll->cfg.logit_scale != 1.f) LAUNCH(m, launch_scale_add_rows(m->norm_final, ll->cfg.logit_scale, nullptr, 1, W, m->stream));
+  if (ll->cfg.logit_scale != 0.f && ll->cfg.logit_scale != 1.f) {
+    LAUNCH(m, launch_scale_add_rows(m->norm_final, ll->cfg.logit_scale, nullptr, 1, W, m->stream));
+    if (ll->final_b) LAUNCH(m, launch_scale_add_rows(ll->final_b, ll->cfg.logit_scale, nullptr, 1, W, m->stream));
+  }
+  for (auto& L0 : ll->layers)  // an output bias goes with its mixer's scale
+    for (LLLayer* U = &L0; U; U = U->pair)
+      if (U->o_bias) LAUNCH(m, launch_scale_add_rows(U->o_bias, U->mix_scale, nullptr, 1, W, m->stream));
   if (max_xs) CK(m, cudaMalloc((void**)&ll->xs, ct * max_xs * 4));
   if (win_part) {
     CK(m, cudaMalloc((void**)&ll->win_part_o, win_part * 4));
     CK(m, cudaMalloc((void**)&ll->win_part_ml, win_part * 4));
   }
-  if (ll->cfg.loop_in) {
-    CK(m, cudaMalloc((void**)&ll->x0, ct * W * 4));
-    CK(m, cudaMalloc((void**)&ll->cat, ct * 2 * W * 4));
-  }
+  if (ll->cfg.loop_in || ll->cfg.loop_x0) CK(m, cudaMalloc((void**)&ll->x0, ct * W * 4));
+  if (ll->cfg.loop_in) CK(m, cudaMalloc((void**)&ll->cat, ct * 2 * W * 4));
+  if (ll->cfg.dual_norm) CK(m, cudaMalloc((void**)&ll->hf, ct * W * 4));
+  if (max_gu) CK(m, cudaMalloc((void**)&ll->moe_gu, ct * max_gu * 4));
   if (ll->cfg.parallel) {
     if (ll->cfg.depth_avg) CK(m, cudaMalloc((void**)&ll->Xs, (size_t)(ll->cfg.n_layers + 1) * ct * W * 4));
     if (ll->cfg.canon_taps > 0) {
@@ -1010,7 +1100,6 @@ int ll_finalize(L3Model* m) {
     }
     CK(m, cudaMalloc((void**)&ll->y1, ct * W * 4));
     CK(m, cudaMalloc((void**)&ll->y2, ct * W * 4));
-    if (max_gu) CK(m, cudaMalloc((void**)&ll->moe_gu, ct * max_gu * 4));
     size_t part = 0;
     for (auto& L : ll->layers)
       if (L.spec.mixer == L3_MIX_DIFF) part = std::max(part, diff_attn_part_floats(m->maxB * 8, L.spec.heads, L.spec.vdim));
@@ -1028,9 +1117,9 @@ int ll_finalize(L3Model* m) {
   for (const LLLayer& L0 : ll->layers)
     for (const LLLayer* U = &L0; U; U = U->pair) {
       const L3LayerSpec& s = U->spec;
-      const bool chunked = s.mixer == L3_MIX_DECAY_LINEAR || (units && s.mixer == L3_MIX_SSD);
+      const bool chunked = s.mixer == L3_MIX_DECAY_LINEAR || (units && (s.mixer == L3_MIX_SSD || s.mixer == L3_MIX_MLSTM));
       if (chunked && recur_chunk_shape(s.dim, s.vdim) && ct >= 128)
-        ll->chunk_ws_floats = std::max(ll->chunk_ws_floats, (ct / 64 + m->maxB) * ((size_t)s.heads * s.dim * s.vdim + s.heads));
+        ll->chunk_ws_floats = std::max(ll->chunk_ws_floats, (ct / 64 + m->maxB) * ((size_t)s.heads * s.dim * s.vdim + s.heads + (s.mixer == L3_MIX_MLSTM ? s.heads * s.dim : 0)) + 8);
     }
   if (ll->chunk_ws_floats) CK(m, cudaMalloc((void**)&ll->chunk_ws, ll->chunk_ws_floats * 4));
   // tensor cores: bf16 mode only.  fp32 mode is the exact mode of this family: every product is an fp32 FFMA chain
@@ -1043,7 +1132,8 @@ int ll_finalize(L3Model* m) {
       CK(m, cudaMemsetAsync(m->gemm_cnt, 0, 1024 * sizeof(int), m->stream));
     }
     CK(m, cudaMalloc(&m->xn16, ct * W * 2));  // mirror of the residual stream
-    CK(m, cudaMalloc(&m->ctx16, ct * ll->max_o * 2));
+    CK(m, cudaMalloc(&m->ctx16, ct * ll->max_ctx * 2));
+    CK(m, cudaMemsetAsync(m->ctx16, 0, ct * ll->max_ctx * 2, m->stream));
     CK(m, cudaMalloc(&m->h16, ct * std::max(1, ll->max_ff) * 2));
     CK(m, cudaMalloc(&m->xlast16, (size_t)m->maxB * W * 2));
     CK(m, cudaMalloc(&ll->sg16, ct * std::max(1, sd) * 2));
@@ -1103,25 +1193,26 @@ void ll_destroy(L3Model* m) {
   fr(ll->side_embed); fr(ll->one); fr(ll->X);
   if (m->lm_head == m->embed) m->lm_head = nullptr;  // a tied output projection has no storage of its own
   for (auto& L : ll->layers) {
-    fr(L.w_in); fr(L.w_o); fr(L.w_a2); fr(L.w_g2); fr(L.w13); fr(L.w2); fr(L.side_gate); fr(L.side_proj);
+    fr(L.w_in); fr(L.w_o); fr(L.w_a2); fr(L.w_g2); fr(L.w13); fr(L.h_base ? nullptr : L.w2); fr(L.side_gate); fr(L.side_proj);
     fr(L.norm1); fr(L.norm2); fr(L.side_norm); fr(L.mix_norm); fr(L.q_norm); fr(L.k_norm); fr(L.conv_w);
     fr(L.A_log); fr(L.dt_bias); fr(L.decay);
     fr(L.w_uq); fr(L.w_ukv); fr(L.inv_freq); fr(L.in_bias); fr(L.shift); fr(L.router); fr(L.correction);
     fr(L.canon1); fr(L.canon2); fr(L.canon1t); fr(L.canon2t); fr(L.ls1); fr(L.ls2); fr(L.dwa); fr(L.lam_vec); fr(L.lambda); fr(L.poly);
-    fr(L.head_vec); fr(L.conv_b); fr(L.skip_d); fr(L.a2_bias);
+    fr(L.head_vec); fr(L.conv_b); fr(L.skip_d); fr(L.a2_bias); fr(L.o_bias);
+    for (int q = 0; q < 2; ++q) { fr(L.norm_b[q]); fr(L.norm_alpha[q]); }
     for (int q = 0; q < 2 && ll->cfg.streams > 0; ++q) { fr(L.hc_in[q]); fr(L.hc_out[q]); fr(L.hc_mix[q]); }
     if (LLLayer* R = L.pair) {  // its w_in / w_o are views of the first mixer's
       fr(R->w_a2); fr(R->w_g2); fr(R->mix_norm); fr(R->conv_w); fr(R->A_log); fr(R->dt_bias); fr(R->inv_freq);
-      fr(R->head_vec); fr(R->conv_b); fr(R->skip_d); fr(R->a2_bias);
+      fr(R->head_vec); fr(R->conv_b); fr(R->skip_d); fr(R->a2_bias); fr(R->o_bias); fr(R->q_norm); fr(R->k_norm); fr(R->in_bias);
       delete R;
       L.pair = nullptr;
     }
   }
   for (auto& St : ll->state) {
-    fr(St.ck); fr(St.cv); fr(St.S); fr(St.conv_tail); fr(St.lat_shared ? nullptr : St.lat); fr(St.hprev);
-    if (LLState* P = St.pair) { fr(P->ck); fr(P->cv); fr(P->S); fr(P->conv_tail); delete P; St.pair = nullptr; }
+    fr(St.ck); fr(St.cv); fr(St.S); fr(St.n); fr(St.m); fr(St.conv_tail); fr(St.lat_shared ? nullptr : St.lat); fr(St.hprev);
+    if (LLState* P = St.pair) { fr(P->ck); fr(P->cv); fr(P->S); fr(P->n); fr(P->m); fr(P->conv_tail); delete P; St.pair = nullptr; }
   }
-  fr(ll->loop_in); fr(ll->embed_norm); fr(ll->x0); fr(ll->cat); fr(ll->cat16); fr(ll->win_part_o); fr(ll->win_part_ml); fr(ll->xs);
+  fr(ll->loop_in); fr(ll->embed_norm); fr(ll->final_b); fr(ll->final_alpha); fr(ll->x0); fr(ll->cat); fr(ll->cat16); fr(ll->win_part_o); fr(ll->win_part_ml); fr(ll->xs);
   fr(ll->diff_part_o); fr(ll->diff_part_ml);
   fr(ll->Xs); fr(ll->hn); fr(ll->hf); fr(ll->hf16); fr(ll->y1); fr(ll->y2); fr(ll->moe_gu);
   fr(ll->lat_q16); fr(ll->lat_exp); fr(ll->lat_part_o); fr(ll->lat_part_ml);
@@ -1237,7 +1328,11 @@ extern "C" int l3_read_state(L3Model* m, int layer, int slot, float* S_out, floa
   }
   const size_t per = (size_t)s.heads * s.dim * s.vdim;
   if (S_out) CK(m, cudaMemcpy(S_out, St.S + slot * per, per * 4, cudaMemcpyDeviceToHost));
-  if (conv_out) {
+  if (conv_out && s.mixer == L3_MIX_MLSTM) {
+    const size_t pn = (size_t)s.heads * s.dim;
+    CK(m, cudaMemcpy(conv_out, St.n + slot * pn, pn * 4, cudaMemcpyDeviceToHost));
+    CK(m, cudaMemcpy(conv_out + pn, St.m + (size_t)slot * s.heads, s.heads * 4, cudaMemcpyDeviceToHost));
+  } else if (conv_out) {
     REQUIRE(m, unit_conv_channels(s) > 0, "layer run %d has no convolution", layer);
     const size_t pc = (size_t)unit_conv_channels(s) * (s.conv_taps - 1);
     if (pc) CK(m, cudaMemcpy(conv_out, St.conv_tail + slot * pc, pc * 4, cudaMemcpyDeviceToHost));
@@ -1348,19 +1443,22 @@ static int ll_mix_unit(L3Model* m, LLLayer& Ly, LLState& St, const float* pin, i
   const int ntok = B * L, H = s.heads, G = s.kv_heads, DK = s.dim, DV = s.vdim, O = H * DV;
   const float eps = ll->cfg.norm_eps;
   int* d_pos = m->d_scal + 0;
-  float* ctx = m->ctx + Ly.ctx_base;
+  // fp32 rows only for a projection that reads them
+  float* ctx = m->ctx16 && ll_takes_mirror(m, ntok, m->D, Ly.ctx_ld) ? nullptr : m->ctx + Ly.ctx_base;
   bf16* ctx16 = m->ctx16 ? (bf16*)m->ctx16 + Ly.ctx_base : nullptr;
   int rc;
   if (s.mixer == L3_MIX_WINDOW) {
     WinPrepArgs pa{};
     pa.proj = pin; pa.ld = ld; pa.q_off = Ly.off_q; pa.k_off = Ly.off_k; pa.v_off = Ly.off_v; pa.inv_freq = Ly.inv_freq;
     pa.rot_dims = s.rot_dims; pa.rot_layout = s.rot_layout; pa.unit_norm = s.qk_unit; pa.eps = eps;
+    pa.bias = Ly.in_bias; pa.wq = Ly.q_norm; pa.wk = Ly.k_norm;
     pa.q_out = m->q; pa.cache_k = St.ck; pa.cache_v = St.cv; pa.pos_ptr = d_pos;
     pa.L = L; pa.H = H; pa.G = G; pa.DK = DK; pa.DV = DV; pa.M = m->M;
     LAUNCH(m, launch_win_prep(pa, ntok, m->bf16, m->stream));
     WinAttnArgs at{};
     at.q = m->q; at.cache_k = St.ck; at.cache_v = St.cv; at.out = ctx; at.out16 = ctx16; at.ld_out = Ly.ctx_ld; at.out_scale = Ly.mix_scale;
     at.head_vec = Ly.head_vec; at.pos_ptr = d_pos; at.scale = s.scale; at.kind = s.attn_kind; at.window = s.window; at.keep_first = s.keep_first;
+    at.chunked = s.chunked; at.gate = s.head_gate ? pin + Ly.off_g : nullptr; at.ld_gate = ld;
     at.B = B; at.L = L; at.H = H; at.G = G; at.DK = DK; at.DV = DV; at.M = m->M;
     at.nsplit = win_attn_splits(B, L, H, G, s.window, s.keep_first, m->M, 32);
     at.part_o = ll->win_part_o; at.part_ml = ll->win_part_ml;
@@ -1372,7 +1470,28 @@ static int ll_mix_unit(L3Model* m, LLLayer& Ly, LLState& St, const float* pin, i
   mo.o = ll->o; mo.n = O; mo.DV = DV; mo.eps = eps; mo.out_scale = Ly.mix_scale; mo.out = ctx; mo.out16 = ctx16; mo.ld_out = Ly.ctx_ld;
   RecurArgs ra{};
   ra.state = St.S; ra.out = ll->o; ra.B = B; ra.L = L; ra.H = H; ra.DK = DK; ra.DV = DV;
-  if (s.mixer == L3_MIX_SSD) {
+  if (s.mixer == L3_MIX_MLSTM) {
+    const float q_mul = 1.0f / sqrtf((float)DK);
+    if (L == 1) {  // decode: the whole mixer between its projections
+      MlstmStepArgs sa{};
+      sa.proj = pin; sa.ld = ld; sa.q_off = Ly.off_q; sa.k_off = Ly.off_k; sa.v_off = Ly.off_v; sa.g_off = Ly.off_g; sa.i_off = Ly.off_b; sa.f_off = Ly.off_b + H;
+      sa.bias = Ly.in_bias; sa.cap = s.gate_cap; sa.q_mul = q_mul; sa.eps = eps; sa.out_scale = Ly.mix_scale; sa.w = Ly.mix_norm;
+      sa.S = St.S; sa.n = St.n; sa.m = St.m; sa.out = ctx; sa.out16 = ctx16; sa.ld_out = Ly.ctx_ld; sa.H = H; sa.DK = DK; sa.DV = DV;
+      LAUNCH(m, launch_mlstm_step(sa, B, m->stream));
+      return L3_OK;
+    }
+    MlstmGateArgs ga{};
+    const size_t nh = (size_t)ntok * H;
+    ga.proj = pin; ga.ld = ld; ga.i_off = Ly.off_b; ga.f_off = Ly.off_b + H; ga.bias = Ly.in_bias; ga.cap = s.gate_cap; ga.m = St.m;
+    ga.decay = ll->rg; ga.log_decay = ll->rg + nh; ga.k_scale = ll->rg + 2 * nh; ga.floor = ll->rg + 3 * nh; ga.L = L; ga.H = H;
+    LAUNCH(m, launch_mlstm_gates(ga, B, m->stream));
+    ra.mode = 2; ra.q = pin + Ly.off_q; ra.k = pin + Ly.off_k; ra.v = pin + Ly.off_v; ra.ld_q = ra.ld_k = ra.ld_v = ld; ra.rep = 1;
+    ra.g = ga.decay; ra.g_head = 1; ra.log_g = ga.log_decay; ra.k_scale = ga.k_scale; ra.q_mul = q_mul; ra.n_state = St.n; ra.nq = ll->rg + 4 * nh;
+    ra.ws = ll->chunk_ws; ra.ws_floats = ll->chunk_ws_floats;
+    LAUNCH(m, launch_recur(ra, m->stream));
+    mo.nq = ra.nq; mo.floor = ga.floor; mo.gate = pin + Ly.off_g; mo.ld_gate = ld; mo.gate_act = 0; mo.pre_gate = 0;
+    mo.w = Ly.mix_norm; mo.wlen = O; mo.group = DV;
+  } else if (s.mixer == L3_MIX_SSD) {
     const int gn = G * DK;
     SsdPrepArgs pa{};
     pa.proj = pin; pa.ld = ld; pa.xbc_off = Ly.off_q; pa.dt_off = Ly.off_b; pa.conv_w = Ly.conv_w; pa.conv_b = Ly.conv_b;
@@ -1464,7 +1583,9 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
   int rc;
   ll->xcur = m->x;
   const float embed_mul = ll->cfg.embed_scale != 0.f ? ll->cfg.embed_scale : 1.f;
-  if (embed_mul != 1.f && !ll->streams) LAUNCH(m, launch_scale_add_rows(m->x, embed_mul, nullptr, ntok, W, m->stream));
+  const bool dual = ll->cfg.dual_norm, tanh_n = ll->cfg.norm_tanh;
+  const bool fold_mul = tanh_n && !ll->loop_in;  // the first layer's entry launch scales the embedding rows
+  if (embed_mul != 1.f && !ll->streams && !fold_mul) LAUNCH(m, launch_scale_add_rows(m->x, embed_mul, nullptr, ntok, W, m->stream));
   StreamArgs sa{};  // the streams' side of the step: sa.y is the sublayer result they have not taken yet
   sa.x0 = m->x; sa.x_mul = embed_mul; sa.X = ll->X; sa.eps = eps; sa.S = ll->streams; sa.D = W;
   // the normed input of sublayer q into hn / hn16 (or, for few rows of a streamed stack, its un-normed form: *in_norm)
@@ -1497,7 +1618,10 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
   };
   const int ng = std::max(1, ll->cfg.norm_groups);
   if (ll->embed_norm) LAUNCH(m, launch_rmsnorm_rows(m->x, ll->embed_norm, eps, ntok, W, 1, 0, nullptr, m->x, nullptr, m->stream, ng));  // in place, row by row
-  if (ll->x0) CK(m, cudaMemcpyAsync(ll->x0, m->x, (size_t)ntok * W * 4, cudaMemcpyDeviceToDevice, m->stream));  // the embedding output
+  if (ll->x0 && !fold_mul) CK(m, cudaMemcpyAsync(ll->x0, m->x, (size_t)ntok * W * 4, cudaMemcpyDeviceToDevice, m->stream));  // the embedding output
+  // the feed-forward's input: rows of its own where both sublayers read one stream
+  float* h2 = dual ? ll->hf : hn;
+  bf16* h2_16 = dual ? (bf16*)ll->hf16 : hn16;
   for (int ri = 0; ri < (int)ll->runs.size(); ++ri) {
     LLLayer& Ly = ll->layers[ll->runs[ri].layer];
     LLState& St = ll->state[ri];
@@ -1506,10 +1630,49 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
     if (ll->runs[ri].pass >= 0 && ll->loop_in) {  // a pass starts: x <- W_in [x ; x0]
       LAUNCH(m, launch_concat_rows(m->x, ll->x0, ntok, W, ll->cat, (bf16*)ll->cat16, m->stream));
       if ((rc = ll_linear(m, ll->loop_in, ll->cat, ll->cat16, 0, ntok, W, 2 * W, EPI_STORE, store_to(m->x, nullptr, W))) != L3_OK) return rc;
-    } else if (ll->runs[ri].pass >= 0)
-      LAUNCH(m, launch_scale_add_rows(m->x, 1.0f, ll->loop_step + (size_t)ll->runs[ri].pass * W, ntok, W, m->stream));
-    const float* in_norm;
-    if ((rc = sublayer_in(Ly, 0, Ly.norm1, Ly.shift, St.hprev, Ly.n_in, &in_norm)) != L3_OK) return rc;
+    }
+    const int pass = ll->runs[ri].pass;
+    const float* step = pass >= 0 && ll->loop_step ? ll->loop_step + (size_t)pass * W : nullptr;
+    const float* again = pass > 0 && ll->cfg.loop_x0 ? ll->x0 : nullptr;
+    const float* in_norm = nullptr;
+    const bool has_ff = s.ff > 0;
+    // element-wise norms into the sublayers' inputs, together with everything that joins the stream here
+    TanhNormArgs na{};
+    na.x = m->x; na.mul = 1.f; na.D = W; na.src_mul = 1;
+    auto tanh_norm = [&](int q, float* out, bf16* out16, int n_out, bool keep32) {
+      const int k = na.n_norm++;
+      na.w[k] = q ? Ly.norm2 : Ly.norm1; na.b[k] = Ly.norm_b[q]; na.alpha[k] = Ly.norm_alpha[q];
+      na.out16[k] = out16;
+      na.out[k] = !keep32 && out16 && ll_takes_mirror(m, ntok, n_out, W) ? nullptr : out;
+    };
+    const int n_up = s.ff_kind == L3_FF_RELU2 ? s.ff : 2 * s.ff;
+    if (tanh_n) {
+      if (ri == 0 && fold_mul) { na.mul = embed_mul; na.x0_out = ll->x0; }
+      na.vec = step; na.rows = again; na.post = Ly.o_bias;
+      na.write = na.mul != 1.f || step || again || Ly.o_bias;
+      tanh_norm(0, hn, hn16, Ly.n_in, false);
+      if (dual && has_ff) tanh_norm(1, h2, h2_16, n_up, s.experts > 0);
+      LAUNCH(m, launch_tanh_norms(na, ntok, m->stream));
+    } else {
+      if (again) {
+        na.vec = step; na.rows = again; na.write = 1;
+        LAUNCH(m, launch_tanh_norms(na, ntok, m->stream));
+      } else if (step) LAUNCH(m, launch_scale_add_rows(m->x, 1.0f, step, ntok, W, m->stream));
+      if ((rc = sublayer_in(Ly, 0, Ly.norm1, Ly.shift, St.hprev, Ly.n_in, &in_norm)) != L3_OK) return rc;
+      if (dual && has_ff) LAUNCH(m, launch_prenorm_shift(m->x, Ly.norm2, eps, nullptr, nullptr, B, L, W, h2, h2_16, m->stream, ng));
+      if (Ly.o_bias) LAUNCH(m, launch_scale_add_rows(m->x, 1.0f, Ly.o_bias, ntok, W, m->stream));
+    }
+    if (Ly.pair && Ly.pair->o_bias) LAUNCH(m, launch_scale_add_rows(m->x, 1.0f, Ly.pair->o_bias, ntok, W, m->stream));
+    // ahead of a feed-forward that reads the stream the mixer has left
+    auto ff_in = [&](bool keep32) -> int {
+      if (dual) return L3_OK;
+      if (!tanh_n) { LAUNCH(m, launch_prenorm_shift(m->x, Ly.norm2, eps, nullptr, nullptr, B, L, W, hn, hn16, m->stream, ng)); return L3_OK; }
+      na = TanhNormArgs{};
+      na.x = m->x; na.mul = 1.f; na.D = W; na.src_mul = 1;
+      tanh_norm(1, hn, hn16, n_up, keep32);
+      LAUNCH(m, launch_tanh_norms(na, ntok, m->stream));
+      return L3_OK;
+    };
     // every projection of the mixer's input in one GEMM
     if ((rc = ll_linear(m, Ly.w_in, hn, hn16, 0, ntok, Ly.n_in, W, EPI_STORE, store_to(ll->pin, nullptr, Ly.n_in), nullptr, in_norm)) != L3_OK) return rc;
     int n_ctx = H * DV;
@@ -1561,33 +1724,63 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
       set_err(m, "mixer %d is not built for pre-norm layers", s.mixer);
       return L3_EINVAL;
     }
+    auto glu_epi = [&](EpiArgs& e) {
+      if (s.ff_kind == L3_FF_RELU2) e.unary = UNARY_RELU2;
+      else if (s.ff_kind == L3_FF_CLAMP) { e.act = GLU_CLAMP; e.act_limit = s.ff_limit; e.act_slope = s.ff_slope; }
+      else e.act = ll->cfg.glu_act;
+    };
+    if (Ly.h_base) {  // the hidden values join the mixer's columns: one output projection for both sublayers
+      EpiArgs e = store_to(m->ctx16 && ll_takes_mirror(m, ntok, W, n_ctx) ? nullptr : m->ctx + Ly.h_base,
+                           m->ctx16 ? (bf16*)m->ctx16 + Ly.h_base : nullptr, n_ctx);
+      glu_epi(e);
+      if ((rc = ll_linear(m, Ly.w13, h2, h2_16, 0, ntok, n_up, W, s.ff_kind == L3_FF_RELU2 ? EPI_STORE : EPI_SWIGLU, e)) != L3_OK) return rc;
+    }
     if ((rc = ll_linear(m, Ly.w_o, m->ctx, m->ctx16, 0, ntok, W, n_ctx, out_epi, out_e)) != L3_OK) return rc;
     sublayer_out(Ly, 0);
-    if (s.experts > 0) {
+    if (Ly.ff_total) {  // gated experts, weights on their outputs, a shared expert
+      const int E = s.experts, ff = s.ff, F = Ly.ff_total;
+      if ((rc = ff_in(true)) != L3_OK) return rc;
+      const bool few = ntok <= 8;
+      MoeRouteArgs ra{};
+      ra.h = h2; ra.router = Ly.router; ra.D = W; ra.E = E; ra.top = s.top; ra.groups = 1; ra.keep = 1; ra.kind = 2; ra.scale = 1.0f; ra.shared_gate = s.shared_gate;
+      ra.sel = ll->moe_sel; ra.w = ll->moe_w; ra.dense = few ? nullptr : ll->moe_dense; ra.idw = ll->moe_idw;
+      LAUNCH(m, launch_moe_route(ra, ntok, m->stream));
+      const float* sw = s.shared_gate ? ll->moe_idw : nullptr;
+      if (few) {
+        LAUNCH(m, launch_moe_glu_rows(h2, Ly.w13, Ly.w2, m->bf16, ll->moe_sel, ll->moe_w, sw, true, ntok, W, E, ff, s.shared_ff, s.top, m->h, m->x, true, m->stream));
+        m->launch_acc += 1;
+      } else {
+        if ((rc = ll_linear(m, Ly.w13, h2, h2_16, 0, ntok, 2 * F, W, EPI_STORE, store_to(ll->moe_gu, nullptr, 2 * F))) != L3_OK) return rc;
+        LAUNCH(m, launch_moe_glu_act(ll->moe_gu, ll->moe_dense, sw, true, ntok, E, ff, s.shared_ff, m->h16 && ll_takes_mirror(m, ntok, W, F) ? nullptr : m->h,
+                                     (bf16*)m->h16, m->stream));
+        if ((rc = ll_linear(m, Ly.w2, m->h, m->h16, 0, ntok, W, F, EPI_RESID, resid_into(m->x, W))) != L3_OK) return rc;
+      }
+    } else if (s.experts > 0) {
       const int E = s.experts, ff = s.ff;
-      LAUNCH(m, launch_prenorm_shift(m->x, Ly.norm2, eps, nullptr, nullptr, B, L, W, hn, hn16, m->stream, ng));
+      if ((rc = ff_in(true)) != L3_OK) return rc;
       const bool few = ntok <= 8;  // few rows read only their chosen experts' weights; many share one GEMM over all experts
       MoeRouteArgs ra{};
-      ra.h = hn; ra.router = Ly.router; ra.correction = Ly.correction; ra.D = W; ra.E = E; ra.I = s.identity; ra.top = s.top;
+      ra.h = h2; ra.router = Ly.router; ra.correction = Ly.correction; ra.D = W; ra.E = E; ra.I = s.identity; ra.top = s.top;
       ra.groups = s.groups; ra.keep = s.groups_keep; ra.scale = s.router_scale;
       ra.sel = ll->moe_sel; ra.w = ll->moe_w; ra.dense = few ? nullptr : ll->moe_dense; ra.idw = ll->moe_idw;
       LAUNCH(m, launch_moe_route(ra, ntok, m->stream));
       if (few) {
-        LAUNCH(m, launch_moe_rows(hn, Ly.w13, Ly.w2, m->bf16, ll->moe_sel, ll->moe_w, ll->moe_idw, ntok, W, E, ff, s.top, m->h, m->x, m->stream));
+        LAUNCH(m, launch_moe_rows(h2, Ly.w13, Ly.w2, m->bf16, ll->moe_sel, ll->moe_w, ll->moe_idw, ntok, W, E, ff, s.top, m->h, m->x, m->stream));
         m->launch_acc += 1;
       } else {
-        if ((rc = ll_linear(m, Ly.w13, hn, hn16, 0, ntok, E * ff, W, EPI_STORE, store_to(m->h, nullptr, E * ff))) != L3_OK) return rc;
+        if ((rc = ll_linear(m, Ly.w13, h2, h2_16, 0, ntok, E * ff, W, EPI_STORE, store_to(m->h, nullptr, E * ff))) != L3_OK) return rc;
         LAUNCH(m, launch_moe_act_mask(m->h, ll->moe_dense, ntok, E, ff, (bf16*)m->h16, m->stream));
         if ((rc = ll_linear(m, Ly.w2, m->h, m->h16, 0, ntok, W, E * ff, EPI_RESID, resid_into(m->x, W))) != L3_OK) return rc;
-        if (s.identity > 0) LAUNCH(m, launch_moe_identity(m->x, hn, ll->moe_idw, ntok, W, m->stream));
+        if (s.identity > 0) LAUNCH(m, launch_moe_identity(m->x, h2, ll->moe_idw, ntok, W, m->stream));
       }
-    } else if (s.ff > 0) {
+    } else if (s.ff > 0 && !Ly.h_base) {
       const bool glu = s.ff_kind != L3_FF_RELU2;
-      const int n_up = glu ? 2 * s.ff : s.ff;
-      if ((rc = sublayer_in(Ly, 1, Ly.norm2, nullptr, nullptr, n_up, &in_norm)) != L3_OK) return rc;
+      in_norm = nullptr;
+      if (dual || tanh_n) { if ((rc = ff_in(false)) != L3_OK) return rc; }
+      else if ((rc = sublayer_in(Ly, 1, Ly.norm2, nullptr, nullptr, n_up, &in_norm)) != L3_OK) return rc;
       EpiArgs e = store_to(m->h16 && ll_takes_mirror(m, ntok, W, s.ff) ? nullptr : m->h, m->h16, s.ff);
-      if (glu) e.act = ll->cfg.glu_act; else e.unary = UNARY_RELU2;
-      if ((rc = ll_linear(m, Ly.w13, hn, hn16, 0, ntok, n_up, W, glu ? EPI_SWIGLU : EPI_STORE, e, nullptr, in_norm)) != L3_OK) return rc;
+      glu_epi(e);
+      if ((rc = ll_linear(m, Ly.w13, h2, h2_16, 0, ntok, n_up, W, glu ? EPI_SWIGLU : EPI_STORE, e, nullptr, in_norm)) != L3_OK) return rc;
       if ((rc = ll_linear(m, Ly.w2, m->h, m->h16, 0, ntok, W, s.ff, out_epi, out_e)) != L3_OK) return rc;
       sublayer_out(Ly, 1);
     }
@@ -1658,7 +1851,7 @@ static int ll_enqueue_parallel(L3Model* m, int B, int L, float* d_resid) {
       ra.sel = ll->moe_sel; ra.w = ll->moe_w; ra.dense = few ? nullptr : ll->moe_dense; ra.idw = ll->moe_idw;
       LAUNCH(m, launch_moe_route(ra, ntok, m->stream));
       if (few) {
-        LAUNCH(m, launch_moe_glu_rows(hf, Ly.w13, Ly.w2, m->bf16, ll->moe_sel, ll->moe_w, ntok, W, E, ff, s.shared_ff, s.top, m->h, ll->y2, m->stream));
+        LAUNCH(m, launch_moe_glu_rows(hf, Ly.w13, Ly.w2, m->bf16, ll->moe_sel, ll->moe_w, nullptr, false, ntok, W, E, ff, s.shared_ff, s.top, m->h, ll->y2, false, m->stream));
         m->launch_acc += 1;
       } else {
         // gate | up of every expert and of the shared one in ONE projection, then the routing weight (zero for experts the
@@ -1672,7 +1865,7 @@ static int ll_enqueue_parallel(L3Model* m, int B, int L, float* d_resid) {
           if ((rc = ll_linear(m, Ly.w13, hf, hf16, 0, ntok, 2 * F, W, EPI_SWIGLU, e)) != L3_OK) return rc;
         } else {
           if ((rc = ll_linear(m, Ly.w13, hf, hf16, 0, ntok, 2 * F, W, EPI_STORE, store_to(ll->moe_gu, nullptr, 2 * F))) != L3_OK) return rc;
-          LAUNCH(m, launch_moe_glu_act(ll->moe_gu, ll->moe_dense, ntok, E, ff, s.shared_ff, m->h, (bf16*)m->h16, m->stream));
+          LAUNCH(m, launch_moe_glu_act(ll->moe_gu, ll->moe_dense, nullptr, false, ntok, E, ff, s.shared_ff, m->h, (bf16*)m->h16, m->stream));
         }
         if ((rc = ll_linear(m, Ly.w2, m->h, m->h16, 0, ntok, W, F, EPI_STORE, store_to(ll->y2, nullptr, W))) != L3_OK) return rc;
       }
@@ -1834,7 +2027,12 @@ int ll_ensure_head_rows(L3Model* m, int n) {
 
 int ll_enqueue_head(L3Model* m, int B, int L, const int32_t* d_rows, int n_rows) {
   const int rows = d_rows ? n_rows : B;
-  if (m->ll->cfg.norm_center)
+  if (m->ll->cfg.norm_tanh) {
+    TanhNormArgs na{};
+    na.x = m->ll->xcur; na.mul = 1.f; na.n_norm = 1; na.w[0] = m->norm_final; na.b[0] = m->ll->final_b; na.alpha[0] = m->ll->final_alpha;
+    na.out[0] = m->xlast; na.out16[0] = (bf16*)m->xlast16; na.D = m->D; na.src_mul = L; na.src_add = L - 1; na.src_rows = d_rows;
+    LAUNCH(m, launch_tanh_norms(na, rows, m->stream));
+  } else if (m->ll->cfg.norm_center)
     LAUNCH(m, launch_layernorm_rows(m->ll->xcur, m->norm_final, m->ll->cfg.norm_eps, 1, rows, m->D, L, L - 1, d_rows, m->xlast, (bf16*)m->xlast16, m->stream));
   else
     LAUNCH(m, launch_rmsnorm_rows(m->ll->xcur, m->norm_final, m->ll->cfg.norm_eps, rows, m->D, L, L - 1, d_rows, m->xlast, (bf16*)m->xlast16, m->stream,

@@ -58,7 +58,14 @@ struct LLLayer {
   // w_in holds in_ld rows, this mixer's segment starts at row / output column in_base - and feed ONE output projection:
   // w_o is [width, ctx_ld], this mixer's columns start at ctx_base.  A single mixer has in_base = ctx_base = 0.
   // The pair's w_in / w_o point into the first mixer's allocations.
+  // window attention with biases: in_bias [columns up to the end of v], o_bias [width] (times mix_scale from finalize on); with a
+  // gate per head: w_in rows at off_g.  mLSTM: w_in = q | k | v | g | input-gate and forget-gate logits (off_b), in_bias [2 heads]
+  float* o_bias = nullptr;
+  float *norm_b[2] = {nullptr, nullptr}, *norm_alpha[2] = {nullptr, nullptr};  // element-wise norms: bias [width], alpha [1]
   LLLayer* pair = nullptr;
+  // > 0: the feed-forward's hidden values are columns [h_base, h_base + ff) of the output projection's input and w2 is the same
+  // columns of w_o: mixer and feed-forward leave through ONE product (dual_norm stacks, dense feed-forward)
+  int h_base = 0;
   int in_base = 0, in_ld = 0, ctx_base = 0, ctx_ld = 0, n_ctx = 0;
   float mix_scale = 1.f;  // multiplier of this mixer's result (applied to its slice of the output projection's input)
 };
@@ -75,6 +82,7 @@ struct LLState {
   // parallel layers with a convolution: conv_tail [maxB, width, taps - 1] the last rows of the layer's normed input
   // window attention: ck [maxB, kv_heads, M, dim], cv [maxB, kv_heads, M, vdim]; state-space mixer: S [maxB, heads, state, vdim],
   // conv_tail [maxB, heads vdim + 2 groups state, taps - 1]; gated linear attention: S
+  float *n = nullptr, *m = nullptr;   // mLSTM, beside S: normalisers [maxB, heads, dim], running maxima [maxB, heads]
   LLState* pair = nullptr;            // state of the layer's second mixer
 };
 
@@ -94,6 +102,7 @@ struct LayerList {
   float* loop_step = nullptr;    // [loop_times, width] fp32
   void* loop_in = nullptr;       // [width, 2 width] of WT: the looped block's entry projection (loop_in)
   float* embed_norm = nullptr;   // [width]
+  float *final_b = nullptr, *final_alpha = nullptr;  // element-wise final norm
   float *x0 = nullptr, *cat = nullptr;  // the embedding output [cap_tok, width]; [x | x0] rows [cap_tok, 2 width]
   void* cat16 = nullptr;
   float *win_part_o = nullptr, *win_part_ml = nullptr;  // split scratch of the window attention
@@ -127,7 +136,7 @@ struct LayerList {
   float *y1 = nullptr, *y2 = nullptr;      // the two sublayers' results [cap_tok, width] (with streams: y1 alone)
   float* moe_gu = nullptr;                 // [cap_tok, 2 ff_total] gate | up of every expert
   float *diff_part_o = nullptr, *diff_part_ml = nullptr;  // split scratch of the differential decode attention
-  int max_in = 0, max_o = 0, max_ff = 0;
+  int max_in = 0, max_o = 0, max_ctx = 0, max_ff = 0;  // max_ctx: columns of an output projection's input
   int head_rows = 0;  // rows the LM head's buffers hold
 };
 

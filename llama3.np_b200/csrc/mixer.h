@@ -70,6 +70,11 @@ struct RecurArgs {
   float* state;           // [maxB, H, DK, DV]
   float* out;             // [B * L, H * DV]
   int B, L, H, rep, DK, DV;
+  // mode 2 with g_head, each may be null / 0:
+  const float* k_scale;   // [B * L, H] multiplies the key of (token, head)
+  float q_mul;            // multiplies the queries (0: 1)
+  float* n_state;         // [maxB, H, DK] a running sum of the keys with the state's own decay (the normaliser of an mLSTM) ...
+  float* nq;              // ... and its product with the query, [B * L, H]
   float* ws;              // mode 0, may be null: room for one state matrix per (sequence, head, chunk of 64 tokens);
   size_t ws_floats;       // with it, prompts of the common shapes run in the chunk-parallel form (recur_chunk.cu)
 };
@@ -271,12 +276,14 @@ struct MoeRouteArgs {
   const float* router;   // [E + I, D] fp32
   const float* correction;
   int D, E, I, top, groups, keep;
-  int kind;              // 0: softmax scores + correction + groups; 1: scores = sigmoid(logit), the top scores win, weight = score
+  int kind;              // 0: softmax scores + correction + groups; 1: scores = sigmoid(logit), the top scores win, weight = score;
+                         // 2: softmax scores, the top scores win, weight = score / (sum of the chosen scores + 1e-20)
+  int shared_gate;       // 1: row E + I of `router` is a shared expert's gate; idw then receives its sigmoid
   float scale;
   int32_t* sel;          // [rows, top] chosen slots, best first
   float* w;              // [rows, top] their weights
   float* dense;          // [rows, E] weight of every expert (0: not chosen); may be null
-  float* idw;            // [rows] summed weight of the chosen identity slots
+  float* idw;            // [rows] summed weight of the chosen identity slots (shared_gate: the shared expert's weight)
 };
 cudaError_t launch_moe_route(const MoeRouteArgs& a, int rows, cudaStream_t s);
 // u[r, c] <- relu(u[r, c])^2 * dense[r, c / ff]  (+ bf16 mirror)
@@ -291,15 +298,16 @@ cudaError_t launch_moe_rows(const float* h, const void* w_up, const void* w_down
 
 // Gated experts whose routing weight multiplies their INPUT (L3_ROUTE_SIGMOID_IN): expert e = down_e(silu(w gate_e h) * (w up_e h)).
 // Weights: w_gu [2 (E ff + sff), D] rows interleaved (gate_j, up_j), expert e at rows [2 e ff, 2 (e + 1) ff), the shared expert
-// (width sff, weight 1, every token; sff 0: none) behind them; w_down [D, E ff + sff].
+// (width sff, weight shared_w[row], or 1 where shared_w is null, every token; sff 0: none) behind them; w_down [D, E ff + sff].
+// w_out: the weight multiplies the expert's OUTPUT instead (L3_ROUTE_SOFTMAX_GLU): w down_e(silu(gate_e h) * (up_e h)).
 // masked-dense path: gu [rows, 2 F] (F = E ff + sff) -> hid [rows, F] = silu(w g) * (w u), zero where the row did not choose the expert
-cudaError_t launch_moe_glu_act(const float* gu, const float* dense, int rows, int E, int ff, int sff, float* hid, bf16* hid16,
-                               cudaStream_t s);
+cudaError_t launch_moe_glu_act(const float* gu, const float* dense, const float* shared_w, bool w_out, int rows, int E, int ff,
+                               int sff, float* hid, bf16* hid16, cudaStream_t s);
 // few rows: only the chosen experts' (and the shared expert's) weights are read.  hid [rows * (top + 1), max(ff, sff)] scratch;
-// y[r] = sum over the row's experts of down_e hid
+// y[r] = (add: y[r] +) sum over the row's experts of down_e hid
 cudaError_t launch_moe_glu_rows(const float* h, const void* w_gu, const void* w_down, bool w_bf16, const int32_t* sel,
-                                const float* w, int rows, int D, int E, int ff, int sff, int top, float* hid, float* y,
-                                cudaStream_t s);
+                                const float* w, const float* shared_w, bool w_out, int rows, int D, int E, int ff, int sff, int top,
+                                float* hid, float* y, bool add, cudaStream_t s);
 
 // ---- sliding-window attention with kept first tokens, sink softmax or sigmoid weights (attn_window.cu)
 struct WinPrepArgs {
@@ -309,6 +317,8 @@ struct WinPrepArgs {
   int rot_dims, rot_layout;  // layout 0: entries (2i, 2i + 1) turn together; 1: entries (i, i + rot_dims / 2)
   int unit_norm;         // 1: q and k over their root mean square per head, after the rotation
   float eps;
+  const float* bias;     // [columns of proj up to the end of v] added to q, k and v (null: none)
+  const float *wq, *wk;  // [DK]: q and k over their root mean square per head, times these, ahead of the rotation (null: none)
   float* q_out;          // [rows, H, DK]
   void* cache_k;         // [maxB, G, M, DK] of KVT
   void* cache_v;         // [maxB, G, M, DV]
@@ -320,15 +330,18 @@ struct WinAttnArgs {
   const float* q;        // [B * L, H, DK]
   const void* cache_k;   // [maxB, G, M, DK]
   const void* cache_v;   // [maxB, G, M, DV]
-  float* out;            // out[r * ld_out + h * DV + d] (+ bf16 mirror, may be null), times out_scale
+  float* out;            // out[r * ld_out + h * DV + d] and its bf16 mirror (either may be null), times out_scale
   bf16* out16;
   int ld_out;
   float out_scale;
   const float* head_vec; // [H]: the sink's logit (softmax; null: no sink) or the bias inside the sigmoid
+  const float* gate;     // head h of row r is multiplied by sigmoid(gate[r * ld_gate + h]) (null: none)
+  int ld_gate;
   const int* pos_ptr;    // token t of the call sits at *pos_ptr + t
   float scale;
-  int kind;              // L3_ATTN_SINK | L3_ATTN_SIGMOID
+  int kind;              // L3_ATTN_SINK | L3_ATTN_SIGMOID | L3_ATTN_SOFTMAX
   int window, keep_first;  // query i sees key j <= i with i - j < window (0: all) or j < keep_first
+  int chunked;           // 1: instead of i - j < window, i / window == j / window (chunks counted from position 0)
   int B, L, H, G, DK, DV, M;
   int nsplit;            // > 1: the key tiles of a query spread over that many CTAs; partials in part_o / part_ml
   float *part_o, *part_ml;
@@ -370,10 +383,58 @@ struct MixOutArgs {
   const float* gate; int ld_gate; int gate_act, pre_gate;
   const float* w; int wlen, group;
   float eps, out_scale;
-  float* out; bf16* out16; int ld_out;
+  float* out; bf16* out16; int ld_out;  // either may be null
+  // mLSTM (null: off): y is divided by max(|nq|, floor) + 1e-6 of its (row, head) first, [rows, n / DV] each; `group` divides DV
+  const float *nq, *floor;
 };
 cudaError_t launch_mix_out(const MixOutArgs& a, int rows, cudaStream_t s);
 // x <- cap * tanh(x / cap), n values
 cudaError_t launch_softcap(float* x, int64_t n, float cap, cudaStream_t s);
 // out[r] = [a[r] | b[r]] (D values each; + bf16 mirror)
 cudaError_t launch_concat_rows(const float* a, const float* b, int rows, int D, float* out, bf16* out16, cudaStream_t s);
+
+// ---- element-wise norms (tanh_norm.cu)
+// The entry of a layer in one pass over the stream:  v = x * mul (+ vec) (+ rows);  x0_out <- x * mul;  per norm q < n_norm
+//   out_q[r] = tanh(alpha_q v) * w_q + b_q   (+ bf16 mirror; either may be null)
+// and, when `write`, x <- v + post.  Any pointer but x may be null; with src_rows / src_mul the rows are gathered (write 0).
+struct TanhNormArgs {
+  float* x;
+  float mul;
+  const float *vec, *rows, *post;  // [D], [rows, D], [D]
+  float* x0_out;
+  int write;
+  int n_norm;
+  const float *w[2], *b[2], *alpha[2];
+  float* out[2];
+  bf16* out16[2];
+  int D, src_mul, src_add;
+  const int32_t* src_rows;
+};
+cudaError_t launch_tanh_norms(const TanhNormArgs& a, int rows, cudaStream_t s);
+
+// ---- matrix memory with exponential gates (mlstm.cu)
+// Gates of every (token, head):  i = cap tanh((z_i + b_i) / cap),  f = logsigmoid(cap tanh((z_f + b_f) / cap)),
+// m_t = max(f + m_(t-1), i); decay = exp(log_decay), log_decay = f + m_(t-1) - m_t; k_scale = exp(i - m_t); floor = exp(-m_t)
+struct MlstmGateArgs {
+  const float* proj;     // [rows, ld]: H input-gate logits at i_off, H forget-gate logits at f_off
+  int ld, i_off, f_off;
+  const float* bias;     // [2 H]: input gates, forget gates
+  float cap;
+  float* m;              // [maxB, H] running maximum, read and written
+  float *decay, *log_decay, *k_scale, *floor;  // [rows, H]
+  int L, H;
+};
+cudaError_t launch_mlstm_gates(const MlstmGateArgs& a, int B, cudaStream_t s);
+// One token per sequence, everything from the projections to the output projection's input in one launch
+struct MlstmStepArgs {
+  const float* proj;     // [B, ld]: q, k (H DK), v, output gate (H DV) at their offsets, gate logits as above
+  int ld, q_off, k_off, v_off, g_off, i_off, f_off;
+  const float* bias;
+  float cap, q_mul, eps, out_scale;
+  const float* w;        // [H * DV]
+  float *S, *n, *m;      // [maxB, H, DK, DV], [maxB, H, DK], [maxB, H]
+  float* out;            // out[b * ld_out + h * DV + d] and its bf16 mirror (either may be null)
+  bf16* out16;
+  int ld_out, H, DK, DV;
+};
+cudaError_t launch_mlstm_step(const MlstmStepArgs& a, int B, cudaStream_t s);

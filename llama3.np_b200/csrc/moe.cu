@@ -16,6 +16,8 @@
 //  * moe_glu_act_kernel    masked-dense path: [rows, 2 F] interleaved (gate, up) of all experts and the shared one ->
 //                          [rows, F] hidden values, zero where the row did not choose the expert
 //  * moe_glu_up_rows / moe_glu_down_rows   few rows: only the chosen experts' and the shared expert's rows are read
+//  Router kind 2 (softmax scores, the largest win, weights = scores over the chosen scores' sum, applied to the expert's
+//  OUTPUT) runs the same gated experts; the shared expert's weight is the sigmoid of one more logit of the router launch.
 #include "common.cuh"
 #include "mixer.h"
 
@@ -55,7 +57,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(MoeRouteArgs a) {
   pdl_launch();
   pdl_wait();
   const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  const int n = a.E + a.I, D = a.D;
+  const int n = a.E + a.I, nl = n + a.shared_gate, D = a.D;  // slots; logits (a shared expert's gate behind the slots)
   const float* h = a.h + (size_t)r * D;
   // logits: every warp takes one slice of the input's coordinates for ALL slots (eight slots at a time, so that eight
   // independent weight loads are in flight per input load), the slices' partial sums meet in shared memory and are added
@@ -63,7 +65,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(MoeRouteArgs a) {
   const int per_w = ((D + nw - 1) / nw + 3) & ~3;
   const int k_lo = min(D, warp * per_w), k_hi = min(D, k_lo + per_w);
   const bool vec4 = (D % 4 == 0) && (((uintptr_t)h & 15) == 0) && (((uintptr_t)a.router & 15) == 0);
-  for (int e0 = 0; e0 < n; e0 += 8) {
+  for (int e0 = 0; e0 < nl; e0 += 8) {
     float acc[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) acc[j] = 0.f;
@@ -72,7 +74,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(MoeRouteArgs a) {
         const float4 hv = *reinterpret_cast<const float4*>(h + k);
 #pragma unroll
         for (int j = 0; j < 8; ++j)
-          if (e0 + j < n) {
+          if (e0 + j < nl) {
             const float4 wv = *reinterpret_cast<const float4*>(a.router + (size_t)(e0 + j) * D + k);
             acc[j] = fmaf(wv.x, hv.x, acc[j]); acc[j] = fmaf(wv.y, hv.y, acc[j]);
             acc[j] = fmaf(wv.z, hv.z, acc[j]); acc[j] = fmaf(wv.w, hv.w, acc[j]);
@@ -83,17 +85,17 @@ __global__ void __launch_bounds__(256) moe_route_kernel(MoeRouteArgs a) {
         const float hv = h[k];
 #pragma unroll
         for (int j = 0; j < 8; ++j)
-          if (e0 + j < n) acc[j] = fmaf(a.router[(size_t)(e0 + j) * D + k], hv, acc[j]);
+          if (e0 + j < nl) acc[j] = fmaf(a.router[(size_t)(e0 + j) * D + k], hv, acc[j]);
       }
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const float t = warp_sum(acc[j]);
-      if (lane == 0 && e0 + j < n) s_part[(e0 + j) * 8 + warp] = t;
+      if (lane == 0 && e0 + j < nl) s_part[(e0 + j) * 8 + warp] = t;
     }
   }
   __syncthreads();
-  for (int e = threadIdx.x; e < n; e += blockDim.x) {
+  for (int e = threadIdx.x; e < nl; e += blockDim.x) {
     float t = 0.f;
     for (int w = 0; w < nw; ++w) t += s_part[e * 8 + w];
     s_score[e] = t;
@@ -114,7 +116,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(MoeRouteArgs a) {
   for (int e = lane; e < n; e += 32) {
     const float sc = s_score[e] * inv;
     s_score[e] = sc;
-    s_choice[e] = sc + a.correction[e];
+    s_choice[e] = a.kind == 2 ? sc : sc + a.correction[e];
   }
   __syncwarp();
   }
@@ -148,7 +150,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(MoeRouteArgs a) {
   if (a.dense)
     for (int e = lane; e < a.E; e += 32) a.dense[(size_t)r * a.E + e] = 0.f;
   __syncwarp();
-  float idw = 0.f;
+  float idw = 0.f, chosen = 0.f;
   for (int k = 0; k < a.top; ++k) {
     float bv = -INFINITY; int bi = 0x7fffffff;
     for (int e = lane; e < n; e += 32) {
@@ -167,6 +169,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(MoeRouteArgs a) {
       const float w = ok ? s_score[e] * a.scale : 0.f;
       a.sel[(size_t)r * a.top + k] = e;
       a.w[(size_t)r * a.top + k] = w;
+      chosen += w;
       if (ok) {
         s_choice[e] = -INFINITY;
         if (e >= a.E) idw += w;
@@ -175,7 +178,15 @@ __global__ void __launch_bounds__(256) moe_route_kernel(MoeRouteArgs a) {
     }
     __syncwarp();
   }
-  if (lane == 0) a.idw[r] = idw;
+  if (a.kind == 2 && lane == 0) {  // the chosen scores over their sum
+    const float inv = 1.0f / (chosen + 1e-20f);
+    for (int k = 0; k < a.top; ++k) {
+      const float w = a.w[(size_t)r * a.top + k] * inv;
+      a.w[(size_t)r * a.top + k] = w;
+      if (a.dense) a.dense[(size_t)r * a.E + a.sel[(size_t)r * a.top + k]] = w;
+    }
+  }
+  if (lane == 0) a.idw[r] = a.shared_gate ? 1.0f / (1.0f + expf(-s_score[n])) : idw;
 }
 
 __global__ void moe_act_mask_kernel(float* __restrict__ u, const float* __restrict__ dense, int64_t n, int E, int ff,
@@ -241,8 +252,8 @@ __global__ void __launch_bounds__(256) moe_down_rows_kernel(const float* __restr
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 
-__global__ void moe_glu_act_kernel(const float* __restrict__ gu, const float* __restrict__ dense, int64_t n, int E, int ff, int sff,
-                                   float* __restrict__ hid, bf16* __restrict__ hid16) {
+__global__ void moe_glu_act_kernel(const float* __restrict__ gu, const float* __restrict__ dense, const float* __restrict__ shared_w,
+                                   int w_out, int64_t n, int E, int ff, int sff, float* __restrict__ hid, bf16* __restrict__ hid16) {
   pdl_launch();
   pdl_wait();
   const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -250,13 +261,13 @@ __global__ void moe_glu_act_kernel(const float* __restrict__ gu, const float* __
   const int64_t F = (int64_t)E * ff + sff;
   const int64_t r = i / F;
   const int64_t c = i - r * F;
-  const float w = c < (int64_t)E * ff ? dense[r * E + c / ff] : 1.0f;
+  const float w = c < (int64_t)E * ff ? dense[r * E + c / ff] : shared_w ? shared_w[r] : 1.0f;
   float o = 0.f;
   if (w != 0.f) {
     const float2 p = *reinterpret_cast<const float2*>(gu + 2 * i);
-    o = silu_f(w * p.x) * (w * p.y);
+    o = w_out ? w * silu_f(p.x) * p.y : silu_f(w * p.x) * (w * p.y);
   }
-  hid[i] = o;
+  if (hid) hid[i] = o;
   if (hid16) hid16[i] = __float2bfloat16_rn(o);
 }
 
@@ -264,8 +275,8 @@ __global__ void moe_glu_act_kernel(const float* __restrict__ gu, const float* __
 template <typename WT>
 __global__ void __launch_bounds__(256) moe_glu_up_rows_kernel(const float* __restrict__ h, const WT* __restrict__ w_gu,
                                                               const int32_t* __restrict__ sel, const float* __restrict__ wsel,
-                                                              int D, int E, int ff, int sff, int top, int hs,
-                                                              float* __restrict__ hid) {
+                                                              const float* __restrict__ shared_w, int w_out, int D, int E, int ff,
+                                                              int sff, int top, int hs, float* __restrict__ hid) {
   pdl_launch();
   pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -275,17 +286,17 @@ __global__ void __launch_bounds__(256) moe_glu_up_rows_kernel(const float* __res
   const int e = shared ? E : sel[row * top + k];
   const int width = shared ? sff : ff;
   if (j >= width || e > E || (!shared && e >= E)) return;
-  const float w = shared ? 1.0f : wsel[row * top + k];
+  const float w = !shared ? wsel[row * top + k] : shared_w ? shared_w[row] : 1.0f;
   const WT* wr = w_gu + ((size_t)2 * ((size_t)e * ff + j)) * D;
   const float* hr = h + (size_t)row * D;
   const float g = warp_dot(wr, hr, D, lane), u = warp_dot(wr + D, hr, D, lane);
-  if (lane == 0) hid[(size_t)slot * hs + j] = silu_f(w * g) * (w * u);
+  if (lane == 0) hid[(size_t)slot * hs + j] = w_out ? w * silu_f(g) * u : silu_f(w * g) * (w * u);
 }
 
 // grid (ceil(D / 8), rows): y[row, i] = sum over the row's slots of down_e[i] . hid[slot]
 template <typename WT>
 __global__ void __launch_bounds__(256) moe_glu_down_rows_kernel(const WT* __restrict__ w_down, const int32_t* __restrict__ sel,
-                                                                int D, int E, int ff, int sff, int top, int hs,
+                                                                int D, int E, int ff, int sff, int top, int hs, int add,
                                                                 const float* __restrict__ hid, float* __restrict__ y) {
   pdl_launch();
   pdl_wait();
@@ -301,35 +312,35 @@ __global__ void __launch_bounds__(256) moe_glu_down_rows_kernel(const WT* __rest
     if (!shared && e >= E) continue;
     acc += warp_dot(w_down + (size_t)i * F + (size_t)e * ff, hid + ((size_t)row * (top + 1) + k) * hs, shared ? sff : ff, lane);
   }
-  if (lane == 0) y[(size_t)row * D + i] = acc;
+  if (lane == 0) y[(size_t)row * D + i] = add ? y[(size_t)row * D + i] + acc : acc;
 }
 
 }  // namespace
 
-cudaError_t launch_moe_glu_act(const float* gu, const float* dense, int rows, int E, int ff, int sff, float* hid, bf16* hid16,
-                               cudaStream_t s) {
+cudaError_t launch_moe_glu_act(const float* gu, const float* dense, const float* shared_w, bool w_out, int rows, int E, int ff,
+                               int sff, float* hid, bf16* hid16, cudaStream_t s) {
   const int64_t n = (int64_t)rows * ((int64_t)E * ff + sff);
-  return launch_k(moe_glu_act_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, s, gu, dense, n, E, ff, sff, hid, hid16);
+  return launch_k(moe_glu_act_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, s, gu, dense, shared_w, (int)w_out, n, E, ff, sff, hid, hid16);
 }
 
 cudaError_t launch_moe_glu_rows(const float* h, const void* w_gu, const void* w_down, bool w_bf16, const int32_t* sel,
-                                const float* w, int rows, int D, int E, int ff, int sff, int top, float* hid, float* y,
-                                cudaStream_t s) {
+                                const float* w, const float* shared_w, bool w_out, int rows, int D, int E, int ff, int sff, int top,
+                                float* hid, float* y, bool add, cudaStream_t s) {
   const int hs = ff > sff ? ff : sff;
   const dim3 gu((hs + 7) / 8, rows * (top + 1)), gd((D + 7) / 8, rows);
   cudaError_t e;
   if (w_bf16) {
-    e = launch_k(moe_glu_up_rows_kernel<bf16>, gu, dim3(256), 0, s, h, (const bf16*)w_gu, sel, w, D, E, ff, sff, top, hs, hid);
+    e = launch_k(moe_glu_up_rows_kernel<bf16>, gu, dim3(256), 0, s, h, (const bf16*)w_gu, sel, w, shared_w, (int)w_out, D, E, ff, sff, top, hs, hid);
     if (e != cudaSuccess) return e;
-    return launch_k(moe_glu_down_rows_kernel<bf16>, gd, dim3(256), 0, s, (const bf16*)w_down, sel, D, E, ff, sff, top, hs, (const float*)hid, y);
+    return launch_k(moe_glu_down_rows_kernel<bf16>, gd, dim3(256), 0, s, (const bf16*)w_down, sel, D, E, ff, sff, top, hs, (int)add, (const float*)hid, y);
   }
-  e = launch_k(moe_glu_up_rows_kernel<float>, gu, dim3(256), 0, s, h, (const float*)w_gu, sel, w, D, E, ff, sff, top, hs, hid);
+  e = launch_k(moe_glu_up_rows_kernel<float>, gu, dim3(256), 0, s, h, (const float*)w_gu, sel, w, shared_w, (int)w_out, D, E, ff, sff, top, hs, hid);
   if (e != cudaSuccess) return e;
-  return launch_k(moe_glu_down_rows_kernel<float>, gd, dim3(256), 0, s, (const float*)w_down, sel, D, E, ff, sff, top, hs, (const float*)hid, y);
+  return launch_k(moe_glu_down_rows_kernel<float>, gd, dim3(256), 0, s, (const float*)w_down, sel, D, E, ff, sff, top, hs, (int)add, (const float*)hid, y);
 }
 
 cudaError_t launch_moe_route(const MoeRouteArgs& a, int rows, cudaStream_t s) {
-  if (a.E + a.I > MOE_MAX_SLOTS || a.groups < 1 || (a.E + a.I) % a.groups) return cudaErrorInvalidValue;
+  if (a.E + a.I + a.shared_gate > MOE_MAX_SLOTS || a.groups < 1 || (a.E + a.I) % a.groups) return cudaErrorInvalidValue;
   return launch_k(moe_route_kernel, dim3(rows), dim3(256), 0, s, a);
 }
 

@@ -17,6 +17,10 @@
 //   3. lin_chunk_out_kernel     A = (Q K^T) .* lam^(i-j) (causal), o = lam^(i+1) Q P_c + A V
 // Every product is an fp32 FFMA chain over shared-memory tiles (4 x 4 outputs per thread, operands stored with the
 // summed index outermost so that both are read as 16-byte vectors); the powers of lam come from double precision.
+// With a normaliser (NRM: RecurArgs::n_state, the mLSTM) a column n of the state with values 1 runs along: a chunk adds
+// the column sums of its scaled keys, and n . q is q . P_n plus the row sums of A.  Keys carry a factor per token
+// (k_scale), and the decays' running sums are kept in double precision: a log decay can be as large as -30, and the
+// difference of two sums of 64 of them is what enters the exponential.
 // The sums run in another order than the token-by-token kernel, so the two agree to fp32 rounding, not bit for bit.
 #include <stdint.h>
 
@@ -59,16 +63,17 @@ __device__ __forceinline__ void fill_powers(float* pw, float lam) {
 }
 
 // cl[j] = sum over t <= j of the chunk's log decays (tokens >= n add nothing): warp 0 scans, 32 tokens at a time
-__device__ __forceinline__ void fill_cumlog(float* cl, const float* __restrict__ lg, size_t stride, int n) {
+template <typename T>
+__device__ __forceinline__ void fill_cumlog(T* cl, const float* __restrict__ lg, size_t stride, int n) {
   if (threadIdx.x >= 32) return;
   const int lane = threadIdx.x;
-  float carry = 0.f;
+  T carry = 0;
   for (int j0 = 0; j0 < CH; j0 += 32) {
     const int j = j0 + lane;
-    float v = j < n ? lg[(size_t)j * stride] : 0.f;
+    T v = j < n ? (T)lg[(size_t)j * stride] : (T)0;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
-      const float t = __shfl_up_sync(L3_FULL, v, o);
+      const T t = __shfl_up_sync(L3_FULL, v, o);
       if (lane >= o) v += t;
     }
     v += carry;
@@ -79,6 +84,10 @@ __device__ __forceinline__ void fill_cumlog(float* cl, const float* __restrict__
 
 // where the chunks' total decays live inside the workspace: behind the chunk states
 __device__ __forceinline__ float* chunk_decays(const RecurArgs& a, int NC) { return a.ws + (size_t)a.B * a.H * NC * a.DK * a.DV; }
+// and the chunks' normaliser columns [B, H, NC, DK] behind those (on a multiple of four floats)
+__device__ __forceinline__ float* chunk_norms(const RecurArgs& a, int NC) {
+  return a.ws + (size_t)a.B * a.H * NC * a.DK * a.DV + (((size_t)a.B * a.H * NC + 3) & ~(size_t)3);
+}
 
 // rows [n, CH) of a natural [token][cols] tile and tokens >= n of the operands are zero: they add nothing
 __device__ __forceinline__ void load_natural(float* dst, int ld_dst, const float* src, size_t ld_src, int n, int cols, int act_in,
@@ -99,7 +108,7 @@ __device__ __forceinline__ void load_natural(float* dst, int ld_dst, const float
 
 // dst[channel][token] from rows [token][channel]: a lane takes four channels of one token (one 16-byte load), and
 // adjacent lanes take adjacent tokens, so the four scalar stores of a warp fall into distinct banks
-__device__ __forceinline__ void load_transposed(float* dst, const float* src, size_t ld_src, int n, int cols, int act_in) {
+__device__ __forceinline__ void load_transposed(float* dst, const float* src, size_t ld_src, int n, int cols, int act_in, float mul = 1.f) {
   const int c4 = cols / 4;
   for (int idx = threadIdx.x; idx < CH * c4; idx += blockDim.x) {
     const int j = idx % CH, c = (idx / CH) * 4;
@@ -107,6 +116,7 @@ __device__ __forceinline__ void load_transposed(float* dst, const float* src, si
     if (j < n) {
       v = *reinterpret_cast<const float4*>(src + (size_t)j * ld_src + c);
       v.x = act_silu(act_in, v.x); v.y = act_silu(act_in, v.y); v.z = act_silu(act_in, v.z); v.w = act_silu(act_in, v.w);
+      v.x *= mul; v.y *= mul; v.z *= mul; v.w *= mul;
     }
     dst[(size_t)(c + 0) * LDT + j] = v.x;
     dst[(size_t)(c + 1) * LDT + j] = v.y;
@@ -116,9 +126,10 @@ __device__ __forceinline__ void load_transposed(float* dst, const float* src, si
 }
 
 // ---------------------------------------------------------------------------- 1. what a chunk adds to the state
-template <bool DEC>
+template <bool DEC, bool NRM>
 __global__ void __launch_bounds__(256) lin_chunk_state_kernel(RecurArgs a, int NC) {
   extern __shared__ __align__(16) float sm[];
+  __shared__ double pd[NRM ? CH : 1];
   float* pw = sm;                 // [CH + 1] + scale per token [CH]
   float* sc = pw + CH + 4;        // lam^(n - 1 - j)
   float* Ks = sc + CH;            // [CH][DK]
@@ -128,15 +139,28 @@ __global__ void __launch_bounds__(256) lin_chunk_state_kernel(RecurArgs a, int N
   const int c = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
   const int n = min(CH, a.L - c * CH);
   const size_t row0 = (size_t)b * a.L + (size_t)c * CH;
-  if (DEC) fill_cumlog(pw, a.log_g + row0 * a.H + h, a.H, n);
+  if (NRM) fill_cumlog(pd, a.log_g + row0 * a.H + h, a.H, n);
+  else if (DEC) fill_cumlog(pw, a.log_g + row0 * a.H + h, a.H, n);
   else fill_powers(pw, a.head_decay[h]);
   __syncthreads();
-  for (int j = tid; j < CH; j += blockDim.x) sc[j] = j < n ? (DEC ? expf(pw[n - 1] - pw[j]) : pw[n - 1 - j]) : 0.f;
-  if (DEC && tid == 0) chunk_decays(a, NC)[((size_t)b * a.H + h) * NC + c] = expf(pw[n - 1]);
+  if (NRM) {
+    for (int j = tid; j < CH; j += blockDim.x) sc[j] = j < n ? expf((float)(pd[n - 1] - pd[j])) * a.k_scale[(row0 + j) * a.H + h] : 0.f;
+    if (tid == 0) chunk_decays(a, NC)[((size_t)b * a.H + h) * NC + c] = expf((float)pd[n - 1]);
+  } else {
+    for (int j = tid; j < CH; j += blockDim.x) sc[j] = j < n ? (DEC ? expf(pw[n - 1] - pw[j]) : pw[n - 1 - j]) : 0.f;
+    if (DEC && tid == 0) chunk_decays(a, NC)[((size_t)b * a.H + h) * NC + c] = expf(pw[n - 1]);
+  }
   __syncthreads();
   load_natural(Ks, a.DK, a.k + row0 * a.ld_k + (size_t)(h / a.rep) * a.DK, a.ld_k, n, a.DK, a.act_in, sc);
   load_natural(Vs, a.DV, a.v + row0 * a.ld_v + (size_t)h * a.DV, a.ld_v, n, a.DV, a.act_in, nullptr);
   __syncthreads();
+  if (NRM)
+    for (int d = tid; d < a.DK; d += blockDim.x) {
+      float t = 0.f;
+#pragma unroll 8
+      for (int j = 0; j < CH; ++j) t += Ks[(size_t)j * a.DK + d];
+      chunk_norms(a, NC)[(((size_t)b * a.H + h) * NC + c) * a.DK + d] = t;
+    }
   const int tx = tid & 15, ty = tid >> 4;
   float* D = a.ws + (((size_t)b * a.H + h) * NC + c) * a.DK * a.DV;
   for (int d0 = 0; d0 < a.DK; d0 += 64)
@@ -152,20 +176,30 @@ __global__ void __launch_bounds__(256) lin_chunk_state_kernel(RecurArgs a, int N
 }
 
 // ---------------------------------------------------------------------------- 2. the states between the chunks
-template <bool DEC>
+template <bool DEC, bool NRM>
 __global__ void __launch_bounds__(256) lin_chunk_scan_kernel(RecurArgs a, int NC) {
   pdl_launch();
   pdl_wait();
   const int h = blockIdx.y, b = blockIdx.z;
-  const size_t n4 = (size_t)a.DK * a.DV / 4;
-  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i >= n4) return;
+  size_t n4 = (size_t)a.DK * a.DV / 4;
+  size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  const bool is_n = NRM && i >= n4;  // the normaliser's column, behind the matrix
+  if (i >= n4 + (NRM ? a.DK / 4 : 0)) return;
   const float lam = DEC ? 0.f : a.head_decay[h];
   const float full = DEC ? 0.f : (float)pow((double)lam, (double)CH);
   const float last = DEC ? 0.f : (float)pow((double)lam, (double)(a.L - (NC - 1) * CH));
   const float* cdec = DEC ? chunk_decays(a, NC) + ((size_t)b * a.H + h) * NC : nullptr;
-  float4* st = reinterpret_cast<float4*>(a.state + ((size_t)b * a.H + h) * a.DK * a.DV) + i;
-  float4* W = reinterpret_cast<float4*>(a.ws + ((size_t)b * a.H + h) * NC * a.DK * a.DV) + i;
+  float4* st;
+  float4* W;
+  if (is_n) {
+    i -= n4;
+    n4 = a.DK / 4;
+    st = reinterpret_cast<float4*>(a.n_state + ((size_t)b * a.H + h) * a.DK) + i;
+    W = reinterpret_cast<float4*>(chunk_norms(a, NC) + ((size_t)b * a.H + h) * NC * a.DK) + i;
+  } else {
+    st = reinterpret_cast<float4*>(a.state + ((size_t)b * a.H + h) * a.DK * a.DV) + i;
+    W = reinterpret_cast<float4*>(a.ws + ((size_t)b * a.H + h) * NC * a.DK * a.DV) + i;
+  }
   float4 S = *st;
   // the chunk sums do not depend on S: four loads stay in flight ahead of the chain
   constexpr int AHEAD = 4;
@@ -189,9 +223,11 @@ __global__ void __launch_bounds__(256) lin_chunk_scan_kernel(RecurArgs a, int NC
 }
 
 // ---------------------------------------------------------------------------- 3. the outputs of a chunk
-template <bool DEC>
+template <bool DEC, bool NRM>
 __global__ void __launch_bounds__(256) lin_chunk_out_kernel(RecurArgs a, int NC) {
   extern __shared__ __align__(16) float sm[];
+  __shared__ double pd[NRM ? CH : 1];
+  __shared__ float ks[NRM ? CH : 1];
   float* pw = sm;                            // [CH + 1]
   float* Qt = pw + CH + 4;                   // [DK][LDT]
   float* Kt = Qt + (size_t)a.DK * LDT;       // [DK][LDT]
@@ -203,9 +239,12 @@ __global__ void __launch_bounds__(256) lin_chunk_out_kernel(RecurArgs a, int NC)
   const int c = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
   const int n = min(CH, a.L - c * CH);
   const size_t row0 = (size_t)b * a.L + (size_t)c * CH;
-  if (DEC) fill_cumlog(pw, a.log_g + row0 * a.H + h, a.H, n);
+  if (NRM) {
+    fill_cumlog(pd, a.log_g + row0 * a.H + h, a.H, n);
+    if (tid >= 32 && tid < 32 + CH) ks[tid - 32] = tid - 32 < n ? a.k_scale[(row0 + tid - 32) * a.H + h] : 0.f;
+  } else if (DEC) fill_cumlog(pw, a.log_g + row0 * a.H + h, a.H, n);
   else fill_powers(pw, a.head_decay[h]);
-  load_transposed(Qt, a.q + row0 * a.ld_q + (size_t)(h / a.rep) * a.DK, a.ld_q, n, a.DK, a.act_in);
+  load_transposed(Qt, a.q + row0 * a.ld_q + (size_t)(h / a.rep) * a.DK, a.ld_q, n, a.DK, a.act_in, NRM ? a.q_mul : 1.f);
   load_transposed(Kt, a.k + row0 * a.ld_k + (size_t)(h / a.rep) * a.DK, a.ld_k, n, a.DK, a.act_in);
   __syncthreads();
   const int tx = tid & 15, ty = tid >> 4;
@@ -221,10 +260,23 @@ __global__ void __launch_bounds__(256) lin_chunk_out_kernel(RecurArgs a, int NC)
 #pragma unroll
       for (int r = 0; r < 4; ++r) {
         const int i = ty * 4 + r;
-        op[r] = j <= i ? acc[r][cc] * (DEC ? expf(pw[i] - pw[j]) : pw[i - j]) : 0.f;
+        if (NRM) op[r] = j <= i ? acc[r][cc] * (expf((float)(pd[i] - pd[j])) * ks[j]) : 0.f;
+        else op[r] = j <= i ? acc[r][cc] * (DEC ? expf(pw[i] - pw[j]) : pw[i - j]) : 0.f;
       }
       *reinterpret_cast<float4*>(At + (size_t)j * LDT + ty * 4) = o;
     }
+  }
+  if (NRM) {  // n . q of every token: four threads per row
+    const float* Pn = chunk_norms(a, NC) + (((size_t)b * a.H + h) * NC + c) * a.DK;
+    __syncthreads();  // At is written
+    const int i = tid >> 2, part = tid & 3;
+    float t = 0.f;
+    for (int d = part; d < a.DK; d += 4) t = fmaf(Qt[(size_t)d * LDT + i], Pn[d], t);
+    t *= expf((float)pd[i]);
+    for (int j = part; j <= i; j += 4) t += At[(size_t)j * LDT + i];
+    t += __shfl_xor_sync(L3_FULL, t, 1);
+    t += __shfl_xor_sync(L3_FULL, t, 2);
+    if (part == 0 && i < n) a.nq[(row0 + i) * a.H + h] = t;
   }
   const float* P = a.ws + (((size_t)b * a.H + h) * NC + c) * a.DK * a.DV;
   const int O = a.H * a.DV;
@@ -241,7 +293,7 @@ __global__ void __launch_bounds__(256) lin_chunk_out_kernel(RecurArgs a, int NC)
     mm44(Qt + ty * 4, LDT, Ps + tx * 4, 64, a.DK, acc);
 #pragma unroll
     for (int r = 0; r < 4; ++r) {
-      const float f = DEC ? expf(pw[ty * 4 + r]) : pw[ty * 4 + r + 1];
+      const float f = NRM ? expf((float)pd[ty * 4 + r]) : DEC ? expf(pw[ty * 4 + r]) : pw[ty * 4 + r + 1];
 #pragma unroll
       for (int cc = 0; cc < 4; ++cc) acc[r][cc] *= f;
     }
@@ -262,10 +314,10 @@ bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
 
 size_t recur_chunk_ws_floats(int B, int L, int H, int DK, int DV) {
   const size_t NC = (L + CH - 1) / CH;
-  return (size_t)B * H * NC * DK * DV + (size_t)B * H * NC;  // chunk states, then the chunks' total decays
+  return (size_t)B * H * NC * DK * DV + (size_t)B * H * NC + 4 + (size_t)B * H * NC * DK;  // chunk states, total decays, normalisers
 }
 
-bool recur_chunk_shape(int DK, int DV) { return (DK == 64 || DK == 128) && DV % 64 == 0 && DV >= 64 && DV <= 512; }
+bool recur_chunk_shape(int DK, int DV) { return DK % 64 == 0 && DK <= 256 && DV % 64 == 0 && DV >= 64 && DV <= 512; }
 
 bool recur_chunk_supported(const RecurArgs& a) {
   const bool per_token = a.mode == 2 && a.g_head && a.log_g;  // one decay per head and token
@@ -282,18 +334,16 @@ cudaError_t launch_recur_chunk(const RecurArgs& a, cudaStream_t s) {
   const dim3 grid(NC, a.H, a.B);
   const size_t sm1 = (size_t)(CH + 4 + CH + CH * a.DK + CH * a.DV) * sizeof(float);
   const size_t sm3 = (size_t)(CH + 4 + 2 * a.DK * LDT + CH * LDT + CH * 64) * sizeof(float);
-  cudaError_t e;
-  const int n4 = a.DK * a.DV / 4;
-  if (a.mode == 2) {
-    if ((e = cudaFuncSetAttribute(lin_chunk_state_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm1)) != cudaSuccess) return e;
-    if ((e = cudaFuncSetAttribute(lin_chunk_out_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm3)) != cudaSuccess) return e;
-    if ((e = launch_k(lin_chunk_state_kernel<true>, grid, dim3(256), sm1, s, a, NC)) != cudaSuccess) return e;
-    if ((e = launch_k(lin_chunk_scan_kernel<true>, dim3((n4 + 255) / 256, a.H, a.B), dim3(256), 0, s, a, NC)) != cudaSuccess) return e;
-    return launch_k(lin_chunk_out_kernel<true>, grid, dim3(256), sm3, s, a, NC);
-  }
-  if ((e = cudaFuncSetAttribute(lin_chunk_state_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm1)) != cudaSuccess) return e;
-  if ((e = cudaFuncSetAttribute(lin_chunk_out_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm3)) != cudaSuccess) return e;
-  if ((e = launch_k(lin_chunk_state_kernel<false>, grid, dim3(256), sm1, s, a, NC)) != cudaSuccess) return e;
-  if ((e = launch_k(lin_chunk_scan_kernel<false>, dim3((n4 + 255) / 256, a.H, a.B), dim3(256), 0, s, a, NC)) != cudaSuccess) return e;
-  return launch_k(lin_chunk_out_kernel<false>, grid, dim3(256), sm3, s, a, NC);
+  const int n4 = (a.DK * a.DV + (a.n_state ? a.DK : 0)) / 4;
+  auto go = [&](auto k_state, auto k_scan, auto k_out) {
+    cudaError_t e;
+    if ((e = cudaFuncSetAttribute(k_state, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm1)) != cudaSuccess) return e;
+    if ((e = cudaFuncSetAttribute(k_out, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm3)) != cudaSuccess) return e;
+    if ((e = launch_k(k_state, grid, dim3(256), sm1, s, a, NC)) != cudaSuccess) return e;
+    if ((e = launch_k(k_scan, dim3((n4 + 255) / 256, a.H, a.B), dim3(256), 0, s, a, NC)) != cudaSuccess) return e;
+    return launch_k(k_out, grid, dim3(256), sm3, s, a, NC);
+  };
+  if (a.n_state) return go(lin_chunk_state_kernel<true, true>, lin_chunk_scan_kernel<true, true>, lin_chunk_out_kernel<true, true>);
+  if (a.mode == 2) return go(lin_chunk_state_kernel<true, false>, lin_chunk_scan_kernel<true, false>, lin_chunk_out_kernel<true, false>);
+  return go(lin_chunk_state_kernel<false, false>, lin_chunk_scan_kernel<false, false>, lin_chunk_out_kernel<false, false>);
 }

@@ -5,6 +5,8 @@
 //   mode 0   S <- decay_h S + k v^T                                   o = S^T q
 //   mode 1   S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T    o = S^T q   (o sees this token's write)
 //   mode 2   S <- diag(g) S + k v^T                                   o = S^T q   (g per key channel, or one per head)
+//            With RecurArgs::n_state one more column n runs beside the values, n <- g n + k, and nq = n . q goes out (the
+//            normaliser of an mLSTM): column DV of a head, with the value 1 for every token.
 //
 // The columns of S never mix: column j needs v_j, the token's k, q, g (shared by all columns) and nothing of
 // any other column.  So a CTA owns a tile of CPB columns of one (slot, head) for the whole call; a column is
@@ -36,19 +38,22 @@ __global__ void __launch_bounds__(256) recur_kernel(RecurArgs a, int TPC, int CP
   pdl_launch();
   pdl_wait();
   const int tid = threadIdx.x, nthr = blockDim.x;
-  const int ntile = (a.DV + CPB - 1) / CPB;
+  const int ncol = a.DV + (MODE == 2 && a.n_state ? 1 : 0);  // columns of a head
+  const int ntile = (ncol + CPB - 1) / CPB;
   const int h = blockIdx.x / ntile, tile = blockIdx.x - h * ntile, b = blockIdx.y;
   const int kvh = h / a.rep;
   const int cl = tid / TPC, s = tid - cl * TPC;
   const int j = tile * CPB + cl;
   const bool live = cl < CPB;  // a CTA is padded to a whole warp when CPB * TPC < 32
-  const bool col_ok = live && j < a.DV;
-  float* Sg = a.state + ((size_t)b * a.H + h) * a.DK * a.DV;
+  const bool col_ok = live && j < ncol;
+  float* Sg = a.state + ((size_t)b * a.H + h) * a.DK * a.DV + j;
+  int s_ld = a.DV;
+  if (MODE == 2 && j >= a.DV && a.n_state) { Sg = a.n_state + ((size_t)b * a.H + h) * a.DK; s_ld = 1; }
   float S[R];
 #pragma unroll
   for (int r = 0; r < R; ++r) {
     const int i = s + r * TPC;
-    S[r] = (col_ok && i < a.DK) ? Sg[(size_t)i * a.DV + j] : 0.f;
+    S[r] = (col_ok && i < a.DK) ? Sg[(size_t)i * s_ld] : 0.f;
   }
   const float lam = MODE == 0 ? a.head_decay[h] : 0.f;
 
@@ -63,6 +68,7 @@ __global__ void __launch_bounds__(256) recur_kernel(RecurArgs a, int TPC, int CP
         qv = a.q[row * a.ld_q + (size_t)kvh * a.DK + i];
         kv = a.k[row * a.ld_k + (size_t)kvh * a.DK + i];
         if (a.act_in) { qv = silu_ref(qv); kv = silu_ref(kv); }
+        if (MODE == 2 && a.k_scale) { kv *= a.k_scale[row * (size_t)a.H + h]; qv *= a.q_mul; }
         if (MODE >= 1) gv = a.g_head ? a.g[row * (size_t)a.H + h] : a.g[row * ((size_t)a.H * a.DK) + (size_t)h * a.DK + i];
       }
       sq[idx] = qv;
@@ -76,7 +82,7 @@ __global__ void __launch_bounds__(256) recur_kernel(RecurArgs a, int TPC, int CP
       if (jj < a.DV) {
         vv = a.v[((size_t)b * a.L + t0 + tok) * a.ld_v + (size_t)h * a.DV + jj];
         if (a.act_in) vv = silu_ref(vv);
-      }
+      } else if (MODE == 2 && jj == a.DV && a.n_state) vv = 1.f;
       sv[idx] = vv;
     }
     if (MODE == 1)
@@ -127,12 +133,13 @@ __global__ void __launch_bounds__(256) recur_kernel(RecurArgs a, int TPC, int CP
       const int tok = idx / CPB, c = idx - tok * CPB;
       const int jj = tile * CPB + c;
       if (jj < a.DV) a.out[((size_t)b * a.L + t0 + tok) * ((size_t)a.H * a.DV) + (size_t)h * a.DV + jj] = so[idx];
+      else if (MODE == 2 && jj == a.DV && a.n_state) a.nq[((size_t)b * a.L + t0 + tok) * a.H + h] = so[idx];
     }
   }
 #pragma unroll
   for (int r = 0; r < R; ++r) {
     const int i = s + r * TPC;
-    if (col_ok && i < a.DK) Sg[(size_t)i * a.DV + j] = S[r];
+    if (col_ok && i < a.DK) Sg[(size_t)i * s_ld] = S[r];
   }
 }
 
@@ -159,18 +166,21 @@ __global__ void __launch_bounds__(256) recur_pipe_kernel(RecurArgs a) {
   pdl_wait();
   const int tid = threadIdx.x;
   constexpr int ntile_den = CPB;
-  const int ntile = (a.DV + ntile_den - 1) / ntile_den;
+  const int ncol = a.DV + (MODE == 2 && a.n_state ? 1 : 0);  // columns of a head
+  const int ntile = (ncol + ntile_den - 1) / ntile_den;
   const int h = blockIdx.x / ntile, tile = blockIdx.x - h * ntile, b = blockIdx.y;
   const int kvh = h / a.rep;
   const int cl = tid / TPC, s = tid % TPC;
   const int j = tile * CPB + cl;
-  const bool col_ok = j < a.DV;
-  float* Sg = a.state + ((size_t)b * a.H + h) * a.DK * a.DV;
+  const bool col_ok = j < ncol;
+  float* Sg = a.state + ((size_t)b * a.H + h) * a.DK * a.DV + j;
+  int s_ld = a.DV;
+  if (MODE == 2 && j >= a.DV && a.n_state) { Sg = a.n_state + ((size_t)b * a.H + h) * a.DK; s_ld = 1; }
   float S[R];
 #pragma unroll
   for (int r = 0; r < R; ++r) {
     const int i = 4 * (s + (r >> 2) * TPC) + (r & 3);
-    S[r] = (col_ok && i < a.DK) ? Sg[(size_t)i * a.DV + j] : 0.f;
+    S[r] = (col_ok && i < a.DK) ? Sg[(size_t)i * s_ld] : 0.f;
   }
   const float lam = MODE == 0 ? a.head_decay[h] : 0.f;
   const size_t row0 = (size_t)b * a.L;
@@ -181,6 +191,9 @@ __global__ void __launch_bounds__(256) recur_pipe_kernel(RecurArgs a) {
   constexpr int TSTEP = 256 / DKP, VSTEP = CPB >= 256 ? 1 : 256 / CPB;
   const int i_f = tid % DKP, tok_f = tid / DKP, c_f = tid % CPB, tok_v = tid / CPB;
   const bool i_ok = i_f < a.DK, c_ok = tile * CPB + c_f < a.DV;
+  const bool c_one = MODE == 2 && a.n_state && tile * CPB + c_f == a.DV;  // the normaliser's column: value 1
+  const float q_mul = MODE == 2 && a.k_scale ? a.q_mul : 1.f;
+  const float* ks_f = MODE == 2 && a.k_scale ? a.k_scale + (row0 + tok_f) * a.H + h : nullptr;
   const float* q_f = a.q + (row0 + tok_f) * a.ld_q + (size_t)kvh * a.DK + i_f;
   const float* k_f = a.k + (row0 + tok_f) * a.ld_k + (size_t)kvh * a.DK + i_f;
   // the decays: one per (head, key channel), or with g_head one per head
@@ -197,13 +210,14 @@ __global__ void __launch_bounds__(256) recur_pipe_kernel(RecurArgs a) {
       const bool ok = i_ok && t0 + tok_f + n * TSTEP < a.L;
       pq[n] = ok ? qp[n * q_st] : 0.f;
       pk[n] = ok ? kp[n * k_st] : 0.f;
+      if (MODE == 2 && ks_f) { pk[n] *= ok ? ks_f[(size_t)(t0 + n * TSTEP) * a.H] : 0.f; pq[n] *= q_mul; }
       if (MODE >= 1) pg[n] = ok ? gp[n * g_st] : 0.f;
     }
     const float* vp = v_f + (size_t)t0 * a.ld_v;
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
       const bool ok = c_ok && tok_v + n * VSTEP < TCH && t0 + tok_v + n * VSTEP < a.L;
-      pv[n] = ok ? vp[n * v_st] : 0.f;
+      pv[n] = ok ? vp[n * v_st] : MODE == 2 && c_one ? 1.f : 0.f;
     }
     if (MODE == 1 && tid < TCH) pb = t0 + tid < a.L ? a.beta[(row0 + t0 + tid) * a.H + h] : 0.f;
   };
@@ -350,13 +364,14 @@ __global__ void __launch_bounds__(256) recur_pipe_kernel(RecurArgs a) {
       const int tok = e / CPB, c = e % CPB;
       const int jj = tile * CPB + c;
       if (jj < a.DV) a.out[(row0 + t0 + tok) * ((size_t)a.H * a.DV) + (size_t)h * a.DV + jj] = so[e];
+      else if (MODE == 2 && jj == a.DV && a.n_state) a.nq[(row0 + t0 + tok) * a.H + h] = so[e];
     }
     __syncthreads();  // the next chunk's compute writes `so` again
   }
 #pragma unroll
   for (int r = 0; r < R; ++r) {
     const int i = 4 * (s + (r >> 2) * TPC) + (r & 3);
-    if (col_ok && i < a.DK) Sg[(size_t)i * a.DV + j] = S[r];
+    if (col_ok && i < a.DK) Sg[(size_t)i * s_ld] = S[r];
   }
 }
 
@@ -365,7 +380,7 @@ cudaError_t launch_recur_pipe(const RecurArgs& a, cudaStream_t s) {
   constexpr int DKP = 8 * TPC, CPB = 256 / TPC;
   const int NA = a.mode >= 1 ? 3 : 2;
   const size_t smem = (size_t)(2 * (RP_TCH * (NA * DKP + CPB) + RP_TCH) + RP_TCH * CPB) * sizeof(float);
-  const dim3 grid(a.H * ((a.DV + CPB - 1) / CPB), a.B);
+  const dim3 grid(a.H * ((a.DV + (a.n_state ? 1 : 0) + CPB - 1) / CPB), a.B);
   auto go = [&](auto kern) {
     if (smem > 48 * 1024) {
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -391,7 +406,7 @@ cudaError_t launch_recur_r(const RecurArgs& a, cudaStream_t s) {
   const int per_tok = (a.mode >= 1 ? 3 : 2) * DKP + 2 * CPB + 1;
   const int TCH = std::max(1, std::min(32, 11000 / per_tok));
   const size_t smem = (size_t)TCH * per_tok * sizeof(float);
-  const int ntile = (a.DV + CPB - 1) / CPB;
+  const int ntile = (a.DV + (a.n_state ? 1 : 0) + CPB - 1) / CPB;
   const dim3 grid(a.H * ntile, a.B);
   if (a.mode == 0) return launch_k(recur_kernel<R, 0>, grid, dim3(threads), smem, s, a, TPC, CPB, TCH);
   if (a.mode == 2) return launch_k(recur_kernel<R, 2>, grid, dim3(threads), smem, s, a, TPC, CPB, TCH);
@@ -404,6 +419,7 @@ bool recur_supported(int DK, int DV) { return DK >= 1 && DK <= 1024 && DV >= 1; 
 
 cudaError_t launch_recur(const RecurArgs& a, cudaStream_t s) {
   if (!recur_supported(a.DK, a.DV)) return cudaErrorInvalidValue;
+  if ((a.n_state || a.k_scale) && (a.mode != 2 || !a.k_scale || !a.nq)) return cudaErrorInvalidValue;
   static const bool chunk_on = !(getenv("L3_RECUR_CHUNK") && atoi(getenv("L3_RECUR_CHUNK")) == 0);
   if (chunk_on && recur_chunk_supported(a)) return launch_recur_chunk(a, s);  // prompts of the common shapes
   static const bool pipe_on = !(getenv("L3_RECUR_PIPE") && atoi(getenv("L3_RECUR_PIPE")) == 0);

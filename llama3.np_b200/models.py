@@ -57,8 +57,15 @@ def _gifudra(model_dir, config, *, dtype, max_seq_len, max_batch_size, device):
                    max_seq_len=max_seq_len or 256, max_batch_size=max_batch_size, device=device)
 
 
+def _vupitar(model_dir, config, *, dtype, max_seq_len, max_batch_size, device):
+    from .vupitar import Vupitar
+    from .utils import read_safetensors
+    return Vupitar(config, read_safetensors(os.path.join(model_dir, "model.safetensors")), dtype=dtype,
+                   max_seq_len=max_seq_len or 256, max_batch_size=max_batch_size, device=device)
+
+
 ARCHITECTURES = {"Llama": _llama, "Risalix": _risalix, "Rakelorn": _rakelorn, "Mabedra": _mabedra, "Debuzen": _debuzen,
-                 "Gifudra": _gifudra}
+                 "Gifudra": _gifudra, "Vupitar": _vupitar}
 
 
 def load_model(model_dir, *, dtype: str = "float32", max_seq_len: int = 0, max_batch_size: int = 1, device: int = 0):

@@ -19,10 +19,10 @@ from . import _cabi
 
 SOFTMAX, DECAY_LINEAR, GATED_DELTA = _cabi.MIX_SOFTMAX, _cabi.MIX_DECAY_LINEAR, _cabi.MIX_GATED_DELTA
 LATENT, MINGRU, DIFF = _cabi.MIX_LATENT, _cabi.MIX_MINGRU, _cabi.MIX_DIFF
-WINDOW, SSD, GLA = _cabi.MIX_WINDOW, _cabi.MIX_SSD, _cabi.MIX_GLA
-ATTN_SINK, ATTN_SIGMOID = _cabi.ATTN_SINK, _cabi.ATTN_SIGMOID
-FF_GLU, FF_POLYNORM, FF_RELU2 = _cabi.FF_GLU, _cabi.FF_POLYNORM, _cabi.FF_RELU2
-ROUTE_SOFTMAX, ROUTE_SIGMOID_IN = _cabi.ROUTE_SOFTMAX, _cabi.ROUTE_SIGMOID_IN
+WINDOW, SSD, GLA, MLSTM = _cabi.MIX_WINDOW, _cabi.MIX_SSD, _cabi.MIX_GLA, _cabi.MIX_MLSTM
+ATTN_SINK, ATTN_SIGMOID, ATTN_SOFTMAX = _cabi.ATTN_SINK, _cabi.ATTN_SIGMOID, _cabi.ATTN_SOFTMAX
+FF_GLU, FF_POLYNORM, FF_RELU2, FF_CLAMP = _cabi.FF_GLU, _cabi.FF_POLYNORM, _cabi.FF_RELU2, _cabi.FF_CLAMP
+ROUTE_SOFTMAX, ROUTE_SIGMOID_IN, ROUTE_SOFTMAX_GLU = _cabi.ROUTE_SOFTMAX, _cabi.ROUTE_SIGMOID_IN, _cabi.ROUTE_SOFTMAX_GLU
 _DTYPES = {"float32": _cabi.DTYPE_F32, "fp32": _cabi.DTYPE_F32, "bfloat16": _cabi.DTYPE_BF16, "bf16": _cabi.DTYPE_BF16}
 
 
@@ -53,11 +53,11 @@ class LayerSpec:
     window: int = 0               # DIFF: keys a query sees, itself included; 0 = all
     diff: float = 0.0             # DIFF: constant of lambda and of the output multiplier 1 - diff
     rot_scaling: Optional[Tuple[float, float, float, int]] = None   # DIFF: (factor, low, high, original) or None
-    ff_kind: int = 0              # FF_GLU | FF_POLYNORM | FF_RELU2
-    router_kind: int = 0          # ROUTE_SOFTMAX | ROUTE_SIGMOID_IN
-    shared_ff: int = 0            # ROUTE_SIGMOID_IN: width of the shared expert
+    ff_kind: int = 0              # FF_GLU | FF_POLYNORM | FF_RELU2 | FF_CLAMP
+    router_kind: int = 0          # ROUTE_SOFTMAX | ROUTE_SIGMOID_IN | ROUTE_SOFTMAX_GLU
+    shared_ff: int = 0            # ROUTE_SIGMOID_IN, ROUTE_SOFTMAX_GLU: width of the shared expert
     keep_first: int = 0           # WINDOW: the first tokens that stay visible behind the window
-    attn_kind: int = 0            # WINDOW: ATTN_SINK (softmax with a sink per head) | ATTN_SIGMOID (sigmoid(score + bias), not normalised)
+    attn_kind: int = 0            # WINDOW: ATTN_SINK (softmax with a sink per head) | ATTN_SIGMOID (sigmoid(score + bias), not normalised) | ATTN_SOFTMAX
     rot_layout: int = 0           # WINDOW, LATENT: 0 = entries (2i, 2i + 1) turn together, 1 = entries (i, i + rot_dims / 2)
     qk_unit: bool = False         # WINDOW: q and k over their root mean square per head, after the rotation
     out_norm_groups: int = 1      # SSD: parts of the output norm
@@ -68,6 +68,14 @@ class LayerSpec:
     kv_from: Optional[int] = None  # LATENT: the layer whose cache rows this one attends over (None: its own)
     sink: bool = False            # LATENT: a learned logit per head in the softmax denominator
     gate_wide: bool = False       # LATENT: the output gate has one entry per value instead of one per head
+    chunked: bool = False         # WINDOW: `window` is a chunk size: i sees j <= i only where i // window == j // window
+    qk_norm: bool = False         # WINDOW: RMS norm per head with a weight on q and k, ahead of the rotation
+    proj_bias: bool = False       # WINDOW: biases of the q, k, v and output projections
+    head_gate: bool = False       # WINDOW: a sigmoid gate per head on the output
+    gate_cap: float = 0.0         # MLSTM: soft cap of the gates' logits
+    ff_limit: float = 0.0         # FF_CLAMP
+    ff_slope: float = 0.0         # FF_CLAMP
+    shared_gate: bool = False     # ROUTE_SOFTMAX_GLU: the shared expert has a sigmoid gate of its own
 
 
 @dataclass
@@ -97,6 +105,9 @@ class StackConfig:
     streams: int = 0              # pre-norm stacks: residual rows per token (0: one row, plain sums), mixed by l<i>.hc1 / hc2 tensors
     tied_head: bool = False       # the output projection is the embedding table
     logit_scale: float = 1.0      # multiplier of the logits
+    norm_tanh: bool = False       # every norm is tanh(alpha x) w + b
+    dual_norm: bool = False       # both sublayers read the same stream, each through its own norm
+    loop_x0: bool = False         # ahead of every pass of the loop but the first the embedding output joins the stream
     max_seq_len: int = 256
     max_batch_size: int = 1
     dtype: str = "float32"
@@ -141,7 +152,9 @@ class StackDecoder:
                                          pair=C.pointer(pair) if pair is not None else None,
                                          mix_scale=float(l.mix_scale), pair_scale=float(l.pair_scale),
                                          kv_source=0 if l.kv_from is None else int(l.kv_from) + 1, sink=int(l.sink),
-                                         gate_wide=int(l.gate_wide))
+                                         gate_wide=int(l.gate_wide), chunked=int(l.chunked), qk_norm=int(l.qk_norm),
+                                         proj_bias=int(l.proj_bias), head_gate=int(l.head_gate), gate_cap=float(l.gate_cap),
+                                         ff_limit=float(l.ff_limit), ff_slope=float(l.ff_slope), shared_gate=int(l.shared_gate))
 
         for i, l in enumerate(cfg.layers):
             specs[i] = c_spec(i, l)
@@ -156,7 +169,8 @@ class StackDecoder:
                                 norm_center=int(cfg.norm_center), layer_scale=int(cfg.layer_scale),
                                 canon_taps=int(cfg.canon_taps), depth_avg=int(cfg.depth_avg), norm_groups=int(cfg.norm_groups),
                                 embed_norm=int(cfg.embed_norm), loop_in=int(cfg.loop_in), logit_softcap=float(cfg.logit_softcap),
-                                streams=int(cfg.streams), tied_head=int(cfg.tied_head), logit_scale=float(cfg.logit_scale))
+                                streams=int(cfg.streams), tied_head=int(cfg.tied_head), logit_scale=float(cfg.logit_scale),
+                                norm_tanh=int(cfg.norm_tanh), dual_norm=int(cfg.dual_norm), loop_x0=int(cfg.loop_x0))
         _cabi.check(self._lib.l3_create_stack(C.byref(c), specs, C.byref(self._h)))
         n = C.c_int()
         _cabi.check(self._lib.l3_stack_runs(self._h, C.byref(n)), self._h)
@@ -307,8 +321,8 @@ class StackDecoder:
         return run - span * (times - 1)
 
     def read_state(self, layer: int, slot: int = 0):
-        """(S [heads, dim, vdim], conv tail [channels, taps - 1] or None) of a recurrent layer run's slot; for a
-        latent-attention run S is the cache it reads, `[max_seq_len, kv_rank + rot_dim]`.  `layer` counts layer runs."""
+        """(S [heads, dim, vdim], conv tail [channels, taps - 1] or None) of a recurrent layer run's slot - for an mLSTM
+        the second item is [normalisers [heads, dim] | running maxima [heads]] as one vector; for a latent-attention run S is the cache it reads, `[max_seq_len, kv_rank + rot_dim]`.  `layer` counts layer runs."""
         l = self.cfg.layers[self.run_layer(layer)]
         if l.pair is not None and l.mixer == WINDOW:   # two mixers side by side: the recurrent one
             l = l.pair
@@ -322,6 +336,8 @@ class StackDecoder:
             g = l.kv_heads or l.heads
             ch = 2 * g * l.dim + l.heads * l.vdim
             tail = np.empty((ch, max(0, l.conv_taps - 1)), dtype=np.float32)
+        elif l.mixer == MLSTM:
+            tail = np.empty((l.heads * (l.dim + 1),), dtype=np.float32)
         _cabi.check(self._lib.l3_read_state(self._h, layer, slot, _cabi.f32p(S), _cabi.f32p(tail) if tail is not None and tail.size else None),
                     self._h)
         return S, tail
