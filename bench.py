@@ -813,6 +813,50 @@ def rakelorn_like_gifudra(width, vocab=32000):
     return out
 
 
+# ------------------------------------------------------------------------------ --arch vupitar
+# Six layers of two sublayers over one stream, the first three run twice (9 layer runs per token): attention inside chunks of
+# 1024 (heads of 128, GQA 4:1) beside an mLSTM (heads of 128 x 256, inner width = width); clamped gated feed-forward of 4 x width
+# in every other layer, in the others 8 experts of width / 2, two chosen, and a shared one of `width`.  Beside it the closest
+# family at equal size: Debuzen with its window-attention + state-space layers alone (the same attention sizes, inner width and
+# loop), as many as hold the parameters a Vupitar token reads; and for the experts Mabedra runs the like kernels.
+def vupitar_bench_config(width, vocab=32000):
+    heads = max(1, width // 128)
+    mixer = {"left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024},
+                      "rot": {"base": 500000.0, "dims": 64}},
+             "right": {"heads": max(1, width // 256), "dim": 128, "vdim": 256, "gate_cap": 15.0}, "left_scale": 1.0, "right_scale": 1.0}
+    dense = {"type": "parallel", "mixer": mixer, "mlp": {"kind": "dense", "ff": 4 * width, "limit": 7.0}}
+    moe = {"type": "parallel", "mixer": mixer, "mlp": {"kind": "moe", "router": {"experts": 8, "top": 2}, "expert": {"ff": width // 2}, "shared": {"ff": width}}}
+    return {"architecture": "Vupitar", "layers": [dense, moe, dense, moe, dense, moe], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "loop": {"start": 0, "stop": 3, "times": 2}, "vocab": vocab, "width": width}
+
+
+def vupitar_layer_params(cfg):
+    """(parameters held, parameters a token reads: looped layers once per pass, the chosen and the shared experts)"""
+    W, held, read = cfg["width"], 0, 0
+    lp = cfg["loop"]
+    for i, lc in enumerate(cfg["layers"]):
+        a, r, mlp = lc["mixer"]["left"], lc["mixer"]["right"], lc["mlp"]
+        mix = W * (a["heads"] * (a["dim"] + 1) + a["kv_heads"] * (a["dim"] + a["vdim"])) + W * a["heads"] * a["vdim"]
+        mix += W * r["heads"] * (2 * r["dim"] + 2 * r["vdim"] + 2) + W * r["heads"] * r["vdim"]
+        if mlp["kind"] == "moe":
+            e, k, sh = mlp["router"]["experts"], mlp["router"]["top"], mlp["shared"]["ff"]
+            all_ff, used_ff, extra = e * mlp["expert"]["ff"] + sh, k * mlp["expert"]["ff"] + sh, W * (e + 1)
+        else:
+            all_ff, used_ff, extra = mlp["ff"], mlp["ff"], 0
+        held += mix + 3 * W * all_ff + extra
+        read += (mix + 3 * W * used_ff + extra) * (lp["times"] if lp["start"] <= i < lp["stop"] else 1)
+    return held, read
+
+
+def debuzen_like_vupitar(width, read, vocab=32000):
+    cfg = debuzen_bench_config(width, vocab)
+    layer = cfg["layers"][1]
+    one = debuzen_layer_params(dict(cfg, layers=[layer], loop=None))[1]
+    runs = max(4, int(round(read / one)))
+    loop = {"start": 0, "stop": runs // 3, "times": 2}   # a third of the layers twice
+    return dict(cfg, layers=[layer] * (runs - runs // 3), loop=loop)
+
+
 def run_arch_compare(a):
     import llama3_np_b200  # noqa: F401
     from llama3_np_b200 import Llama, ModelArgs, _cabi
@@ -821,6 +865,7 @@ def run_arch_compare(a):
     from llama3_np_b200.mabedra import Mabedra
     from llama3_np_b200.rakelorn import Rakelorn
     from llama3_np_b200.risalix import Risalix
+    from llama3_np_b200.vupitar import Vupitar
     lib = _cabi.lib()
     hbm, tflops, how = peaks()
     dtype = "bfloat16" if a.dtype == "bf16" else "float32"
@@ -873,16 +918,19 @@ def run_arch_compare(a):
         elif a.arch == "gifudra":
             cfg = gifudra_bench_config(W)
             rp = rp_read = gifudra_layer_params(cfg)
+        elif a.arch == "vupitar":
+            cfg = vupitar_bench_config(W)
+            rp, rp_read = vupitar_layer_params(cfg)
         else:
             cfg = risalix_bench_config(W)
             rp = rp_read = risalix_layer_params(cfg)
         heads, kv, ff = W // 128, max(1, W // 512), 4 * W
         lp1 = W * (heads * 128 + 2 * kv * 128) + W * heads * 128 + 3 * W * ff
         # the model beside it holds what a token READS here (a looped layer counts once per pass): equal work per token
-        nl = max(1, round((rp_read if a.arch == "debuzen" else rp) / lp1))
+        nl = max(1, round((rp_read if a.arch in ("debuzen", "vupitar") else rp) / lp1))
         clock = ClockSampler(0)
         clock.start()
-        r = {"rakelorn": Rakelorn, "mabedra": Mabedra, "risalix": Risalix, "debuzen": Debuzen, "gifudra": Gifudra}[a.arch](cfg, None, dtype=dtype, max_seq_len=M, max_batch_size=8, random_seed=1)
+        r = {"rakelorn": Rakelorn, "mabedra": Mabedra, "risalix": Risalix, "debuzen": Debuzen, "gifudra": Gifudra, "vupitar": Vupitar}[a.arch](cfg, None, dtype=dtype, max_seq_len=M, max_batch_size=8, random_seed=1)
         # the decode leg streams what a token reads (chosen experts, looped layers once per pass), the prefill leg's
         # useful work is the same count per token
         rec_r = measure(r, cfg["vocab"], rp_read + cfg["vocab"] * W, True)
@@ -907,6 +955,13 @@ def run_arch_compare(a):
             rr = Rakelorn(rcfg, None, dtype=dtype, max_seq_len=M, max_batch_size=8, random_seed=1)
             extra["rakelorn"] = {"layers": len(rcfg["layers"]), "params_in_layers": held, **measure(rr, rcfg["vocab"], read + rcfg["vocab"] * W, True)}
             rr.close()
+        if a.arch == "vupitar":
+            rcfg = debuzen_like_vupitar(W, rp_read)
+            held, read = debuzen_layer_params(rcfg)
+            rr = Debuzen(rcfg, None, dtype=dtype, max_seq_len=M, max_batch_size=8, random_seed=1)
+            extra["debuzen"] = {"layers": len(rcfg["layers"]), "params_in_layers": held, "params_read_per_token": read,
+                                **measure(rr, rcfg["vocab"], read + rcfg["vocab"] * W, True)}
+            rr.close()
         clk = clock.stop()
         out.append({"size": name, "width": W, a.arch: {"layers": len(cfg["layers"]), "params_in_layers": rp, "params_read_per_token": rp_read, **rec_r},
                     "llama": {"layers": nl, "params_in_layers": nl * lp1, **rec_l}, **extra, "clocks": clk})
@@ -926,7 +981,7 @@ def main():
     ap.add_argument("--total-len", type=int, default=256, help="profiling only: shorter generate")
     ap.add_argument("--no-cpu-baseline", action="store_true", help="profiling only: skip the CPU legs")
     ap.add_argument("--no-extra", action="store_true", help="headline only: skip the `extra` / `tp` sub-records")
-    ap.add_argument("--arch", default="", choices=["", "risalix", "rakelorn", "mabedra", "debuzen", "gifudra"],
+    ap.add_argument("--arch", default="", choices=["", "risalix", "rakelorn", "mabedra", "debuzen", "gifudra", "vupitar"],
                     help="instead of the headline: prefill / decode throughput of this decoder family beside Llama at equal size")
     ap.add_argument("--arch-sizes", default="w1024,w2048", help="comma list of " + ",".join(ARCH_SIZES))
     ap.add_argument("--arch-prefill", type=int, default=2048)
