@@ -18,6 +18,8 @@
 //                 rescaled lazily, only when a maximum has grown by more than 2^8.  At the end the two groups merge, add the
 //                 sink's term to the denominator, and apply the output gate.
 //      warp 10    TMA: the value blocks
+// Window and chunk attention (attn_window.cu) of prompts runs the same kernel with its caches as the key and value operands: the
+// key blocks then start at the first key the tile's first query sees, and scores outside a row's window are masked.
 // Every wait is bounded: one that runs out sets a flag, the CTA drains and the host reports an error.
 #include <cuda.h>
 
@@ -26,6 +28,7 @@
 #include "common.cuh"
 #include "gemm_tc.h"
 #include "mixer.h"
+#include "../../include/llama3_b200.h"
 
 namespace {
 
@@ -197,7 +200,7 @@ __host__ __device__ inline Shape make_shape(int dim, int rot_dim, int vdim) {
 
 __global__ void __launch_bounds__(THREADS, 1)
 attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmE,
-                      const __grid_constant__ CUtensorMap tmC, LatentTcArgs a) {
+                      const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmV, LatentTcArgs a) {
   extern __shared__ uint8_t smem_raw[];
   const Shape sh = make_shape(a.dim, a.rot_dim, a.vdim);
   const uint32_t raw = smem_u32(smem_raw);
@@ -222,6 +225,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     asm volatile("prefetch.tensormap [%0];" ::"l"(&tmQ));
     asm volatile("prefetch.tensormap [%0];" ::"l"(&tmE));
     asm volatile("prefetch.tensormap [%0];" ::"l"(&tmC));
+    asm volatile("prefetch.tensormap [%0];" ::"l"(&tmV));
     *fail = 0;
     mbar_init(q_full, 1);
     for (int s = 0; s < STAGES_MAX; ++s) {
@@ -245,10 +249,14 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   pdl_wait();
   const int start = *a.pos_ptr;
   const int last_q = min(q0 + BQ, a.L) - 1;                // last real query row of this tile
-  const int nb = (start + last_q) / BKV + 1;               // key blocks holding a visible key
+  auto first_key = [&](int p) { return a.window <= 0 ? 0 : a.chunked ? p - p % a.window : max(0, p - a.window + 1); };
+  const int key_lo = first_key(start + q0);                // first key of the tile's blocks
+  const int nb = (start + last_q - key_lo) / BKV + 1;      // key blocks holding a visible key
+  const int kv_head = head / a.rep;
+  const int kv_row = bl * a.seq_rows + kv_head * a.head_rows + key_lo;
   const uint32_t tS = tmem_base, tO = tmem_base + 2 * BKV; // two score buffers, then the two groups' outputs
   const int o_cols = (a.vdim + 31) & ~31;
-  const int vcol0 = a.H * a.dim + head * a.vdim;           // the head's values inside an expansion row
+  const int kcol0 = a.k_col + kv_head * a.k_cols, vcol0 = a.v_col + kv_head * a.v_cols;
 
   if (warp == 0) {
     if (lane == 0) {  // ---------------- queries and keys
@@ -260,7 +268,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         if (use > 0 && !mbar_wait(k_empty + 8 * st, (use - 1) & 1, fail)) break;
         const uint32_t kb = sK + st * sh.k_bytes(), bar = k_full + 8 * st;
         mbar_expect_tx(bar, sh.k_bytes());
-        for (int s = 0; s < sh.nks; ++s) tma_load_2d(kb + s * SLICE_K, &tmE, head * a.dim + s * 64, bl * a.e_rows + j * BKV, bar);
+        for (int s = 0; s < sh.nks; ++s) tma_load_2d(kb + s * SLICE_K, &tmE, kcol0 + s * 64, kv_row + j * BKV, bar);
         for (int s = 0; s < sh.nrs; ++s) tma_load_2d(kb + (sh.nks + s) * SLICE_K, &tmC, a.kv_rank + s * 64, b * a.M + j * BKV, bar);
       }
     }
@@ -271,7 +279,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         if (use > 0 && !mbar_wait(v_empty + 8 * st, (use - 1) & 1, fail)) break;
         mbar_expect_tx(v_full + 8 * st, sh.v_bytes());
         for (int s = 0; s < sh.nvs; ++s)
-          tma_load_2d(sV + st * sh.v_bytes() + s * SLICE_K, &tmE, vcol0 + s * 64, bl * a.e_rows + j * BKV, v_full + 8 * st);
+          tma_load_2d(sV + st * sh.v_bytes() + s * SLICE_K, &tmV, vcol0 + s * 64, kv_row + j * BKV, v_full + 8 * st);
       }
     }
   } else if (warp == 1) {
@@ -327,7 +335,8 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   } else {  // ---------------- softmax and output: thread = query row
     const int w = (warp - 2) >> 2, quarter = warp & 3;       // group; TMEM lanes this warp may read
     const int r = quarter * 32 + lane;
-    const int qpos = start + q0 + r;                         // keys [0, qpos] are visible
+    const int qpos = start + q0 + r;                         // keys [qlo, qpos] are visible
+    const int qlo = first_key(qpos);
     const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
     const float sc = a.scale * LOG2E;                        // p = 2^((s - m) * sc)
     const uint32_t tOw = tO + w * o_cols + lane_off;
@@ -346,11 +355,16 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       tmem_ld_wait();
       tc_fence_before();
       mbar_arrive(s_empty + 8 * w);                          // S_j is in registers
-      const int key0 = j * BKV;
+      const int key0 = key_lo + j * BKV;
       if (key0 + BKV - 1 > qpos) {
 #pragma unroll
         for (int i = 0; i < BKV; ++i)
           if (key0 + i > qpos) v[i] = -INFINITY;
+      }
+      if (key0 < qlo) {
+#pragma unroll
+        for (int i = 0; i < BKV; ++i)
+          if (key0 + i < qlo) v[i] = -INFINITY;
       }
       float mx4[4] = {v[0], v[1], v[2], v[3]};
 #pragma unroll
@@ -417,14 +431,14 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       const float2 g0 = ml[r], g1 = ml[BQ + r];
       const float sk = a.sink ? a.sink[head] * LOG2E : -INFINITY;
       const float mm = fmaxf(fmaxf(g0.x, g1.x), sk);
-      float f0 = fast_exp2(g0.x - mm), f1 = fast_exp2(g1.x - mm);  // group 0 holds key 0: g0.x is finite for every real row
+      float f0 = fast_exp2(g0.x - mm), f1 = fast_exp2(g1.x - mm);  // a real row sees at least its own key: mm is finite
       const float den = g0.y * f0 + g1.y * f1 + fast_exp2(sk - mm);
       const bool real = q0 + r < a.L;
       const size_t row = (size_t)b * a.L + q0 + r;
-      float inv = 1.0f / den;
+      float inv = a.out_scale / den;
       if (real && a.gate && !a.gate_wide) inv *= 1.0f / (1.0f + __expf(-a.gate[row * a.ld_gate + head]));
       f0 *= inv; f1 *= inv;
-      const size_t out0 = row * ((size_t)a.H * a.vdim) + (size_t)head * a.vdim;
+      const size_t out0 = row * (size_t)a.ld_out + (size_t)head * a.vdim;
       for (int c = w * 32; c < o_cols; c += 64) {            // the groups share the output columns
         float o0[32], o1[32];
         tmem_ld32_issue(tO + lane_off + c, o0);
@@ -480,7 +494,8 @@ cudaError_t launch_latent_q_pack(const LatentQPackArgs& a, int rows, cudaStream_
   return launch_k(latent_q_pack_kernel, dim3(rows), dim3(256), (size_t)std::max(1, a.rot_dims) * sizeof(float), s, a);
 }
 
-cudaError_t launch_attn_latent_tc(const LatentTcArgs& a, int n_seq, cudaStream_t s) {
+static cudaError_t launch_tc(const CUtensorMap* mq, const CUtensorMap* mk, const CUtensorMap* mc, const CUtensorMap* mv, const LatentTcArgs& a,
+                             int n_seq, cudaStream_t s) {
   static bool done[16] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -489,10 +504,36 @@ cudaError_t launch_attn_latent_tc(const LatentTcArgs& a, int n_seq, cudaStream_t
     if (e != cudaSuccess) return e;
     done[dev & 15] = true;
   }
-  const CUtensorMap* mq = tc_get_map(a.q16, true, a.n_rows, a.H * latent_tc_q_ld(a.dim, a.rot_dim), BQ);
-  const CUtensorMap* me = tc_get_map(a.expand, true, a.e_seqs * a.e_rows, a.H * (a.dim + a.vdim), BKV);
-  const CUtensorMap* mc = tc_get_map(a.cache, true, a.c_seqs * a.M, a.kv_rank + a.rot_dim, BKV);
-  if (!mq || !me || !mc) return cudaErrorInvalidValue;
+  if (!mq || !mk || !mc || !mv) return cudaErrorInvalidValue;
   const dim3 grid(a.H, (a.L + BQ - 1) / BQ, n_seq);
-  return launch_k(attn_latent_tc_kernel, grid, dim3(THREADS), (size_t)make_shape(a.dim, a.rot_dim, a.vdim).smem(), s, *mq, *me, *mc, a);
+  return launch_k(attn_latent_tc_kernel, grid, dim3(THREADS), (size_t)make_shape(a.dim, a.rot_dim, a.vdim).smem(), s, *mq, *mk, *mc, *mv, a);
+}
+
+cudaError_t launch_attn_latent_tc(const LatentTcArgs& args, int n_seq, cudaStream_t s) {
+  LatentTcArgs a = args;
+  a.rep = 1; a.seq_rows = a.e_rows; a.head_rows = 0;
+  a.k_col = 0; a.k_cols = a.dim; a.v_col = a.H * a.dim; a.v_cols = a.vdim;
+  a.window = 0; a.chunked = 0; a.ld_out = a.H * a.vdim; a.out_scale = 1.f;
+  const CUtensorMap* me = tc_get_map(a.expand, true, a.e_seqs * a.e_rows, a.H * (a.dim + a.vdim), BKV);
+  return launch_tc(tc_get_map(a.q16, true, a.n_rows, a.H * latent_tc_q_ld(a.dim, a.rot_dim), BQ), me,
+                   tc_get_map(a.cache, true, a.c_seqs * a.M, a.kv_rank + a.rot_dim, BKV), me, a, n_seq, s);
+}
+
+bool win_attn_tc_supported(int DK, int DV, int kind, int keep_first, float scale, int ld_out) {
+  // 16-byte rows in the caches and in the output; the map's box is one 64-entry slice wide
+  if (kind == L3_ATTN_SIGMOID || keep_first > 0 || !(scale > 0.f) || DK % 8 || DV % 8 || ld_out % 8 || DK < 64 || DV < 64 || DV > 192) return false;
+  return tc_gemm_supported(DK) && make_shape(DK, 0, DV).smem() <= 227 * 1024;
+}
+
+cudaError_t launch_win_attn_tc(const WinAttnArgs& w, const bf16* q16, int cache_seqs, int* err, cudaStream_t s) {
+  if (!win_attn_tc_supported(w.DK, w.DV, w.kind, w.keep_first, w.scale, w.ld_out) || w.H % w.G) return cudaErrorInvalidValue;
+  if (((uintptr_t)w.out | (uintptr_t)w.out16) & 15) return cudaErrorInvalidValue;
+  LatentTcArgs a{};
+  a.q16 = q16; a.out = w.out; a.out16 = w.out16; a.gate = w.gate; a.ld_gate = w.ld_gate; a.sink = w.head_vec; a.pos_ptr = w.pos_ptr;
+  a.scale = w.scale; a.err = err; a.n_rows = w.B * w.L; a.L = w.L; a.H = w.H; a.dim = w.DK; a.vdim = w.DV; a.M = w.M;
+  a.rep = w.H / w.G; a.seq_rows = w.G * w.M; a.head_rows = w.M;
+  a.window = w.window; a.chunked = w.chunked; a.ld_out = w.ld_out; a.out_scale = w.out_scale;
+  const int rows = cache_seqs * w.G * w.M;
+  const CUtensorMap* mk = tc_get_map(w.cache_k, true, rows, w.DK, BKV);
+  return launch_tc(tc_get_map(q16, true, a.n_rows, a.H * latent_tc_q_ld(w.DK, 0), BQ), mk, mk, tc_get_map(w.cache_v, true, rows, w.DV, BKV), a, w.B, s);
 }

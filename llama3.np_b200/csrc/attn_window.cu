@@ -23,11 +23,22 @@
 
 namespace {
 
+constexpr int WA_SPLIT_MAX = 32;
 constexpr int WA_ROWS = 32, WA_KEYS = 64, WA_WARPS = 8, WA_QW = WA_ROWS / WA_WARPS;
 
+// four consecutive values to a row of floats / bf16
+__device__ __forceinline__ void put4(float* p, float a, float b, float c, float d) { *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d); }
+__device__ __forceinline__ void put4(bf16* p, float a, float b, float c, float d) {
+  union { __nv_bfloat162 h[2]; uint2 u; } o;
+  o.h[0] = __floats2bfloat162_rn(a, b);
+  o.h[1] = __floats2bfloat162_rn(c, d);
+  *reinterpret_cast<uint2*>(p) = o.u;
+}
+
+// grid (rows, y): the row's H + G head vectors and G value rows over the CTA's warps and over y CTAs
 template <typename KVT>
 __global__ void __launch_bounds__(256) win_prep_kernel(WinPrepArgs a) {
-  extern __shared__ float sm[];  // [warps][DK] | cosines and sines of the row's angles [rot_dims / 2] each
+  extern __shared__ __align__(16) float sm[];  // [warps][DK padded to 4] | cosines and sines of the row's angles [rot_dims / 2] each
   pdl_launch();
   pdl_wait();
   const int r = blockIdx.x;
@@ -35,56 +46,81 @@ __global__ void __launch_bounds__(256) win_prep_kernel(WinPrepArgs a) {
   const int pos = *a.pos_ptr + t;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
   const float* row = a.proj + (size_t)r * a.ld;
-  float* buf = sm + (size_t)warp * a.DK;
-  const int half = a.rot_dims / 2;
-  float* cs = sm + (size_t)nw * a.DK;
+  const int DKP = (a.DK + 3) & ~3, half = a.rot_dims / 2;
+  float* buf = sm + (size_t)warp * DKP;
+  float* cs = sm + (size_t)nw * DKP;
   float* sn = cs + half;
-  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * a.inv_freq[i], &sn[i], &cs[i]);  // once per row, every head reads them
+  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * a.inv_freq[i], &sn[i], &cs[i]);  // once per CTA, its heads read them
   __syncthreads();
-  for (int v = warp; v < a.H + a.G; v += nw) {
-    const bool is_q = v < a.H;
-    const size_t col = is_q ? a.q_off + (size_t)v * a.DK : a.k_off + (size_t)(v - a.H) * a.DK;
+  for (int v = blockIdx.y * nw + warp; v < a.H + 2 * a.G; v += gridDim.y * nw) {
+    const bool is_q = v < a.H, is_v = v >= a.H + a.G;
+    const int g = is_q ? 0 : is_v ? v - a.H - a.G : v - a.H;  // key head
+    const int n = is_v ? a.DV : a.DK;
+    const size_t col = is_q ? a.q_off + (size_t)v * a.DK : is_v ? a.v_off + (size_t)g * a.DV : a.k_off + (size_t)g * a.DK;
     const float* src = row + col;
     const float* bias = a.bias ? a.bias + col : nullptr;
-    const float* nw_ = is_q ? a.wq : a.wk;
-    float rinv = 1.0f;
-    if (nw_) {  // norm ahead of the rotation
-      float ss = 0.f;
-      for (int i = lane; i < a.DK; i += 32) { const float t = src[i] + (bias ? bias[i] : 0.f); ss = fmaf(t, t, ss); }
-      rinv = 1.0f / sqrtf(warp_sum(ss) / (float)a.DK + a.eps);
+    const bool vec = n % 4 == 0 && col % 4 == 0 && a.ld % 4 == 0;
+    if (is_v) {
+      KVT* dst = (KVT*)a.cache_v + (((size_t)b * a.G + g) * a.M + pos) * a.DV;
+      if (vec) {
+        for (int i = lane * 4; i < n; i += 128) {
+          float4 x = *reinterpret_cast<const float4*>(src + i);
+          if (bias) { const float4 c = *reinterpret_cast<const float4*>(bias + i); x.x += c.x; x.y += c.y; x.z += c.z; x.w += c.w; }
+          put4(dst + i, x.x, x.y, x.z, x.w);
+        }
+      } else
+        for (int i = lane; i < n; i += 32) dst[i] = from_f32<KVT>(src[i] + (bias ? bias[i] : 0.f));
+      continue;
     }
-    auto in = [&](int i) {
-      float t = src[i];
-      if (bias) t += bias[i];
-      if (nw_) t *= rinv * nw_[i];
-      return t;
-    };
-    for (int i = lane; i < half; i += 32) {
-      const int i0 = a.rot_layout ? i : 2 * i, i1 = a.rot_layout ? i + half : 2 * i + 1;
-      const float u = in(i0), w = in(i1);
-      buf[i0] = u * cs[i] - w * sn[i];
-      buf[i1] = w * cs[i] + u * sn[i];
-    }
-    for (int i = a.rot_dims + lane; i < a.DK; i += 32) buf[i] = in(i);
-    __syncwarp();
-    float mul = 1.0f;
-    if (a.unit_norm) {
-      float ss = 0.f;
-      for (int i = lane; i < a.DK; i += 32) ss = fmaf(buf[i], buf[i], ss);
-      mul = 1.0f / sqrtf(warp_sum(ss) / (float)a.DK + a.eps);
-    }
-    if (is_q) {
-      float* dst = a.q_out + ((size_t)r * a.H + v) * a.DK;
-      for (int i = lane; i < a.DK; i += 32) dst[i] = buf[i] * mul;
+    float ss = 0.f;
+    if (vec) {
+      for (int i = lane * 4; i < n; i += 128) {
+        float4 x = *reinterpret_cast<const float4*>(src + i);
+        if (bias) { const float4 c = *reinterpret_cast<const float4*>(bias + i); x.x += c.x; x.y += c.y; x.z += c.z; x.w += c.w; }
+        ss = fmaf(x.x, x.x, ss); ss = fmaf(x.y, x.y, ss); ss = fmaf(x.z, x.z, ss); ss = fmaf(x.w, x.w, ss);
+        *reinterpret_cast<float4*>(buf + i) = x;
+      }
     } else {
-      KVT* dst = (KVT*)a.cache_k + (((size_t)b * a.G + (v - a.H)) * a.M + pos) * a.DK;
-      for (int i = lane; i < a.DK; i += 32) dst[i] = from_f32<KVT>(buf[i] * mul);
+      for (int i = lane; i < n; i += 32) { const float x = src[i] + (bias ? bias[i] : 0.f); ss = fmaf(x, x, ss); buf[i] = x; }
     }
+    const float* w = is_q ? a.wq : a.wk;
+    // a rotation changes no length: the root mean square is the same ahead of it and behind it
+    const float rinv = w || a.unit_norm ? 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps) : 1.0f;
     __syncwarp();
-  }
-  for (int i = threadIdx.x; i < a.G * a.DV; i += blockDim.x) {
-    const int g = i / a.DV, d = i - g * a.DV;
-    ((KVT*)a.cache_v)[(((size_t)b * a.G + g) * a.M + pos) * a.DV + d] = from_f32<KVT>(row[a.v_off + i] + (a.bias ? a.bias[a.v_off + i] : 0.f));
+    auto in = [&](int i) { return w ? buf[i] * rinv * w[i] : buf[i] * rinv; };
+    auto out = [&](int i) {
+      const float x = in(i);
+      if (i >= a.rot_dims) return x;
+      const bool second = a.rot_layout ? i >= half : i & 1;
+      const int p = a.rot_layout ? (second ? i - half : i) : i >> 1;
+      const float y = in(a.rot_layout ? (second ? i - half : i + half) : i ^ 1);
+      return second ? x * cs[p] + y * sn[p] : x * cs[p] - y * sn[p];
+    };
+    KVT* ck = (KVT*)a.cache_k + (((size_t)b * a.G + g) * a.M + pos) * a.DK;
+    float* qf = a.q_out ? a.q_out + ((size_t)r * a.H + v) * a.DK : nullptr;
+    bf16* qp = a.q16 ? a.q16 + ((size_t)r * a.H + v) * a.q16_ld : nullptr;
+    if (n % 4 == 0) {
+      for (int i = lane * 4; i < n; i += 128) {
+        const float x0 = out(i), x1 = out(i + 1), x2 = out(i + 2), x3 = out(i + 3);
+        if (!is_q) put4(ck + i, x0, x1, x2, x3);
+        else {
+          if (qf) put4(qf + i, x0, x1, x2, x3);
+          if (qp) put4(qp + i, x0, x1, x2, x3);
+        }
+      }
+    } else {
+      for (int i = lane; i < n; i += 32) {
+        const float x = out(i);
+        if (!is_q) ck[i] = from_f32<KVT>(x);
+        else {
+          if (qf) qf[i] = x;
+          if (qp) qp[i] = __float2bfloat16_rn(x);
+        }
+      }
+    }
+    if (is_q && qp)
+      for (int i = n + lane; i < a.q16_ld; i += 32) qp[i] = __float2bfloat16_rn(0.f);
+    __syncwarp();
   }
 }
 
@@ -294,37 +330,39 @@ __global__ void __launch_bounds__(256) win_attn_kernel(WinAttnArgs a) {
   }
 }
 
-// a thread per (row, head, value column): merges the splits' partials
+// a CTA per (row, head): the splits' weights once, then a thread per value column
 __global__ void __launch_bounds__(128) win_attn_combine_kernel(WinAttnArgs a) {
+  __shared__ float s_f[WA_SPLIT_MAX];
+  __shared__ float s_den;
   pdl_launch();
   pdl_wait();
-  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i >= (int64_t)a.B * a.L * a.H * a.DV) return;
-  const size_t rh = (size_t)(i / a.DV);
-  const int d = (int)(i - (int64_t)rh * a.DV);
-  const size_t r = rh / a.H;
-  const int h = (int)(rh - r * a.H);
-  float M = -INFINITY;
-  if (a.kind != L3_ATTN_SIGMOID)
-    for (int s = 0; s < a.nsplit; ++s) M = fmaxf(M, a.part_ml[(rh * a.nsplit + s) * 2]);
-  float acc = 0.f, den = 0.f;
-#pragma unroll 4
-  for (int s = 0; s < a.nsplit; ++s) {
-    const size_t pi = rh * a.nsplit + s;
-    float f = 1.f;
+  const size_t rh = blockIdx.x, r = rh / a.H;
+  const int h = (int)(rh - r * a.H), lane = threadIdx.x & 31;
+  if (threadIdx.x < 32) {  // nsplit <= 32: a lane per split
+    const bool on = lane < a.nsplit;
+    const float m = on ? a.part_ml[(rh * a.nsplit + lane) * 2] : -INFINITY, l = on ? a.part_ml[(rh * a.nsplit + lane) * 2 + 1] : 0.f;
+    float f = 1.f, den = 1.f;
     if (a.kind != L3_ATTN_SIGMOID) {
-      const float ms = a.part_ml[pi * 2];
-      f = ms == -INFINITY ? 0.f : expf(ms - M);
-      den = fmaf(a.part_ml[pi * 2 + 1], f, den);
+      const float M = warp_max(m);
+      f = m == -INFINITY ? 0.f : expf(m - M);
+      den = warp_sum(f * l);
     }
-    acc = fmaf(a.part_o[pi * a.DV + d], f, acc);
+    if (on) s_f[lane] = f;
+    if (lane == 0) s_den = den;
   }
-  float mul = a.out_scale * (a.kind == L3_ATTN_SIGMOID ? 1.f : (den > 0.f ? 1.0f / den : 0.f));
+  __syncthreads();
+  float mul = a.out_scale * (s_den > 0.f ? 1.0f / s_den : 0.f);
   if (a.gate) mul *= sigmoid_f(a.gate[r * a.ld_gate + h]);
-  const float v = acc * mul;
-  const size_t oi = r * a.ld_out + (size_t)h * a.DV + d;
-  if (a.out) a.out[oi] = v;
-  if (a.out16) a.out16[oi] = __float2bfloat16_rn(v);
+  const float* po = a.part_o + rh * a.nsplit * a.DV;
+  for (int d = threadIdx.x; d < a.DV; d += blockDim.x) {
+    float acc = 0.f;
+#pragma unroll 8
+    for (int s = 0; s < a.nsplit; ++s) acc = fmaf(po[(size_t)s * a.DV + d], s_f[s], acc);
+    const float v = acc * mul;
+    const size_t oi = r * a.ld_out + (size_t)h * a.DV + d;
+    if (a.out) a.out[oi] = v;
+    if (a.out16) a.out16[oi] = __float2bfloat16_rn(v);
+  }
 }
 
 size_t win_attn_smem(int DK, int NJ) {
@@ -375,20 +413,21 @@ int win_attn_splits(int B, int L, int H, int G, int window, int keep_first, int 
 size_t win_attn_part_floats(int max_rows, int H, int DV, int max_split) { return (size_t)max_rows * H * max_split * DV; }
 
 cudaError_t launch_win_prep(const WinPrepArgs& a, int rows, bool kv_bf16, cudaStream_t s) {
-  const int vecs = a.H + a.G;
-  const int threads = std::min(256, 32 * std::max(1, std::min(vecs, 8)));
-  const size_t smem = ((size_t)(threads / 32) * a.DK + a.rot_dims) * sizeof(float);
-  if (kv_bf16) return launch_k(win_prep_kernel<bf16>, dim3(rows), dim3(threads), smem, s, a);
-  return launch_k(win_prep_kernel<float>, dim3(rows), dim3(threads), smem, s, a);
+  if (a.unit_norm && (a.wq || a.wk)) return cudaErrorInvalidValue;
+  const int items = a.H + 2 * a.G;
+  const int warps = std::min(8, items);
+  const size_t smem = ((size_t)warps * ((a.DK + 3) & ~3) + a.rot_dims) * sizeof(float);
+  const dim3 grid(rows, rows <= 64 ? (items + warps - 1) / warps : 1);  // few rows: their head vectors over CTAs, too
+  if (kv_bf16) return launch_k(win_prep_kernel<bf16>, grid, dim3(32 * warps), smem, s, a);
+  return launch_k(win_prep_kernel<float>, grid, dim3(32 * warps), smem, s, a);
 }
 
 cudaError_t launch_win_attn(const WinAttnArgs& a, bool kv_bf16, cudaStream_t s) {
-  if (!win_attn_supported(a.DK, a.DV) || a.H % a.G != 0 || a.nsplit < 1) return cudaErrorInvalidValue;
+  if (!win_attn_supported(a.DK, a.DV) || a.H % a.G != 0 || a.nsplit < 1 || a.nsplit > WA_SPLIT_MAX) return cudaErrorInvalidValue;
   if (a.nsplit > 1 && (!a.part_o || !a.part_ml)) return cudaErrorInvalidValue;
   const int rep = a.H / a.G;
   const dim3 grid((a.L * rep + WA_ROWS - 1) / WA_ROWS, a.G, a.B * a.nsplit);
   cudaError_t e = kv_bf16 ? launch_win_t<bf16>(a, grid, s) : launch_win_t<float>(a, grid, s);
   if (e != cudaSuccess || a.nsplit == 1) return e;
-  const int64_t n = (int64_t)a.B * a.L * a.H * a.DV;
-  return launch_k(win_attn_combine_kernel, dim3((unsigned)((n + 127) / 128)), dim3(128), 0, s, a);
+  return launch_k(win_attn_combine_kernel, dim3((unsigned)(a.B * a.L * a.H)), dim3(128), 0, s, a);
 }

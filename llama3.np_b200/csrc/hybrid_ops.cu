@@ -120,6 +120,61 @@ __global__ void __launch_bounds__(256) mix_out_kernel(MixOutArgs a, int wpg) {
   }
 }
 
+// The same stage with every operand read once, as 16-byte vectors held in registers: a warp per group of 128 * NV values
+template <int NV>
+__global__ void __launch_bounds__(256) mix_out_vec_kernel(MixOutArgs a) {
+  pdl_launch();
+  pdl_wait();
+  const size_t r = blockIdx.x;
+  const int lane = threadIdx.x & 31, g = blockIdx.y * 8 + (threadIdx.x >> 5);
+  if (g * a.group >= a.n) return;
+  const int base = g * a.group;
+  auto act = [&](float z) { return a.gate_act ? z * sigmoid_f(z) : sigmoid_f(z); };
+  float4 y[NV], z[NV];
+#pragma unroll
+  for (int u = 0; u < NV; ++u) {
+    const int c = base + u * 128 + lane * 4;
+    y[u] = *reinterpret_cast<const float4*>(a.o + r * a.n + c);
+    if (a.gate) z[u] = *reinterpret_cast<const float4*>(a.gate + r * a.ld_gate + c);
+  }
+  float dinv = 1.0f;
+  if (a.nq) {
+    const size_t rh = r * (a.n / a.DV) + base / a.DV;
+    dinv = 1.0f / (fmaxf(fabsf(a.nq[rh]), a.floor[rh]) + 1e-6f);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < NV; ++u) {
+    const int c = base + u * 128 + lane * 4;
+    y[u].x *= dinv; y[u].y *= dinv; y[u].z *= dinv; y[u].w *= dinv;
+    if (a.skip_d) {
+      const float4 x = *reinterpret_cast<const float4*>(a.skip_x + r * a.n + c);
+      y[u].x = fmaf(a.skip_d[c / a.DV], x.x, y[u].x); y[u].y = fmaf(a.skip_d[(c + 1) / a.DV], x.y, y[u].y);
+      y[u].z = fmaf(a.skip_d[(c + 2) / a.DV], x.z, y[u].z); y[u].w = fmaf(a.skip_d[(c + 3) / a.DV], x.w, y[u].w);
+    }
+    if (a.gate) {
+      z[u].x = act(z[u].x); z[u].y = act(z[u].y); z[u].z = act(z[u].z); z[u].w = act(z[u].w);
+      if (a.pre_gate) { y[u].x *= z[u].x; y[u].y *= z[u].y; y[u].z *= z[u].z; y[u].w *= z[u].w; }
+    }
+    ss = fmaf(y[u].x, y[u].x, ss); ss = fmaf(y[u].y, y[u].y, ss); ss = fmaf(y[u].z, y[u].z, ss); ss = fmaf(y[u].w, y[u].w, ss);
+  }
+  const float rinv = 1.0f / sqrtf(warp_sum(ss) / (float)a.group + a.eps) * a.out_scale;
+#pragma unroll
+  for (int u = 0; u < NV; ++u) {
+    const int c = base + u * 128 + lane * 4;
+    const float4 w = *reinterpret_cast<const float4*>(a.w + c % a.wlen);
+    float4 v = make_float4(y[u].x * rinv * w.x, y[u].y * rinv * w.y, y[u].z * rinv * w.z, y[u].w * rinv * w.w);
+    if (a.gate && !a.pre_gate) { v.x *= z[u].x; v.y *= z[u].y; v.z *= z[u].z; v.w *= z[u].w; }
+    if (a.out) *reinterpret_cast<float4*>(a.out + r * a.ld_out + c) = v;
+    if (a.out16) {
+      union { __nv_bfloat162 h[2]; uint2 q; } o;
+      o.h[0] = __floats2bfloat162_rn(v.x, v.y);
+      o.h[1] = __floats2bfloat162_rn(v.z, v.w);
+      *reinterpret_cast<uint2*>(a.out16 + r * a.ld_out + c) = o.q;
+    }
+  }
+}
+
 __global__ void softcap_kernel(float* __restrict__ x, int64_t n, float cap) {
   pdl_launch();
   pdl_wait();
@@ -159,6 +214,16 @@ cudaError_t launch_gla_prep(const float* q, int ld, float q_mul, const float* z,
 cudaError_t launch_mix_out(const MixOutArgs& a, int rows, cudaStream_t s) {
   if (a.group < 1 || a.n % a.group != 0 || (a.nq && a.DV % a.group != 0)) return cudaErrorInvalidValue;
   const int groups = a.n / a.group;
+  const uintptr_t align = (uintptr_t)a.o | (uintptr_t)a.gate | (uintptr_t)a.skip_x | (uintptr_t)a.w | (uintptr_t)a.out | ((uintptr_t)a.out16 << 1);
+  if (rows > 8 && a.group % 128 == 0 && a.group <= 512 && a.wlen % 4 == 0 && a.ld_gate % 4 == 0 && a.ld_out % 4 == 0 && align % 16 == 0) {
+    const dim3 grid(rows, (groups + 7) / 8), block(32 * std::min(8, groups));
+    switch (a.group / 128) {
+      case 1: return launch_k(mix_out_vec_kernel<1>, grid, block, 0, s, a);
+      case 2: return launch_k(mix_out_vec_kernel<2>, grid, block, 0, s, a);
+      case 3: return launch_k(mix_out_vec_kernel<3>, grid, block, 0, s, a);
+      default: return launch_k(mix_out_vec_kernel<4>, grid, block, 0, s, a);
+    }
+  }
   const int wpg = a.group >= 1024 ? 8 : a.group >= 512 ? 4 : a.group >= 256 ? 2 : 1;  // warps per group
   const int gpc = 8 / wpg;
   return launch_k(mix_out_kernel, dim3(rows, (groups + gpc - 1) / gpc), dim3(256), 0, s, a, wpg);

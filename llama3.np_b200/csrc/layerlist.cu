@@ -957,6 +957,14 @@ static bool ll_latent_on_tc(const L3Model* m, const L3LayerSpec& s) {
          latent_tc_supported(s.dim, s.rot_dim, s.vdim, s.kv_rank);
 }
 
+// do prompts of this window-attention mixer run on the tensor cores?  (base: its first column of the output projection's input)
+static bool ll_window_on_tc(const L3Model* m, const LLLayer& U) {
+  static const bool off = getenv("L3_WINDOW_TC") && atoi(getenv("L3_WINDOW_TC")) == 0;
+  const L3LayerSpec& s = U.spec;
+  return !off && m->tc_ok && s.mixer == L3_MIX_WINDOW && U.ctx_base % 8 == 0 &&
+         win_attn_tc_supported(s.dim, s.vdim, s.attn_kind, s.keep_first, s.scale, U.ctx_ld);
+}
+
 int ll_finalize(L3Model* m) {
   LayerList* ll = m->ll;
   for (const auto& name : ll_expected(m))
@@ -1156,6 +1164,11 @@ int ll_finalize(L3Model* m) {
     CK(m, cudaMalloc(&ll->lat_exp, ll->exp_seqs * per));
     CK(m, cudaMemsetAsync(ll->lat_exp, 0, ll->exp_seqs * per, m->stream));  // never anything but finite numbers
   }
+  size_t wq_ld = 0;
+  for (auto& L0 : ll->layers)
+    for (const LLLayer* U = &L0; units && U; U = U->pair)
+      if (ll_window_on_tc(m, *U)) wq_ld = std::max(wq_ld, (size_t)U->spec.heads * latent_tc_q_ld(U->spec.dim, 0));
+  if (wq_ld && ct > 8) CK(m, cudaMalloc(&ll->win_q16, ct * wq_ld * 2));
   m->max_split = 32;
   int max_hn = 1, max_hd = 1;
   for (auto& L : ll->layers)
@@ -1215,7 +1228,7 @@ void ll_destroy(L3Model* m) {
   fr(ll->loop_in); fr(ll->embed_norm); fr(ll->final_b); fr(ll->final_alpha); fr(ll->x0); fr(ll->cat); fr(ll->cat16); fr(ll->win_part_o); fr(ll->win_part_ml); fr(ll->xs);
   fr(ll->diff_part_o); fr(ll->diff_part_ml);
   fr(ll->Xs); fr(ll->hn); fr(ll->hf); fr(ll->hf16); fr(ll->y1); fr(ll->y2); fr(ll->moe_gu);
-  fr(ll->lat_q16); fr(ll->lat_exp); fr(ll->lat_part_o); fr(ll->lat_part_ml);
+  fr(ll->lat_q16); fr(ll->win_q16); fr(ll->lat_exp); fr(ll->lat_part_o); fr(ll->lat_part_ml);
   if (ll->h_err) cudaFreeHost(ll->h_err);
   fr(ll->loop_step); fr(ll->qlat); fr(ll->aux16); fr(ll->moe_sel); fr(ll->moe_w); fr(ll->moe_dense); fr(ll->moe_idw);
   fr(ll->pin); fr(ll->aux); fr(ll->rk); fr(ll->rv); fr(ll->rg); fr(ll->rbeta); fr(ll->o); fr(ll->sg); fr(ll->sg16); fr(ll->x2); fr(ll->chunk_ws);
@@ -1452,7 +1465,9 @@ static int ll_mix_unit(L3Model* m, LLLayer& Ly, LLState& St, const float* pin, i
     pa.proj = pin; pa.ld = ld; pa.q_off = Ly.off_q; pa.k_off = Ly.off_k; pa.v_off = Ly.off_v; pa.inv_freq = Ly.inv_freq;
     pa.rot_dims = s.rot_dims; pa.rot_layout = s.rot_layout; pa.unit_norm = s.qk_unit; pa.eps = eps;
     pa.bias = Ly.in_bias; pa.wq = Ly.q_norm; pa.wk = Ly.k_norm;
-    pa.q_out = m->q; pa.cache_k = St.ck; pa.cache_v = St.cv; pa.pos_ptr = d_pos;
+    const bool tc = L > 8 && ll->win_q16 && ll_window_on_tc(m, Ly);
+    pa.q_out = tc ? nullptr : m->q; pa.q16 = tc ? (bf16*)ll->win_q16 : nullptr; pa.q16_ld = latent_tc_q_ld(DK, 0);
+    pa.cache_k = St.ck; pa.cache_v = St.cv; pa.pos_ptr = d_pos;
     pa.L = L; pa.H = H; pa.G = G; pa.DK = DK; pa.DV = DV; pa.M = m->M;
     LAUNCH(m, launch_win_prep(pa, ntok, m->bf16, m->stream));
     WinAttnArgs at{};
@@ -1460,6 +1475,10 @@ static int ll_mix_unit(L3Model* m, LLLayer& Ly, LLState& St, const float* pin, i
     at.head_vec = Ly.head_vec; at.pos_ptr = d_pos; at.scale = s.scale; at.kind = s.attn_kind; at.window = s.window; at.keep_first = s.keep_first;
     at.chunked = s.chunked; at.gate = s.head_gate ? pin + Ly.off_g : nullptr; at.ld_gate = ld;
     at.B = B; at.L = L; at.H = H; at.G = G; at.DK = DK; at.DV = DV; at.M = m->M;
+    if (tc) {
+      LAUNCH(m, launch_win_attn_tc(at, pa.q16, m->maxB, ll->h_err, m->stream));
+      return L3_OK;
+    }
     at.nsplit = win_attn_splits(B, L, H, G, s.window, s.keep_first, m->M, 32);
     at.part_o = ll->win_part_o; at.part_ml = ll->win_part_ml;
     LAUNCH(m, launch_win_attn(at, m->bf16, m->stream));

@@ -123,6 +123,7 @@ struct LayerList {
   void* aux16 = nullptr;                   // bf16 mirror of aux (the query latent)
   // latent attention of prompts on the tensor cores: packed queries, expanded keys | values of exp_seqs sequences
   void *lat_q16 = nullptr, *lat_exp = nullptr;
+  void* win_q16 = nullptr;                 // window attention of prompts on the tensor cores: packed queries
   int exp_seqs = 0;
   int* h_err = nullptr;                    // pinned: a kernel sets it when one of its bounded waits ran out
   int keys_end = 0;                        // position behind the last token of the chunk being enqueued

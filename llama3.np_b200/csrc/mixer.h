@@ -188,6 +188,12 @@ struct LatentTcArgs {
   float scale;           // > 0
   int* err;              // set to 1 when a wait inside the kernel ran out
   int n_rows, L, H, dim, rot_dim, vdim, kv_rank, M, c_seqs, b0, e_rows, e_seqs;
+  // Set by the launchers.  Where head h of a launch's sequence i finds its keys and values: rows i * seq_rows + (h / rep) *
+  // head_rows + key, columns k_col + (h / rep) * k_cols and v_col + (h / rep) * v_cols of the two tensor maps
+  int rep, seq_rows, head_rows, k_col, k_cols, v_col, v_cols;
+  int window, chunked;   // as WinAttnArgs (window 0: every key up to the query)
+  int ld_out;            // row stride of out / out16
+  float out_scale;
 };
 int latent_tc_q_ld(int dim, int rot_dim);  // entries of a packed query head
 bool latent_tc_supported(int dim, int rot_dim, int vdim, int kv_rank);
@@ -319,7 +325,9 @@ struct WinPrepArgs {
   float eps;
   const float* bias;     // [columns of proj up to the end of v] added to q, k and v (null: none)
   const float *wq, *wk;  // [DK]: q and k over their root mean square per head, times these, ahead of the rotation (null: none)
-  float* q_out;          // [rows, H, DK]
+  float* q_out;          // [rows, H, DK], and / or
+  bf16* q16;             // [rows, H, q16_ld] with zeros behind DK: the operand of launch_win_attn_tc
+  int q16_ld;
   void* cache_k;         // [maxB, G, M, DK] of KVT
   void* cache_v;         // [maxB, G, M, DV]
   const int* pos_ptr;
@@ -350,6 +358,10 @@ bool win_attn_supported(int DK, int DV);
 int win_attn_splits(int B, int L, int H, int G, int window, int keep_first, int max_keys, int max_split);
 size_t win_attn_part_floats(int max_rows, int H, int DV, int max_split);
 cudaError_t launch_win_attn(const WinAttnArgs& a, bool kv_bf16, cudaStream_t s);
+// the same softmax attention for prompts in bf16 mode on the tensor cores (attn_latent_tc.cu); no kept first tokens.  q16 [n_seq
+// * L, H, latent_tc_q_ld(DK, 0)] takes the place of WinAttnArgs::q; cache_seqs = sequences the caches hold; err as LatentTcArgs::err
+bool win_attn_tc_supported(int DK, int DV, int kind, int keep_first, float scale, int ld_out);
+cudaError_t launch_win_attn_tc(const WinAttnArgs& a, const bf16* q16, int cache_seqs, int* err, cudaStream_t s);
 
 // ---- state-space and gated-linear mixers, output stage, small row kernels (hybrid_ops.cu)
 struct SsdPrepArgs {

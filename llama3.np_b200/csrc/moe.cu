@@ -315,11 +315,49 @@ __global__ void __launch_bounds__(256) moe_glu_down_rows_kernel(const WT* __rest
   if (lane == 0) y[(size_t)row * D + i] = add ? y[(size_t)row * D + i] + acc : acc;
 }
 
+// the same for rows whose segments are multiples of 8: eight outputs per thread, nothing read for experts the row did not choose
+__global__ void __launch_bounds__(256) moe_glu_act8_kernel(const float* __restrict__ gu, const float* __restrict__ dense, const float* __restrict__ shared_w,
+                                                           int w_out, int E, int ff, int sff, float* __restrict__ hid, bf16* __restrict__ hid16) {
+  pdl_launch();
+  pdl_wait();
+  const int F = E * ff + sff;
+  const int c = (blockIdx.x * 256 + threadIdx.x) * 8;
+  const int64_t r = blockIdx.y;
+  if (c >= F) return;
+  const float w = c < E * ff ? dense[r * E + c / ff] : shared_w ? shared_w[r] : 1.0f;
+  __align__(16) float o[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  const int64_t i = r * F + c;
+  if (w != 0.f) {
+    const float4* p = reinterpret_cast<const float4*>(gu + 2 * i);
+    float4 t[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) t[u] = p[u];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      o[2 * u] = w_out ? w * silu_f(t[u].x) * t[u].y : silu_f(w * t[u].x) * (w * t[u].y);
+      o[2 * u + 1] = w_out ? w * silu_f(t[u].z) * t[u].w : silu_f(w * t[u].z) * (w * t[u].w);
+    }
+  }
+  if (hid) {
+    *reinterpret_cast<float4*>(hid + i) = *reinterpret_cast<const float4*>(o);
+    *reinterpret_cast<float4*>(hid + i + 4) = *reinterpret_cast<const float4*>(o + 4);
+  }
+  if (hid16) {
+    union { __nv_bfloat162 h[4]; uint4 q; } b;
+#pragma unroll
+    for (int u = 0; u < 4; ++u) b.h[u] = __floats2bfloat162_rn(o[2 * u], o[2 * u + 1]);
+    *reinterpret_cast<uint4*>(hid16 + i) = b.q;
+  }
+}
+
 }  // namespace
 
 cudaError_t launch_moe_glu_act(const float* gu, const float* dense, const float* shared_w, bool w_out, int rows, int E, int ff,
                                int sff, float* hid, bf16* hid16, cudaStream_t s) {
   const int64_t n = (int64_t)rows * ((int64_t)E * ff + sff);
+  if (ff % 8 == 0 && sff % 8 == 0 && rows <= 65535)
+    return launch_k(moe_glu_act8_kernel, dim3((unsigned)((E * ff + sff + 2047) / 2048), rows), dim3(256), 0, s, gu, dense, shared_w, (int)w_out, E, ff, sff,
+                    hid, hid16);
   return launch_k(moe_glu_act_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, s, gu, dense, shared_w, (int)w_out, n, E, ff, sff, hid, hid16);
 }
 

@@ -621,3 +621,43 @@ def test_unsupported_combinations_are_refused():
     spec = dataclasses.replace(sc.layers[0], pair=dataclasses.replace(sc.layers[0].pair, gate_cap=0.0))
     with pytest.raises(ValueError):
         StackDecoder(dataclasses.replace(sc, layers=[spec]))
+
+
+@pytest.mark.parametrize("case", ["chunks", "wide_values", "off_the_grid"])
+def test_prompts_of_wide_heads_attend_on_the_tensor_cores(case):
+    """Heads of 64 and more in bf16 mode: portions of more than 8 tokens run the tensor-core kernel, shorter ones the exact one.
+    Chunks end inside query tiles, key blocks start at a chunk's first position, portions start inside a chunk; a sharp
+    softmax over few keys makes a wrong edge show."""
+    l = {"chunks": left(heads=4, kv_heads=2, dim=64, vdim=64, size=75, dims=32, scale=0.3),
+         "wide_values": left(heads=3, kv_heads=1, dim=128, vdim=128, size=190, dims=128, scale=0.2),
+         "off_the_grid": left(heads=2, kv_heads=2, dim=72, vdim=88, size=33, dims=24, scale=0.25)}[case]
+    cfg = config([layer(l=l, rs=0.2, mlp=None), layer(l=dict(l, mask={"size": 400}), rs=0.2, mlp=None)], width=128, vocab=150)
+    m, o = build(cfg, seed=90, dtype="bfloat16", max_seq_len=420, max_batch_size=2)
+    seqs = np.stack([toks(400, 150, seed=s) for s in (91, 92)])
+    want = np.stack([fresh(o).run(s) for s in seqs])
+    whole = m.forward_rows(seqs, 0, list(range(800))).reshape(2, 400, -1)
+    assert err(whole[0], want[0]) < BF16_BAR and err(whole[1], want[1]) < BF16_BAR
+    for cuts in ([130, 2, 64, 9, 100, 8, 1, 1, 50, 17, 1], [12], [399, 1]):
+        assert err(portions(m, seqs[0], cuts), want[0]) < BF16_BAR, cuts
+    m.close()
+
+
+def test_planted_keys_at_chunk_edges_on_the_tensor_cores():
+    """As the planted keys above, for heads the tensor-core kernel takes: the query ends a prompt, or a portion of 20 tokens."""
+    size = 67
+    l = left(heads=4, kv_heads=2, dim=64, vdim=64, size=size, dims=16, scale=0.5)
+    cfg = config([layer(l=l, ls=2.0, rs=0.1, mlp=None)], vocab=40, width=256)
+    KEY, QUERY = 38, 39
+    m, o = build(cfg, dtype="bfloat16", tensors=planted(cfg, random_model(cfg, 19), KEY, QUERY), max_seq_len=300)
+    for n in (4 * size - 9, 3 * size, 3 * size + 2):
+        start = (n - 1) // size * size
+        outs = {}
+        for at in sorted({start, start - 1, n - 2, start - size + 1}):
+            ids = toks(n, 38, seed=20)
+            ids[at], ids[n - 1] = KEY, QUERY
+            want = fresh(o).run(ids)
+            outs[at] = want[-1]
+            assert err(m.forward_rows(ids[None], 0, [n - 1]), want[-1:]) < BF16_BAR, ("prompt", n, at)
+            assert err(portions(m, ids, [n - 20, 20])[-1:], want[-1:]) < BF16_BAR, ("portion", n, at)
+        assert err(outs[start], outs[start - 1]) > 0.3
+    m.close()
