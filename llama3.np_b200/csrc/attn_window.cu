@@ -15,6 +15,12 @@
 //                        arrive as 16-byte broadcasts.  Softmax rows run the online form,
 //                        started at (max = sink, sum = 1) so that the sink needs no key; sigmoid rows just accumulate.
 //                        Calls of few tokens split the key tiles over CTAs (win_attn_combine_kernel merges).
+//  * win_decode_kernel   one token per sequence, groups of 1, 2, 4 or 8 query heads: a CTA per (key split, key head, sequence).
+//                        Four threads per key score it for all heads of the group, a warp per head turns the scores into
+//                        weights, and the values - requested together with the keys - are summed by (16-byte column piece,
+//                        key part) threads.  Other sizes run win_attn_kernel.
+#include <stdlib.h>
+
 #include <algorithm>
 
 #include "common.cuh"
@@ -99,7 +105,31 @@ __global__ void __launch_bounds__(256) win_prep_kernel(WinPrepArgs a) {
     KVT* ck = (KVT*)a.cache_k + (((size_t)b * a.G + g) * a.M + pos) * a.DK;
     float* qf = a.q_out ? a.q_out + ((size_t)r * a.H + v) * a.DK : nullptr;
     bf16* qp = a.q16 ? a.q16 + ((size_t)r * a.H + v) * a.q16_ld : nullptr;
-    if (n % 4 == 0) {
+    if (n % 4 == 0 && a.rot_layout == 1 && half % 4 == 0) {  // a group of four turns with the group half a rotation away
+      for (int i = lane * 4; i < n; i += 128) {
+        auto in4 = [&](int c) {
+          float4 x = *reinterpret_cast<const float4*>(buf + c);
+          x.x *= rinv; x.y *= rinv; x.z *= rinv; x.w *= rinv;
+          if (w) { const float4 k = *reinterpret_cast<const float4*>(w + c); x.x *= k.x; x.y *= k.y; x.z *= k.z; x.w *= k.w; }
+          return x;
+        };
+        float4 x = in4(i);
+        if (i < a.rot_dims) {
+          const bool second = i >= half;
+          const int p = second ? i - half : i;
+          const float4 y = in4(second ? i - half : i + half);
+          const float4 c = *reinterpret_cast<const float4*>(cs + p);
+          float4 n4 = *reinterpret_cast<const float4*>(sn + p);
+          if (!second) { n4.x = -n4.x; n4.y = -n4.y; n4.z = -n4.z; n4.w = -n4.w; }
+          x.x = x.x * c.x + y.x * n4.x; x.y = x.y * c.y + y.y * n4.y; x.z = x.z * c.z + y.z * n4.z; x.w = x.w * c.w + y.w * n4.w;
+        }
+        if (!is_q) put4(ck + i, x.x, x.y, x.z, x.w);
+        else {
+          if (qf) put4(qf + i, x.x, x.y, x.z, x.w);
+          if (qp) put4(qp + i, x.x, x.y, x.z, x.w);
+        }
+      }
+    } else if (n % 4 == 0) {
       for (int i = lane * 4; i < n; i += 128) {
         const float x0 = out(i), x1 = out(i + 1), x2 = out(i + 2), x3 = out(i + 3);
         if (!is_q) put4(ck + i, x0, x1, x2, x3);
@@ -330,6 +360,153 @@ __global__ void __launch_bounds__(256) win_attn_kernel(WinAttnArgs a) {
   }
 }
 
+constexpr int WD_KEYS = 64, WD_KV = 8, WD_VV = 8;  // keys per tile; 16-byte pieces of a key / keys of a value part per thread
+
+template <typename KVT, int REP>
+__global__ void __launch_bounds__(256) win_decode_kernel(WinAttnArgs a) {
+  constexpr int VEC = Vec16<KVT>::N;
+  extern __shared__ __align__(16) float sm[];
+  float* sQ = sm;                          // [REP][DK]
+  float* sS = sQ + (size_t)REP * a.DK;     // [REP][WD_KEYS] scores, then weights
+  float* sA = sS + REP * WD_KEYS;          // [REP] rescaling of the sums so far
+  float* sM = sA + REP;                    // [REP] maximum | [REP] sum, at the end
+  float* sR = sM + 2 * REP + (4 - 3 * REP % 4) % 4;  // [parts][REP][DV]
+  pdl_launch();
+  pdl_wait();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int g = blockIdx.y, b = blockIdx.z, split = blockIdx.x;
+  const int p = *a.pos_ptr;                // the token's position; L == 1
+  const int lo = a.window <= 0 ? 0 : a.chunked ? p - p % a.window : max(0, p - a.window + 1);
+  const int ka = min(a.keep_first, lo), nkeys = ka + p + 1 - lo;
+  const int per = ((nkeys + a.nsplit - 1) / a.nsplit + 7) & ~7;
+  const int k_lo = min(nkeys, split * per), k_hi = min(nkeys, k_lo + per);
+  const KVT* ck = (const KVT*)a.cache_k + ((size_t)b * a.G + g) * a.M * a.DK;
+  const KVT* cv = (const KVT*)a.cache_v + ((size_t)b * a.G + g) * a.M * a.DV;
+  auto key_of = [&](int vi) { return vi < ka ? vi : lo + (vi - ka); };
+  const float* qrow = a.q + ((size_t)b * a.H + (size_t)g * REP) * a.DK;
+  for (int i = tid; i < REP * a.DK; i += 256) sQ[i] = qrow[i];
+  const int nkv = a.DK / VEC, nvv = a.DV / VEC, parts = 256 / nvv;  // pieces of a key, of a value; key parts of the output phase
+  const int kk = tid >> 2, kp = tid & 3;                            // score phase: key, quarter of its pieces
+  const int vc = tid % nvv, vp = tid / nvv;                         // output phase: column piece, key part
+  float m_run = -INFINITY, l_run = 0.f, hv = 0.f;
+  if (warp < REP) {  // warp r keeps head r's maximum and sum
+    hv = a.head_vec ? a.head_vec[g * REP + warp] : 0.f;
+    if (a.kind == L3_ATTN_SINK && a.head_vec && split == 0) { m_run = hv; l_run = 1.f; }
+  }
+  float acc[REP][VEC];
+#pragma unroll
+  for (int r = 0; r < REP; ++r)
+#pragma unroll
+    for (int x = 0; x < VEC; ++x) acc[r][x] = 0.f;
+
+  for (int t0 = k_lo; t0 < k_hi; t0 += WD_KEYS) {
+    uint4 kreg[WD_KV], vreg[WD_VV];
+    const bool k_ok = t0 + kk < k_hi;
+    const KVT* krow = ck + (size_t)key_of(k_ok ? t0 + kk : t0) * a.DK;
+#pragma unroll
+    for (int i = 0; i < WD_KV; ++i)
+      if (kp + 4 * i < nkv) kreg[i] = ldg_stream16(krow + (size_t)(kp + 4 * i) * VEC);
+#pragma unroll
+    for (int i = 0; i < WD_VV; ++i) {
+      const int vi = t0 + vp + i * parts;
+      if (vp + i * parts < WD_KEYS && vi < k_hi) vreg[i] = ldg_stream16(cv + (size_t)key_of(vi) * a.DV + (size_t)vc * VEC);
+    }
+    __syncthreads();  // sQ stands; the previous tile's weights have been used
+    float sc[REP];
+#pragma unroll
+    for (int r = 0; r < REP; ++r) sc[r] = 0.f;
+#pragma unroll
+    for (int i = 0; i < WD_KV; ++i)
+      if (kp + 4 * i < nkv) {
+        float f[VEC];
+        Vec16<KVT>::unpack(kreg[i], f);
+#pragma unroll
+        for (int r = 0; r < REP; ++r) {
+          const float* q = sQ + (size_t)r * a.DK + (kp + 4 * i) * VEC;
+#pragma unroll
+          for (int x = 0; x < VEC; x += 4) {
+            const float4 q4 = *reinterpret_cast<const float4*>(q + x);
+            sc[r] = fmaf(f[x], q4.x, sc[r]); sc[r] = fmaf(f[x + 1], q4.y, sc[r]);
+            sc[r] = fmaf(f[x + 2], q4.z, sc[r]); sc[r] = fmaf(f[x + 3], q4.w, sc[r]);
+          }
+        }
+      }
+#pragma unroll
+    for (int r = 0; r < REP; ++r) {
+      float s = sc[r];
+      s += __shfl_xor_sync(L3_FULL, s, 1);
+      s += __shfl_xor_sync(L3_FULL, s, 2);
+      if (kp == 0) sS[r * WD_KEYS + kk] = k_ok ? s * a.scale : -INFINITY;
+    }
+    __syncthreads();
+    if (warp < REP) {
+      float* s = sS + warp * WD_KEYS;
+      const float s0 = s[lane], s1 = s[lane + 32];
+      float w0, w1, alpha = 1.f;
+      if (a.kind == L3_ATTN_SIGMOID) {
+        w0 = s0 == -INFINITY ? 0.f : sigmoid_f(s0 + hv);
+        w1 = s1 == -INFINITY ? 0.f : sigmoid_f(s1 + hv);
+      } else {
+        const float mnew = fmaxf(m_run, warp_max(fmaxf(s0, s1)));  // a tile holds a key: finite
+        alpha = expf(m_run - mnew);
+        w0 = expf(s0 - mnew);
+        w1 = expf(s1 - mnew);
+        l_run = l_run * alpha + warp_sum(w0 + w1);
+        m_run = mnew;
+      }
+      s[lane] = w0;
+      s[lane + 32] = w1;
+      if (lane == 0) sA[warp] = alpha;
+    }
+    __syncthreads();
+    if (t0 > k_lo) {
+#pragma unroll
+      for (int r = 0; r < REP; ++r)
+#pragma unroll
+        for (int x = 0; x < VEC; ++x) acc[r][x] *= sA[r];
+    }
+#pragma unroll
+    for (int i = 0; i < WD_VV; ++i) {
+      const int vk = vp + i * parts;
+      if (vk < WD_KEYS && t0 + vk < k_hi) {
+        float f[VEC];
+        Vec16<KVT>::unpack(vreg[i], f);
+#pragma unroll
+        for (int r = 0; r < REP; ++r) {
+          const float w = sS[r * WD_KEYS + vk];
+#pragma unroll
+          for (int x = 0; x < VEC; ++x) acc[r][x] = fmaf(w, f[x], acc[r][x]);
+        }
+      }
+    }
+  }
+  if (warp < REP && lane == 0) { sM[warp] = m_run; sM[REP + warp] = l_run; }
+#pragma unroll
+  for (int r = 0; r < REP; ++r)
+#pragma unroll
+    for (int x = 0; x < VEC; x += 4)
+      *reinterpret_cast<float4*>(sR + ((size_t)vp * REP + r) * a.DV + vc * VEC + x) = make_float4(acc[r][x], acc[r][x + 1], acc[r][x + 2], acc[r][x + 3]);
+  __syncthreads();
+  for (int i = tid; i < REP * a.DV; i += 256) {
+    const int r = i / a.DV, d = i - r * a.DV, h = g * REP + r;
+    float t = 0.f;
+#pragma unroll 8
+    for (int q = 0; q < parts; ++q) t += sR[((size_t)q * REP + r) * a.DV + d];
+    const size_t rh = (size_t)b * a.H + h;
+    if (a.nsplit > 1) {
+      const size_t pi = rh * a.nsplit + split;
+      a.part_o[pi * a.DV + d] = t;
+      if (d == 0) { a.part_ml[pi * 2] = sM[r]; a.part_ml[pi * 2 + 1] = sM[REP + r]; }
+      continue;
+    }
+    float mul = a.out_scale * (a.kind == L3_ATTN_SIGMOID ? 1.f : (sM[REP + r] > 0.f ? 1.0f / sM[REP + r] : 0.f));
+    if (a.gate) mul *= sigmoid_f(a.gate[(size_t)b * a.ld_gate + h]);
+    const size_t oi = (size_t)b * a.ld_out + (size_t)h * a.DV + d;
+    if (a.out) a.out[oi] = t * mul;
+    if (a.out16) a.out16[oi] = __float2bfloat16_rn(t * mul);
+  }
+}
+
 // a CTA per (row, head): the splits' weights once, then a thread per value column
 __global__ void __launch_bounds__(128) win_attn_combine_kernel(WinAttnArgs a) {
   __shared__ float s_f[WA_SPLIT_MAX];
@@ -382,8 +559,37 @@ cudaError_t launch_win_nj(const WinAttnArgs& a, dim3 grid, cudaStream_t s) {
   return launch_k(win_attn_kernel<KVT, NJ>, grid, dim3(256), smem, s, a);
 }
 
+// decode sizes: whole 16-byte pieces, a tile's keys and values in registers
+template <typename KVT>
+bool win_decode_supported(const WinAttnArgs& a) {
+  constexpr int VEC = Vec16<KVT>::N;
+  const int rep = a.H / a.G, nvv = a.DV / VEC;
+  return a.L == 1 && (rep == 1 || rep == 2 || rep == 4 || rep == 8) && a.DK % VEC == 0 && a.DV % VEC == 0 && a.DK <= 4 * WD_KV * VEC &&
+         256 % nvv == 0 && WD_KEYS * nvv <= 256 * WD_VV;
+}
+
+template <typename KVT, int REP>
+cudaError_t launch_win_decode(const WinAttnArgs& a, cudaStream_t s) {
+  const int parts = 256 / (a.DV / Vec16<KVT>::N);
+  const size_t smem = ((size_t)REP * a.DK + REP * WD_KEYS + 3 * REP + 4 + (size_t)parts * REP * a.DV) * sizeof(float);
+  if (smem > 40 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(win_decode_kernel<KVT, REP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return e;
+  }
+  return launch_k(win_decode_kernel<KVT, REP>, dim3(a.nsplit, a.G, a.B), dim3(256), smem, s, a);
+}
+
 template <typename KVT>
 cudaError_t launch_win_t(const WinAttnArgs& a, dim3 grid, cudaStream_t s) {
+  static const bool decode_on = !(getenv("L3_WINDOW_DECODE") && atoi(getenv("L3_WINDOW_DECODE")) == 0);
+  if (decode_on && win_decode_supported<KVT>(a)) {
+    switch (a.H / a.G) {
+      case 1: return launch_win_decode<KVT, 1>(a, s);
+      case 2: return launch_win_decode<KVT, 2>(a, s);
+      case 4: return launch_win_decode<KVT, 4>(a, s);
+      default: return launch_win_decode<KVT, 8>(a, s);
+    }
+  }
   switch (win_nj(a.DV)) {
     case 1: return launch_win_nj<KVT, 1>(a, grid, s);
     case 2: return launch_win_nj<KVT, 2>(a, grid, s);

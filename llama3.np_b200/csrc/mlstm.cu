@@ -9,7 +9,7 @@
 // e^(-m) of every token, the recurrence carries n as one more column, and the output stage (mix_out_kernel) divides.
 //
 //  * mlstm_gates_kernel   a CTA per (head, sequence).  m_t as a function of m_0 is x -> max(a + x, b); such maps compose
-//                         ((a1 + a2, max(b1 + a2, b2))), so a tile of 256 tokens is one block-wide scan, tiles in a row.
+//                         ((a1 + a2, max(b1 + a2, b2))), so a tile of 256 or 1024 tokens is one block-wide scan, tiles in a row.
 //                         b stays of the order of the gates however long the tile, and a alone never survives against it.
 //  * mlstm_step_kernel    one token per sequence: gates, state update, normaliser, norm per head, output gate and scale in
 //                         one launch.  A cluster of CTAs shares a head by value columns; the square sum of the head's
@@ -30,11 +30,11 @@ __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
 
-constexpr int GT = 256;  // tokens per tile of the gate scan
-
+// GT: tokens per tile of the gate scan, a thread each
+template <int GT>
 __global__ void __launch_bounds__(GT) mlstm_gates_kernel(MlstmGateArgs a) {
   __shared__ float s_m[GT + 1];
-  __shared__ float w_a[8], w_b[8];
+  __shared__ float w_a[GT / 32], w_b[GT / 32];
   pdl_launch();
   pdl_wait();
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -208,7 +208,8 @@ cudaError_t launch_step(const MlstmStepArgs& a, int B, cudaStream_t s) {
 }  // namespace
 
 cudaError_t launch_mlstm_gates(const MlstmGateArgs& a, int B, cudaStream_t s) {
-  return launch_k(mlstm_gates_kernel, dim3(a.H, B), dim3(GT), 0, s, a);
+  if (a.L > 256) return launch_k(mlstm_gates_kernel<1024>, dim3(a.H, B), dim3(1024), 0, s, a);
+  return launch_k(mlstm_gates_kernel<256>, dim3(a.H, B), dim3(256), 0, s, a);
 }
 
 cudaError_t launch_mlstm_step(const MlstmStepArgs& a, int B, cudaStream_t s) {
