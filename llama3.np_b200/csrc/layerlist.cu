@@ -1505,7 +1505,7 @@ static int ll_mix_unit(L3Model* m, LLLayer& Ly, LLState& St, const float* pin, i
     ga.decay = ll->rg; ga.log_decay = ll->rg + nh; ga.k_scale = ll->rg + 2 * nh; ga.floor = ll->rg + 3 * nh; ga.L = L; ga.H = H;
     LAUNCH(m, launch_mlstm_gates(ga, B, m->stream));
     ra.mode = 2; ra.q = pin + Ly.off_q; ra.k = pin + Ly.off_k; ra.v = pin + Ly.off_v; ra.ld_q = ra.ld_k = ra.ld_v = ld; ra.rep = 1;
-    ra.g = ga.decay; ra.g_head = 1; ra.log_g = ga.log_decay; ra.k_scale = ga.k_scale; ra.q_mul = q_mul; ra.n_state = St.n; ra.nq = ll->rg + 4 * nh;
+    ra.g = ga.decay; ra.g_head = 1; ra.log_g = ga.log_decay; ra.k_scale = ga.k_scale; ra.q_mul = q_mul; ra.n_state = St.n; ra.nq = ll->rg + 4 * nh; ra.bf16_ops = m->tc_ok;
     ra.ws = ll->chunk_ws; ra.ws_floats = ll->chunk_ws_floats;
     LAUNCH(m, launch_recur(ra, m->stream));
     mo.nq = ra.nq; mo.floor = ga.floor; mo.gate = pin + Ly.off_g; mo.ld_gate = ld; mo.gate_act = 0; mo.pre_gate = 0;

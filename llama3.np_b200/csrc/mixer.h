@@ -75,6 +75,7 @@ struct RecurArgs {
   float q_mul;            // multiplies the queries (0: 1)
   float* n_state;         // [maxB, H, DK] a running sum of the keys with the state's own decay (the normaliser of an mLSTM) ...
   float* nq;              // ... and its product with the query, [B * L, H]
+  int bf16_ops;           // with n_state, chunk-parallel form: q, k and v may be rounded to bf16 (they are bf16 projections' outputs)
   float* ws;              // mode 0, may be null: room for one state matrix per (sequence, head, chunk of 64 tokens);
   size_t ws_floats;       // with it, prompts of the common shapes run in the chunk-parallel form (recur_chunk.cu)
 };

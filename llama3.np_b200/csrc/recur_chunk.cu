@@ -21,6 +21,10 @@
 // the column sums of its scaled keys, and n . q is q . P_n plus the row sums of A.  Keys carry a factor per token
 // (k_scale), and the decays' running sums are kept in double precision: a log decay can be as large as -30, and the
 // difference of two sums of 64 of them is what enters the exponential.
+// In bf16 mode (RecurArgs::bf16_ops, mLSTM) steps 1 and 3 run on warp-level tensor products with fp32 accumulation: queries,
+// keys and values, which are outputs of bf16 projections, are operands as they are (bf16), while everything the recurrence
+// itself makes - decayed keys, decayed scores, the states - enters as a pair hi + lo of bf16 values (16 significant bits).
+// A chunk's products are 64 x 64 tiles with 64 .. 256 summed terms, and their operands are built in the kernel.
 // The sums run in another order than the token-by-token kernel, so the two agree to fp32 rounding, not bit for bit.
 #include <stdint.h>
 
@@ -308,6 +312,255 @@ __global__ void __launch_bounds__(256) lin_chunk_out_kernel(RecurArgs a, int NC)
   }
 }
 
+// ---------------------------------------------------------------------------- bf16 mode: the same two kernels on mma.sync
+constexpr int LDE = 64 + 8;  // row length of a 64-wide bf16 tile: rows 144 bytes apart fall into distinct banks
+
+__device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint2 pack4(const float4& v) {
+  union { __nv_bfloat162 h[2]; uint2 u; } o;
+  o.h[0] = __floats2bfloat162_rn(v.x, v.y);
+  o.h[1] = __floats2bfloat162_rn(v.z, v.w);
+  return o.u;
+}
+// v = hi + lo up to 2^-17 of v
+__device__ __forceinline__ void split4(const float4& v, uint2& hi, uint2& lo) {
+  hi = pack4(v);
+  lo = pack4(make_float4(v.x - __uint_as_float(hi.x << 16), v.y - __uint_as_float(hi.x & 0xffff0000u), v.z - __uint_as_float(hi.y << 16),
+                         v.w - __uint_as_float(hi.y & 0xffff0000u)));
+}
+
+// rows x cols floats (rows >= n: zeros) -> bf16 tile, each row times mul
+__device__ __forceinline__ void load_bf16(bf16* dst, int ld_dst, const float* src, size_t ld_src, int rows, int n, int cols, float mul) {
+  const int c4 = cols / 4;
+#pragma unroll 4
+  for (int idx = threadIdx.x; idx < rows * c4; idx += blockDim.x) {
+    const int j = idx / c4, c = (idx - j * c4) * 4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (j < n) v = *reinterpret_cast<const float4*>(src + (size_t)j * ld_src + c);
+    v.x *= mul; v.y *= mul; v.z *= mul; v.w *= mul;
+    *reinterpret_cast<uint2*>(dst + (size_t)j * ld_dst + c) = pack4(v);
+  }
+}
+// the same as a (hi, lo) pair of tiles, row j times row_mul[j] (null: 1)
+__device__ __forceinline__ void load_split(bf16* hi, bf16* lo, int ld_dst, const float* src, size_t ld_src, int rows, int n, int cols, const float* row_mul) {
+  const int c4 = cols / 4;
+#pragma unroll 4
+  for (int idx = threadIdx.x; idx < rows * c4; idx += blockDim.x) {
+    const int j = idx / c4, c = (idx - j * c4) * 4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (j < n) v = *reinterpret_cast<const float4*>(src + (size_t)j * ld_src + c);
+    const float m = row_mul ? row_mul[j] : 1.f;
+    v.x *= m; v.y *= m; v.z *= m; v.w *= m;
+    uint2 h, l;
+    split4(v, h, l);
+    *reinterpret_cast<uint2*>(hi + (size_t)j * ld_dst + c) = h;
+    *reinterpret_cast<uint2*>(lo + (size_t)j * ld_dst + c) = l;
+  }
+}
+
+// grid (NC * NE, H, B): the chunk's D, value columns [e_lo, e_hi) of it.  8 warps on a 64 x 64 tile: 16 rows x 32 columns each
+__global__ void __launch_bounds__(256) lin_chunk_state_mma_kernel(RecurArgs a, int NC, int NE) {
+  extern __shared__ __align__(16) uint8_t smb[];
+  __shared__ double pd[CH];
+  __shared__ float sc[CH];
+  const int LDK = a.DK + 8;
+  bf16* Kh = reinterpret_cast<bf16*>(smb);           // [CH][LDK] decayed keys, hi and lo
+  bf16* Kl = Kh + (size_t)CH * LDK;
+  bf16* Vs = Kl + (size_t)CH * LDK;                  // [CH][LDE]
+  pdl_launch();
+  pdl_wait();
+  const int c = blockIdx.x / NE, ne = blockIdx.x - c * NE, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
+  const int lane = tid & 31, warp = tid >> 5, wm = warp & 3, wn = warp >> 2;
+  const int n = min(CH, a.L - c * CH);
+  const size_t row0 = (size_t)b * a.L + (size_t)c * CH;
+  fill_cumlog(pd, a.log_g + row0 * a.H + h, a.H, n);
+  __syncthreads();
+  for (int j = tid; j < CH; j += 256) sc[j] = j < n ? expf((float)(pd[n - 1] - pd[j])) * a.k_scale[(row0 + j) * a.H + h] : 0.f;
+  if (ne == 0 && tid == 0) chunk_decays(a, NC)[((size_t)b * a.H + h) * NC + c] = expf((float)pd[n - 1]);
+  __syncthreads();
+  load_split(Kh, Kl, LDK, a.k + row0 * a.ld_k + (size_t)(h / a.rep) * a.DK, a.ld_k, CH, n, a.DK, sc);
+  const int per = a.DV / 64 / NE, e_lo = ne * per * 64, e_hi = e_lo + per * 64;
+  float* D = a.ws + (((size_t)b * a.H + h) * NC + c) * a.DK * a.DV;
+  for (int e0 = e_lo; e0 < e_hi; e0 += 64) {
+    if (e0 > e_lo) __syncthreads();  // the previous tile's values are no longer read
+    load_bf16(Vs, LDE, a.v + row0 * a.ld_v + (size_t)h * a.DV + e0, a.ld_v, CH, n, 64, 1.f);
+    __syncthreads();
+    if (ne == 0 && e0 == 0)
+      for (int d = tid; d < a.DK; d += 256) {
+        float t = 0.f;
+#pragma unroll 8
+        for (int j = 0; j < CH; ++j) t += __bfloat162float(Kh[(size_t)j * LDK + d]) + __bfloat162float(Kl[(size_t)j * LDK + d]);
+        chunk_norms(a, NC)[(((size_t)b * a.H + h) * NC + c) * a.DK + d] = t;
+      }
+    for (int d0 = 0; d0 < a.DK; d0 += 64) {
+      float acc[4][4];
+      zero44(acc);
+#pragma unroll
+      for (int k0 = 0; k0 < CH; k0 += 16) {
+        uint32_t ah[4], al[4], v0[4], v1[4];
+        // A = K^T: tokens are rows of the tile, so both operands are read transposed
+        const size_t ka = (size_t)(k0 + (lane & 7) + ((lane >> 4) << 3)) * LDK + d0 + wm * 16 + ((lane >> 3) & 1) * 8;
+        ldsm4t(ah, smem_addr(Kh + ka));
+        ldsm4t(al, smem_addr(Kl + ka));
+        const bf16* vp = Vs + (size_t)(k0 + (lane & 15)) * LDE + wn * 32 + (lane >> 4) * 8;
+        ldsm4t(v0, smem_addr(vp));
+        ldsm4t(v1, smem_addr(vp + 16));
+        mma16816(acc[0], ah, v0[0], v0[1]); mma16816(acc[1], ah, v0[2], v0[3]);
+        mma16816(acc[2], ah, v1[0], v1[1]); mma16816(acc[3], ah, v1[2], v1[3]);
+        mma16816(acc[0], al, v0[0], v0[1]); mma16816(acc[1], al, v0[2], v0[3]);
+        mma16816(acc[2], al, v1[0], v1[1]); mma16816(acc[3], al, v1[2], v1[3]);
+      }
+      float* dp = D + (size_t)(d0 + wm * 16 + (lane >> 2)) * a.DV + e0 + wn * 32 + (lane & 3) * 2;
+#pragma unroll
+      for (int t = 0; t < 4; ++t) {
+        *reinterpret_cast<float2*>(dp + t * 8) = make_float2(acc[t][0], acc[t][1]);
+        *reinterpret_cast<float2*>(dp + (size_t)8 * a.DV + t * 8) = make_float2(acc[t][2], acc[t][3]);
+      }
+    }
+  }
+}
+
+// grid (NC * NE, H, B): the chunk's outputs, value columns as above
+__global__ void __launch_bounds__(256) lin_chunk_out_mma_kernel(RecurArgs a, int NC, int NE) {
+  extern __shared__ __align__(16) uint8_t smb[];
+  __shared__ double pd[CH];
+  __shared__ float ks[CH], s_nq[2][CH];
+  const int LDK = a.DK + 8;
+  bf16* Qs = reinterpret_cast<bf16*>(smb);           // [CH][LDK]
+  bf16* Ks = Qs + (size_t)CH * LDK;                  // [CH][LDK]
+  bf16* Ah = Ks + (size_t)CH * LDK;                  // [CH][LDE] decayed scores, hi and lo
+  bf16* Al = Ah + (size_t)CH * LDE;
+  bf16* Vs = Al + (size_t)CH * LDE;                  // [CH][LDE]
+  bf16* Ph = Vs + (size_t)CH * LDE;                  // [DK][LDE] the state ahead of the chunk, hi and lo
+  bf16* Pl = Ph + (size_t)a.DK * LDE;
+  pdl_launch();
+  pdl_wait();
+  const int c = blockIdx.x / NE, ne = blockIdx.x - c * NE, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
+  const int lane = tid & 31, warp = tid >> 5, wm = warp & 3, wn = warp >> 2;
+  const int n = min(CH, a.L - c * CH);
+  const size_t row0 = (size_t)b * a.L + (size_t)c * CH;
+  fill_cumlog(pd, a.log_g + row0 * a.H + h, a.H, n);
+  if (tid >= 32 && tid < 32 + CH) ks[tid - 32] = tid - 32 < n ? a.k_scale[(row0 + tid - 32) * a.H + h] : 0.f;
+  load_bf16(Qs, LDK, a.q + row0 * a.ld_q + (size_t)(h / a.rep) * a.DK, a.ld_q, CH, n, a.DK, a.q_mul);
+  load_bf16(Ks, LDK, a.k + row0 * a.ld_k + (size_t)(h / a.rep) * a.DK, a.ld_k, CH, n, a.DK, 1.f);
+  __syncthreads();
+  const int r0 = wm * 16 + (lane >> 2);              // this lane's accumulator rows: r0 and r0 + 8
+  const size_t qa = (size_t)(wm * 16 + (lane & 15)) * LDK + (lane >> 4) * 8;
+  {
+    float acc[4][4];
+    zero44(acc);
+    const bf16* kp = Ks + (size_t)(wn * 32 + (lane & 7) + ((lane >> 4) << 3)) * LDK + ((lane >> 3) & 1) * 8;
+#pragma unroll 4
+    for (int k0 = 0; k0 < a.DK; k0 += 16) {
+      uint32_t q[4], k_0[4], k_1[4];
+      ldsm4(q, smem_addr(Qs + qa + k0));
+      ldsm4(k_0, smem_addr(kp + k0));
+      ldsm4(k_1, smem_addr(kp + (size_t)16 * LDK + k0));
+      mma16816(acc[0], q, k_0[0], k_0[1]); mma16816(acc[1], q, k_0[2], k_0[3]);
+      mma16816(acc[2], q, k_1[0], k_1[1]); mma16816(acc[3], q, k_1[2], k_1[3]);
+    }
+    float sum[2] = {0.f, 0.f};
+#pragma unroll
+    for (int t = 0; t < 4; ++t)
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {                  // rows r0, r0 + 8
+        const int i = r0 + u * 8, j = wn * 32 + t * 8 + (lane & 3) * 2;
+        const float x = j <= i ? acc[t][2 * u] * (expf((float)(pd[i] - pd[j])) * ks[j]) : 0.f;
+        const float y = j + 1 <= i ? acc[t][2 * u + 1] * (expf((float)(pd[i] - pd[j + 1])) * ks[j + 1]) : 0.f;
+        sum[u] += x + y;
+        const __nv_bfloat162 hi = __floats2bfloat162_rn(x, y);
+        *reinterpret_cast<__nv_bfloat162*>(Ah + (size_t)i * LDE + j) = hi;
+        *reinterpret_cast<__nv_bfloat162*>(Al + (size_t)i * LDE + j) = __floats2bfloat162_rn(x - __low2float(hi), y - __high2float(hi));
+      }
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      sum[u] += __shfl_xor_sync(L3_FULL, sum[u], 1);
+      sum[u] += __shfl_xor_sync(L3_FULL, sum[u], 2);
+      if ((lane & 3) == 0) s_nq[wn][r0 + u * 8] = sum[u];
+    }
+  }
+  __syncthreads();
+  if (ne == 0) {  // n . q of every token: four threads per row
+    const float* Pn = chunk_norms(a, NC) + (((size_t)b * a.H + h) * NC + c) * a.DK;
+    const int i = tid >> 2, part = tid & 3;
+    float t = 0.f;
+    for (int d = part * 2; d < a.DK; d += 8) {
+      const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Qs + (size_t)i * LDK + d));
+      t = fmaf(q.x, Pn[d], t);
+      t = fmaf(q.y, Pn[d + 1], t);
+    }
+    t += __shfl_xor_sync(L3_FULL, t, 1);
+    t += __shfl_xor_sync(L3_FULL, t, 2);
+    if (part == 0 && i < n) a.nq[(row0 + i) * a.H + h] = fmaf(t, expf((float)pd[i]), s_nq[0][i] + s_nq[1][i]);
+  }
+  const float* P = a.ws + (((size_t)b * a.H + h) * NC + c) * a.DK * a.DV;
+  const int O = a.H * a.DV;
+  const int per = a.DV / 64 / NE, e_lo = ne * per * 64, e_hi = e_lo + per * 64;
+  const float f0 = expf((float)pd[r0]), f1 = expf((float)pd[r0 + 8]);
+  const size_t va = (size_t)(lane & 15) * LDE + wn * 32 + (lane >> 4) * 8, aa = (size_t)(wm * 16 + (lane & 15)) * LDE + (lane >> 4) * 8;
+  for (int e0 = e_lo; e0 < e_hi; e0 += 64) {
+    if (e0 > e_lo) __syncthreads();  // the previous tile's Vs / P are no longer read
+    load_bf16(Vs, LDE, a.v + row0 * a.ld_v + (size_t)h * a.DV + e0, a.ld_v, CH, n, 64, 1.f);
+    load_split(Ph, Pl, LDE, P + e0, a.DV, a.DK, a.DK, 64, nullptr);
+    __syncthreads();
+    float acc[4][4];
+    zero44(acc);
+#pragma unroll 4
+    for (int k0 = 0; k0 < a.DK; k0 += 16) {
+      uint32_t q[4], p0[4], p1[4];
+      ldsm4(q, smem_addr(Qs + qa + k0));
+      const size_t o = (size_t)k0 * LDE + va;
+      ldsm4t(p0, smem_addr(Ph + o));
+      ldsm4t(p1, smem_addr(Ph + o + 16));
+      mma16816(acc[0], q, p0[0], p0[1]); mma16816(acc[1], q, p0[2], p0[3]);
+      mma16816(acc[2], q, p1[0], p1[1]); mma16816(acc[3], q, p1[2], p1[3]);
+      ldsm4t(p0, smem_addr(Pl + o));
+      ldsm4t(p1, smem_addr(Pl + o + 16));
+      mma16816(acc[0], q, p0[0], p0[1]); mma16816(acc[1], q, p0[2], p0[3]);
+      mma16816(acc[2], q, p1[0], p1[1]); mma16816(acc[3], q, p1[2], p1[3]);
+    }
+#pragma unroll
+    for (int t = 0; t < 4; ++t) { acc[t][0] *= f0; acc[t][1] *= f0; acc[t][2] *= f1; acc[t][3] *= f1; }
+#pragma unroll
+    for (int k0 = 0; k0 < CH; k0 += 16) {
+      uint32_t ah[4], al[4], v0[4], v1[4];
+      ldsm4(ah, smem_addr(Ah + aa + k0));
+      ldsm4(al, smem_addr(Al + aa + k0));
+      const size_t o = (size_t)k0 * LDE + va;
+      ldsm4t(v0, smem_addr(Vs + o));
+      ldsm4t(v1, smem_addr(Vs + o + 16));
+      mma16816(acc[0], ah, v0[0], v0[1]); mma16816(acc[1], ah, v0[2], v0[3]);
+      mma16816(acc[2], ah, v1[0], v1[1]); mma16816(acc[3], ah, v1[2], v1[3]);
+      mma16816(acc[0], al, v0[0], v0[1]); mma16816(acc[1], al, v0[2], v0[3]);
+      mma16816(acc[2], al, v1[0], v1[1]); mma16816(acc[3], al, v1[2], v1[3]);
+    }
+    float* op = a.out + (row0 + r0) * O + (size_t)h * a.DV + e0 + wn * 32 + (lane & 3) * 2;
+#pragma unroll
+    for (int t = 0; t < 4; ++t) {
+      if (r0 < n) *reinterpret_cast<float2*>(op + t * 8) = make_float2(acc[t][0], acc[t][1]);
+      if (r0 + 8 < n) *reinterpret_cast<float2*>(op + (size_t)8 * O + t * 8) = make_float2(acc[t][2], acc[t][3]);
+    }
+  }
+}
+
+// CTAs per chunk along the value columns: a divisor of the 64-column tiles, enough that `want` CTAs run
+int value_splits(int ctas, int tiles, int want) {
+  int ne = 1;
+  for (int d = 1; d <= tiles; ++d)
+    if (tiles % d == 0) { ne = d; if (ctas * d >= want) break; }
+  return ne;
+}
+
 bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
 
 }  // namespace
@@ -343,6 +596,17 @@ cudaError_t launch_recur_chunk(const RecurArgs& a, cudaStream_t s) {
     if ((e = launch_k(k_scan, dim3((n4 + 255) / 256, a.H, a.B), dim3(256), 0, s, a, NC)) != cudaSuccess) return e;
     return launch_k(k_out, grid, dim3(256), sm3, s, a, NC);
   };
+  if (a.n_state && a.bf16_ops) {
+    const size_t sb1 = ((size_t)2 * CH * (a.DK + 8) + CH * LDE) * 2, sb3 = ((size_t)2 * CH * (a.DK + 8) + 3 * CH * LDE + 2 * (size_t)a.DK * LDE) * 2;
+    const int ctas = NC * a.H * a.B, tiles = a.DV / 64;
+    const int ne1 = value_splits(ctas, tiles, 4 * 148), ne3 = value_splits(ctas, tiles, 2 * 148);
+    cudaError_t e;
+    if ((e = cudaFuncSetAttribute(lin_chunk_state_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sb1)) != cudaSuccess) return e;
+    if ((e = cudaFuncSetAttribute(lin_chunk_out_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sb3)) != cudaSuccess) return e;
+    if ((e = launch_k(lin_chunk_state_mma_kernel, dim3(NC * ne1, a.H, a.B), dim3(256), sb1, s, a, NC, ne1)) != cudaSuccess) return e;
+    if ((e = launch_k(lin_chunk_scan_kernel<true, true>, dim3((n4 + 255) / 256, a.H, a.B), dim3(256), 0, s, a, NC)) != cudaSuccess) return e;
+    return launch_k(lin_chunk_out_mma_kernel, dim3(NC * ne3, a.H, a.B), dim3(256), sb3, s, a, NC, ne3);
+  }
   if (a.n_state) return go(lin_chunk_state_kernel<true, true>, lin_chunk_scan_kernel<true, true>, lin_chunk_out_kernel<true, true>);
   if (a.mode == 2) return go(lin_chunk_state_kernel<true, false>, lin_chunk_scan_kernel<true, false>, lin_chunk_out_kernel<true, false>);
   return go(lin_chunk_state_kernel<false, false>, lin_chunk_scan_kernel<false, false>, lin_chunk_out_kernel<false, false>);
