@@ -339,41 +339,48 @@ __device__ __forceinline__ void split4(const float4& v, uint2& hi, uint2& lo) {
                          v.w - __uint_as_float(hi.y & 0xffff0000u)));
 }
 
-// rows x cols floats (rows >= n: zeros) -> bf16 tile, each row times mul
-__device__ __forceinline__ void load_bf16(bf16* dst, int ld_dst, const float* src, size_t ld_src, int rows, int n, int cols, float mul) {
-  const int c4 = cols / 4;
-#pragma unroll 4
-  for (int idx = threadIdx.x; idx < rows * c4; idx += blockDim.x) {
-    const int j = idx / c4, c = (idx - j * c4) * 4;
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (j < n) v = *reinterpret_cast<const float4*>(src + (size_t)j * ld_src + c);
-    v.x *= mul; v.y *= mul; v.z *= mul; v.w *= mul;
-    *reinterpret_cast<uint2*>(dst + (size_t)j * ld_dst + c) = pack4(v);
+// A [ROWS][COLS] block of floats on its way into bf16 tiles: fetch() issues every load of the thread's share at once, put() /
+// put_split() converts and stores it; between the two a thread can work on the previous block.  Rows >= n are zeros.
+template <int ROWS, int COLS>
+struct Block {
+  static constexpr int C4 = COLS / 4, N = ROWS * C4 / 256;
+  static_assert(ROWS * C4 % 256 == 0, "a whole number of vectors per thread");
+  float4 v[N];
+  __device__ __forceinline__ void fetch(const float* src, size_t ld, int n) {
+#pragma unroll
+    for (int u = 0; u < N; ++u) {
+      const int idx = threadIdx.x + u * 256, j = idx / C4, c = (idx % C4) * 4;
+      v[u] = j < n ? *reinterpret_cast<const float4*>(src + (size_t)j * ld + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
   }
-}
-// the same as a (hi, lo) pair of tiles, row j times row_mul[j] (null: 1)
-__device__ __forceinline__ void load_split(bf16* hi, bf16* lo, int ld_dst, const float* src, size_t ld_src, int rows, int n, int cols, const float* row_mul) {
-  const int c4 = cols / 4;
-#pragma unroll 4
-  for (int idx = threadIdx.x; idx < rows * c4; idx += blockDim.x) {
-    const int j = idx / c4, c = (idx - j * c4) * 4;
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (j < n) v = *reinterpret_cast<const float4*>(src + (size_t)j * ld_src + c);
-    const float m = row_mul ? row_mul[j] : 1.f;
-    v.x *= m; v.y *= m; v.z *= m; v.w *= m;
-    uint2 h, l;
-    split4(v, h, l);
-    *reinterpret_cast<uint2*>(hi + (size_t)j * ld_dst + c) = h;
-    *reinterpret_cast<uint2*>(lo + (size_t)j * ld_dst + c) = l;
+  __device__ __forceinline__ void put(bf16* dst, int ld_dst, float mul) const {
+#pragma unroll
+    for (int u = 0; u < N; ++u) {
+      const int idx = threadIdx.x + u * 256, j = idx / C4, c = (idx % C4) * 4;
+      *reinterpret_cast<uint2*>(dst + (size_t)j * ld_dst + c) = pack4(make_float4(v[u].x * mul, v[u].y * mul, v[u].z * mul, v[u].w * mul));
+    }
   }
-}
+  // a (hi, lo) pair of tiles, row j times row_mul[j] (null: 1)
+  __device__ __forceinline__ void put_split(bf16* hi, bf16* lo, int ld_dst, const float* row_mul) const {
+#pragma unroll
+    for (int u = 0; u < N; ++u) {
+      const int idx = threadIdx.x + u * 256, j = idx / C4, c = (idx % C4) * 4;
+      const float m = row_mul ? row_mul[j] : 1.f;
+      uint2 h, l;
+      split4(make_float4(v[u].x * m, v[u].y * m, v[u].z * m, v[u].w * m), h, l);
+      *reinterpret_cast<uint2*>(hi + (size_t)j * ld_dst + c) = h;
+      *reinterpret_cast<uint2*>(lo + (size_t)j * ld_dst + c) = l;
+    }
+  }
+};
 
 // grid (NC * NE, H, B): the chunk's D, value columns [e_lo, e_hi) of it.  8 warps on a 64 x 64 tile: 16 rows x 32 columns each
+template <int DK>
 __global__ void __launch_bounds__(256) lin_chunk_state_mma_kernel(RecurArgs a, int NC, int NE) {
   extern __shared__ __align__(16) uint8_t smb[];
   __shared__ double pd[CH];
   __shared__ float sc[CH];
-  const int LDK = a.DK + 8;
+  constexpr int LDK = DK + 8;
   bf16* Kh = reinterpret_cast<bf16*>(smb);           // [CH][LDK] decayed keys, hi and lo
   bf16* Kl = Kh + (size_t)CH * LDK;
   bf16* Vs = Kl + (size_t)CH * LDK;                  // [CH][LDE]
@@ -383,26 +390,33 @@ __global__ void __launch_bounds__(256) lin_chunk_state_mma_kernel(RecurArgs a, i
   const int lane = tid & 31, warp = tid >> 5, wm = warp & 3, wn = warp >> 2;
   const int n = min(CH, a.L - c * CH);
   const size_t row0 = (size_t)b * a.L + (size_t)c * CH;
+  const int per = a.DV / 64 / NE, e_lo = ne * per * 64, e_hi = e_lo + per * 64;
+  const float* vsrc = a.v + row0 * a.ld_v + (size_t)h * a.DV;
+  Block<CH, DK> kb;
+  Block<CH, 64> vb;
+  kb.fetch(a.k + row0 * a.ld_k + (size_t)(h / a.rep) * DK, a.ld_k, n);
+  vb.fetch(vsrc + e_lo, a.ld_v, n);
   fill_cumlog(pd, a.log_g + row0 * a.H + h, a.H, n);
   __syncthreads();
   for (int j = tid; j < CH; j += 256) sc[j] = j < n ? expf((float)(pd[n - 1] - pd[j])) * a.k_scale[(row0 + j) * a.H + h] : 0.f;
   if (ne == 0 && tid == 0) chunk_decays(a, NC)[((size_t)b * a.H + h) * NC + c] = expf((float)pd[n - 1]);
   __syncthreads();
-  load_split(Kh, Kl, LDK, a.k + row0 * a.ld_k + (size_t)(h / a.rep) * a.DK, a.ld_k, CH, n, a.DK, sc);
-  const int per = a.DV / 64 / NE, e_lo = ne * per * 64, e_hi = e_lo + per * 64;
+  kb.put_split(Kh, Kl, LDK, sc);
   float* D = a.ws + (((size_t)b * a.H + h) * NC + c) * a.DK * a.DV;
   for (int e0 = e_lo; e0 < e_hi; e0 += 64) {
     if (e0 > e_lo) __syncthreads();  // the previous tile's values are no longer read
-    load_bf16(Vs, LDE, a.v + row0 * a.ld_v + (size_t)h * a.DV + e0, a.ld_v, CH, n, 64, 1.f);
+    vb.put(Vs, LDE, 1.f);
     __syncthreads();
+    if (e0 + 64 < e_hi) vb.fetch(vsrc + e0 + 64, a.ld_v, n);  // in flight during the products
     if (ne == 0 && e0 == 0)
-      for (int d = tid; d < a.DK; d += 256) {
+      for (int d = tid; d < DK; d += 256) {
         float t = 0.f;
 #pragma unroll 8
         for (int j = 0; j < CH; ++j) t += __bfloat162float(Kh[(size_t)j * LDK + d]) + __bfloat162float(Kl[(size_t)j * LDK + d]);
-        chunk_norms(a, NC)[(((size_t)b * a.H + h) * NC + c) * a.DK + d] = t;
+        chunk_norms(a, NC)[(((size_t)b * a.H + h) * NC + c) * DK + d] = t;
       }
-    for (int d0 = 0; d0 < a.DK; d0 += 64) {
+#pragma unroll 1
+    for (int d0 = 0; d0 < DK; d0 += 64) {
       float acc[4][4];
       zero44(acc);
 #pragma unroll
@@ -431,18 +445,19 @@ __global__ void __launch_bounds__(256) lin_chunk_state_mma_kernel(RecurArgs a, i
 }
 
 // grid (NC * NE, H, B): the chunk's outputs, value columns as above
+template <int DK>
 __global__ void __launch_bounds__(256) lin_chunk_out_mma_kernel(RecurArgs a, int NC, int NE) {
   extern __shared__ __align__(16) uint8_t smb[];
   __shared__ double pd[CH];
   __shared__ float ks[CH], s_nq[2][CH];
-  const int LDK = a.DK + 8;
+  constexpr int LDK = DK + 8;
   bf16* Qs = reinterpret_cast<bf16*>(smb);           // [CH][LDK]
   bf16* Ks = Qs + (size_t)CH * LDK;                  // [CH][LDK]
   bf16* Ah = Ks + (size_t)CH * LDK;                  // [CH][LDE] decayed scores, hi and lo
   bf16* Al = Ah + (size_t)CH * LDE;
   bf16* Vs = Al + (size_t)CH * LDE;                  // [CH][LDE]
   bf16* Ph = Vs + (size_t)CH * LDE;                  // [DK][LDE] the state ahead of the chunk, hi and lo
-  bf16* Pl = Ph + (size_t)a.DK * LDE;
+  bf16* Pl = Ph + (size_t)DK * LDE;
   pdl_launch();
   pdl_wait();
   const int c = blockIdx.x / NE, ne = blockIdx.x - c * NE, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
@@ -451,8 +466,21 @@ __global__ void __launch_bounds__(256) lin_chunk_out_mma_kernel(RecurArgs a, int
   const size_t row0 = (size_t)b * a.L + (size_t)c * CH;
   fill_cumlog(pd, a.log_g + row0 * a.H + h, a.H, n);
   if (tid >= 32 && tid < 32 + CH) ks[tid - 32] = tid - 32 < n ? a.k_scale[(row0 + tid - 32) * a.H + h] : 0.f;
-  load_bf16(Qs, LDK, a.q + row0 * a.ld_q + (size_t)(h / a.rep) * a.DK, a.ld_q, CH, n, a.DK, a.q_mul);
-  load_bf16(Ks, LDK, a.k + row0 * a.ld_k + (size_t)(h / a.rep) * a.DK, a.ld_k, CH, n, a.DK, 1.f);
+  {
+    Block<CH, DK> qb, kb;
+    qb.fetch(a.q + row0 * a.ld_q + (size_t)(h / a.rep) * DK, a.ld_q, n);
+    kb.fetch(a.k + row0 * a.ld_k + (size_t)(h / a.rep) * DK, a.ld_k, n);
+    qb.put(Qs, LDK, a.q_mul);
+    kb.put(Ks, LDK, 1.f);
+  }
+  const float* P = a.ws + (((size_t)b * a.H + h) * NC + c) * DK * a.DV;
+  const float* vsrc = a.v + row0 * a.ld_v + (size_t)h * a.DV;
+  const int O = a.H * a.DV;
+  const int per = a.DV / 64 / NE, e_lo = ne * per * 64, e_hi = e_lo + per * 64;
+  Block<CH, 64> vb;
+  Block<DK, 64> pb;
+  vb.fetch(vsrc + e_lo, a.ld_v, n);  // the first tile's values and state columns: in flight during the scores
+  pb.fetch(P + e_lo, a.DV, DK);
   __syncthreads();
   const int r0 = wm * 16 + (lane >> 2);              // this lane's accumulator rows: r0 and r0 + 8
   const size_t qa = (size_t)(wm * 16 + (lane & 15)) * LDK + (lane >> 4) * 8;
@@ -460,8 +488,8 @@ __global__ void __launch_bounds__(256) lin_chunk_out_mma_kernel(RecurArgs a, int
     float acc[4][4];
     zero44(acc);
     const bf16* kp = Ks + (size_t)(wn * 32 + (lane & 7) + ((lane >> 4) << 3)) * LDK + ((lane >> 3) & 1) * 8;
-#pragma unroll 4
-    for (int k0 = 0; k0 < a.DK; k0 += 16) {
+#pragma unroll
+    for (int k0 = 0; k0 < DK; k0 += 16) {
       uint32_t q[4], k_0[4], k_1[4];
       ldsm4(q, smem_addr(Qs + qa + k0));
       ldsm4(k_0, smem_addr(kp + k0));
@@ -491,10 +519,11 @@ __global__ void __launch_bounds__(256) lin_chunk_out_mma_kernel(RecurArgs a, int
   }
   __syncthreads();
   if (ne == 0) {  // n . q of every token: four threads per row
-    const float* Pn = chunk_norms(a, NC) + (((size_t)b * a.H + h) * NC + c) * a.DK;
+    const float* Pn = chunk_norms(a, NC) + (((size_t)b * a.H + h) * NC + c) * DK;
     const int i = tid >> 2, part = tid & 3;
     float t = 0.f;
-    for (int d = part * 2; d < a.DK; d += 8) {
+#pragma unroll 4
+    for (int d = part * 2; d < DK; d += 8) {
       const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Qs + (size_t)i * LDK + d));
       t = fmaf(q.x, Pn[d], t);
       t = fmaf(q.y, Pn[d + 1], t);
@@ -503,20 +532,18 @@ __global__ void __launch_bounds__(256) lin_chunk_out_mma_kernel(RecurArgs a, int
     t += __shfl_xor_sync(L3_FULL, t, 2);
     if (part == 0 && i < n) a.nq[(row0 + i) * a.H + h] = fmaf(t, expf((float)pd[i]), s_nq[0][i] + s_nq[1][i]);
   }
-  const float* P = a.ws + (((size_t)b * a.H + h) * NC + c) * a.DK * a.DV;
-  const int O = a.H * a.DV;
-  const int per = a.DV / 64 / NE, e_lo = ne * per * 64, e_hi = e_lo + per * 64;
   const float f0 = expf((float)pd[r0]), f1 = expf((float)pd[r0 + 8]);
   const size_t va = (size_t)(lane & 15) * LDE + wn * 32 + (lane >> 4) * 8, aa = (size_t)(wm * 16 + (lane & 15)) * LDE + (lane >> 4) * 8;
   for (int e0 = e_lo; e0 < e_hi; e0 += 64) {
     if (e0 > e_lo) __syncthreads();  // the previous tile's Vs / P are no longer read
-    load_bf16(Vs, LDE, a.v + row0 * a.ld_v + (size_t)h * a.DV + e0, a.ld_v, CH, n, 64, 1.f);
-    load_split(Ph, Pl, LDE, P + e0, a.DV, a.DK, a.DK, 64, nullptr);
+    vb.put(Vs, LDE, 1.f);
+    pb.put_split(Ph, Pl, LDE, nullptr);
     __syncthreads();
+    if (e0 + 64 < e_hi) { vb.fetch(vsrc + e0 + 64, a.ld_v, n); pb.fetch(P + e0 + 64, a.DV, DK); }
     float acc[4][4];
     zero44(acc);
 #pragma unroll 4
-    for (int k0 = 0; k0 < a.DK; k0 += 16) {
+    for (int k0 = 0; k0 < DK; k0 += 16) {
       uint32_t q[4], p0[4], p1[4];
       ldsm4(q, smem_addr(Qs + qa + k0));
       const size_t o = (size_t)k0 * LDE + va;
@@ -599,13 +626,21 @@ cudaError_t launch_recur_chunk(const RecurArgs& a, cudaStream_t s) {
   if (a.n_state && a.bf16_ops) {
     const size_t sb1 = ((size_t)2 * CH * (a.DK + 8) + CH * LDE) * 2, sb3 = ((size_t)2 * CH * (a.DK + 8) + 3 * CH * LDE + 2 * (size_t)a.DK * LDE) * 2;
     const int ctas = NC * a.H * a.B, tiles = a.DV / 64;
-    const int ne1 = value_splits(ctas, tiles, 4 * 148), ne3 = value_splits(ctas, tiles, 2 * 148);
-    cudaError_t e;
-    if ((e = cudaFuncSetAttribute(lin_chunk_state_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sb1)) != cudaSuccess) return e;
-    if ((e = cudaFuncSetAttribute(lin_chunk_out_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sb3)) != cudaSuccess) return e;
-    if ((e = launch_k(lin_chunk_state_mma_kernel, dim3(NC * ne1, a.H, a.B), dim3(256), sb1, s, a, NC, ne1)) != cudaSuccess) return e;
-    if ((e = launch_k(lin_chunk_scan_kernel<true, true>, dim3((n4 + 255) / 256, a.H, a.B), dim3(256), 0, s, a, NC)) != cudaSuccess) return e;
-    return launch_k(lin_chunk_out_mma_kernel, dim3(NC * ne3, a.H, a.B), dim3(256), sb3, s, a, NC, ne3);
+    const int ne1 = value_splits(ctas, tiles, 100), ne3 = value_splits(ctas, tiles, 100);  // measured: only short prompts of few heads gain
+    auto go_mma = [&](auto k_state, auto k_out) {
+      cudaError_t e;
+      if ((e = cudaFuncSetAttribute(k_state, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sb1)) != cudaSuccess) return e;
+      if ((e = cudaFuncSetAttribute(k_out, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sb3)) != cudaSuccess) return e;
+      if ((e = launch_k(k_state, dim3(NC * ne1, a.H, a.B), dim3(256), sb1, s, a, NC, ne1)) != cudaSuccess) return e;
+      if ((e = launch_k(lin_chunk_scan_kernel<true, true>, dim3((n4 + 255) / 256, a.H, a.B), dim3(256), 0, s, a, NC)) != cudaSuccess) return e;
+      return launch_k(k_out, dim3(NC * ne3, a.H, a.B), dim3(256), sb3, s, a, NC, ne3);
+    };
+    switch (a.DK) {
+      case 64: return go_mma(lin_chunk_state_mma_kernel<64>, lin_chunk_out_mma_kernel<64>);
+      case 128: return go_mma(lin_chunk_state_mma_kernel<128>, lin_chunk_out_mma_kernel<128>);
+      case 192: return go_mma(lin_chunk_state_mma_kernel<192>, lin_chunk_out_mma_kernel<192>);
+      default: return go_mma(lin_chunk_state_mma_kernel<256>, lin_chunk_out_mma_kernel<256>);
+    }
   }
   if (a.n_state) return go(lin_chunk_state_kernel<true, true>, lin_chunk_scan_kernel<true, true>, lin_chunk_out_kernel<true, true>);
   if (a.mode == 2) return go(lin_chunk_state_kernel<true, false>, lin_chunk_scan_kernel<true, false>, lin_chunk_out_kernel<true, false>);
