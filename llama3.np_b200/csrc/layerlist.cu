@@ -1759,7 +1759,8 @@ static int ll_enqueue_prenorm(L3Model* m, int B, int L, float* d_resid) {
     if (Ly.ff_total) {  // gated experts, weights on their outputs, a shared expert
       const int E = s.experts, ff = s.ff, F = Ly.ff_total;
       if ((rc = ff_in(true)) != L3_OK) return rc;
-      const bool few = ntok <= 8;
+      // few rows read their own experts' weights, row by row - while that is less than reading all of them once
+      const bool few = ntok <= 8 && ntok * (s.top * ff + s.shared_ff) <= F;
       MoeRouteArgs ra{};
       ra.h = h2; ra.router = Ly.router; ra.D = W; ra.E = E; ra.top = s.top; ra.groups = 1; ra.keep = 1; ra.kind = 2; ra.scale = 1.0f; ra.shared_gate = s.shared_gate;
       ra.sel = ll->moe_sel; ra.w = ll->moe_w; ra.dense = few ? nullptr : ll->moe_dense; ra.idw = ll->moe_idw;
