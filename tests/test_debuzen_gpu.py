@@ -550,3 +550,25 @@ def test_larger_shapes_take_the_tensor_core_projections():
     assert m.launch_count() > 0
     assert close(portions(m, ids, [64, 20, 2, 1]), want, "bfloat16")
     m.close()
+
+
+@pytest.mark.parametrize("case", ["grouped", "wide_values", "off_the_grid"])
+def test_sink_windows_of_wide_heads_on_the_tensor_cores(case):
+    """Softmax windows with heads of 64 and more in bf16 mode: portions of more than 8 tokens run on the tensor cores, shorter ones
+    and single tokens on the exact kernels.  Windows end inside key blocks and portions start inside windows; the sinks take a good
+    part of the softmax."""
+    left = {"grouped": attn(heads=4, kv_heads=2, dim=64, vdim=64, size=70, dims=32, scale=0.15),
+            "wide_values": attn(heads=2, kv_heads=1, dim=128, vdim=192, size=190, dims=64, scale=0.1),
+            "off_the_grid": attn(heads=3, kv_heads=3, dim=72, vdim=88, size=33, dims=24, scale=0.12)}[case]
+    cfg = config([par2(left=left, mlp=None), par2(left=dict(left, mask={"size": 129}), mlp=None)], width=120, vocab=150)
+    t = random_tensors(cfg, 80)
+    for i in range(2):
+        t[f"l{i}.mix.left.sink"] = np.linspace(-1.0, 4.0, left["heads"]).astype(np.float32)
+    m, o = build(cfg, dtype="bfloat16", tensors=t, max_seq_len=320, max_batch_size=2)
+    seqs = np.stack([toks(300, 150, seed=s) for s in (81, 82)])
+    want = np.stack([fresh(o).run(s) for s in seqs])
+    whole = m.forward_rows(seqs, 0, list(range(600))).reshape(2, 300, -1)
+    assert err(whole[0], want[0]) < BF16_BAR and err(whole[1], want[1]) < BF16_BAR
+    for cuts in ([130, 2, 64, 9, 40, 8, 1, 1, 17, 1], [12], [299, 1]):
+        assert err(portions(m, seqs[0], cuts), want[0]) < BF16_BAR, cuts
+    m.close()

@@ -223,14 +223,14 @@ def planted(cfg, t, key_tok, query_tok):
     return t
 
 
-@pytest.mark.parametrize("kv_heads", [1, 4])
+@pytest.mark.parametrize("kv_heads, vdim", [(1, 40), (2, 64), (4, 32)])   # decoded by the tiled kernel / by the decode kernel
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-def test_planted_key_just_inside_and_just_outside_a_chunk(kv_heads, dtype):
+def test_planted_key_just_inside_and_just_outside_a_chunk(kv_heads, vdim, dtype):
     """One key decides the attention's output.  It sits at the chunk's first position, right ahead of it, at the chunk's
     middle, right ahead of the query, in the chunk before; the query is the last token of a prompt, of a portion of two
     tokens, or decoded alone, and sits inside a chunk, at a chunk's last and at a chunk's first position."""
     size = 37
-    l = left(heads=4, kv_heads=kv_heads, dim=24, vdim=40, size=size, dims=8, scale=0.9)
+    l = left(heads=4, kv_heads=kv_heads, dim=24, vdim=vdim, size=size, dims=8, scale=0.9)
     cfg = config([layer(l=l, ls=2.0, rs=0.1, mlp=None)], vocab=60, width=96)
     KEY, QUERY = 58, 59
     t = planted(cfg, random_model(cfg, 19), KEY, QUERY)
@@ -386,6 +386,9 @@ ODD = {
                                        mlp={"kind": "moe", "router": {"experts": 5, "top": 4}, "expert": {"ff": 20}, "shared": {"ff": 36}})], width=120, loop=(0, 2, 2)),
     "odd_width": dict(layers=[layer(l=left(heads=3, kv_heads=1, dim=6, vdim=5, size=9, dims=2), r=right(heads=2, dim=5, vdim=9), mlp={"kind": "dense", "ff": 33, "limit": 0.9}),
                               layer(mlp={"kind": "moe", "router": {"experts": 3, "top": 2}, "expert": {"ff": 15}, "shared": {"ff": 11}})], width=62),
+    "wide_groups": dict(layers=[layer(l=left(heads=8, kv_heads=1, dim=32, vdim=64, size=13, dims=32), r=right(heads=2, dim=16, vdim=16), mlp=None),
+                                layer(l=left(heads=16, kv_heads=1, dim=16, vdim=16, size=150, dims=4), r=right(heads=1, dim=8, vdim=128), mlp=None),
+                                layer(l=left(heads=8, kv_heads=2, dim=256, vdim=32, size=21, dims=0, scale=0.08), mlp=None)], width=96),
     "wide_heads": dict(layers=[layer(l=left(heads=2, kv_heads=1, dim=128, vdim=128, size=17, dims=64, scale=0.09), r=right(heads=1, dim=256, vdim=256)),
                                layer(l=left(heads=2, kv_heads=2, dim=64, vdim=256, size=8, dims=32, scale=0.12), r=right(heads=2, dim=64, vdim=384))], width=128),
 }
@@ -668,5 +671,6 @@ def test_planted_keys_at_chunk_edges_on_the_tensor_cores():
             outs[at] = want[-1]
             assert err(m.forward_rows(ids[None], 0, [n - 1]), want[-1:]) < BF16_BAR, ("prompt", n, at)
             assert err(portions(m, ids, [n - 20, 20])[-1:], want[-1:]) < BF16_BAR, ("portion", n, at)
+            assert err(portions(m, ids, [n - 1, 1])[-1:], want[-1:]) < BF16_BAR, ("decoded", n, at)
         assert err(outs[start], outs[start - 1]) > 0.3
     m.close()
